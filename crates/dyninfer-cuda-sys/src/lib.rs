@@ -207,6 +207,17 @@ unsafe extern "C" {
         out_token: *mut i64,
         want_logits: c_int,
     ) -> c_int;
+    pub fn dyninfer_cuda_session_invoke_portion(
+        session: *mut dyninfer_cuda_session_t,
+        tokens: *const i64,
+        count: usize,
+        start_pos: i64,
+        slot: i64,
+        want: *const i64,
+        want_count: usize,
+        out_logits: *mut *mut f32,
+        out_token: *mut i64,
+    ) -> c_int;
     pub fn dyninfer_cuda_session_decode_batch(
         session: *mut dyninfer_cuda_session_t,
         tokens: *const i64,

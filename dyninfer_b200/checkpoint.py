@@ -25,6 +25,8 @@ import os
 import struct
 from dataclasses import dataclass, field
 
+from . import zupudra
+
 # ggml type code -> (encoding id, elements per block, bytes per block)
 GGML_TYPES = {
     0: ("plain.f32", 1, 4),
@@ -48,7 +50,7 @@ GGML_SCHEMA_ONLY = {
 }
 
 ST_DTYPES = {"F32": ("plain.f32", 4), "F16": ("plain.f16", 2), "BF16": ("plain.bf16", 2),
-             "U32": ("u32", 4), "I64": ("i64", 8), "U8": ("u8", 1)}
+             "U32": ("u32", 4), "I32": ("i32", 4), "I64": ("i64", 8), "U8": ("u8", 1)}
 
 PARAMETER_SCOPE = "weights"
 
@@ -424,8 +426,49 @@ def catalog_from_mlx(path: str) -> Catalog:
     return Catalog(idx.files, cfg, params)
 
 
+def catalog_from_listed_layers(path: str, reader) -> Catalog:
+    """A directory (or its model.safetensors) of an architecture whose reader gives the configuration and the
+    tensor names; tensors are plain, every one the configuration calls for must be there."""
+    st = os.path.join(path, "model.safetensors") if os.path.isdir(path) else path
+    with open(os.path.join(os.path.dirname(st), "config.json")) as f:
+        doc = json.load(f)
+    idx = index_safetensors(st)
+    try:
+        cfg, names = reader.config(doc), reader.tensor_names(doc)
+    except (KeyError, TypeError, ValueError) as e:
+        raise CheckpointError(f"{reader.ARCHITECTURE} config.json: {e!r}") from e
+    params = {}
+    for name, canon in names.items():
+        e = idx.entries.get(name)
+        if e is None:
+            raise CheckpointError(f"{reader.ARCHITECTURE} checkpoint lacks tensor {name}")
+        params[canon] = Parameter(canon, e.type_name, e.shape,
+                                  [Component("data", name, e.type_name, e.shape, 0, e.offset, e.nbytes)])
+    return Catalog(idx.files, cfg, params)
+
+
+# config.json "architecture" -> reader; directories without the key follow the HF / MLX convention
+ARCHITECTURES = {zupudra.ARCHITECTURE: zupudra}
+
+
+def _architecture_reader(path: str):
+    cj = os.path.join(path if os.path.isdir(path) else os.path.dirname(path), "config.json")
+    if not os.path.exists(cj):
+        return None
+    with open(cj) as f:
+        arch = json.load(f).get("architecture")
+    if arch is None:
+        return None
+    if arch not in ARCHITECTURES:
+        raise CheckpointError(f"unknown architecture `{arch}` (known: {', '.join(sorted(ARCHITECTURES))})")
+    return ARCHITECTURES[arch]
+
+
 def open_catalog(path: str) -> Catalog:
     if os.path.isdir(path) or path.endswith(".safetensors"):
+        reader = _architecture_reader(path)
+        if reader is not None:
+            return catalog_from_listed_layers(path, reader)
         return catalog_from_mlx(path)
     return catalog_from_gguf(path)
 

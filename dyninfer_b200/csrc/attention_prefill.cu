@@ -78,6 +78,7 @@ struct FaArgs {
   float* ctx;         // [rows, nh * d]
   int64_t rows, nh, nkv, cap, base_pos, seq;
   int64_t ldq;        // floats between consecutive rows of q
+  float scale;
 };
 
 template <int KV, int HALVES>
@@ -98,7 +99,7 @@ __global__ void __launch_bounds__(fa_threads(HALVES)) attention_prefill_kernel(c
   const int64_t r0 = row_lo + g, r1 = r0 + 8;      // the lane's two rows
   const int64_t r0c = r0 < a.rows ? r0 : a.rows - 1, r1c = r1 < a.rows ? r1 : a.rows - 1;
   const int64_t pos0 = a.base_pos + r0, pos1 = a.base_pos + r1;
-  const float scale = 1.0f / sqrtf((float)FA_D);
+  const float scale = a.scale;
 
   // Q fragments (hi, lo) for the 8 k-steps over the head dim
   uint32_t qh[8][4], ql[8][4];
@@ -279,6 +280,7 @@ int launch_attention_prefill(const AttnArgs& a, int64_t base_pos, int64_t seq, c
   f.q = a.q, f.kcache = a.kcache, f.vcache = a.vcache, f.ctx = a.ctx;
   f.rows = a.rows, f.nh = a.nh, f.nkv = a.nkv, f.cap = a.cap, f.base_pos = base_pos, f.seq = seq;
   f.ldq = a.ldq ? a.ldq : a.nh * FA_D;
+  f.scale = a.scale != 0.f ? a.scale : 1.0f / sqrtf((float)FA_D);
   const dim3 grid((unsigned)a.nh, (unsigned)((a.rows + FA_BR - 1) / FA_BR));
   // a grid that fits the GPU in one round: eight warps and pairs of key blocks; larger: four warps, two CTAs per SM
   const bool pairs = (int64_t)grid.x * grid.y <= std::max(1, sm_count());

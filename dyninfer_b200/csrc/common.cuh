@@ -334,6 +334,7 @@ struct AttnArgs {
   // row_pos / row_seq are given (prefill chunks); lets the tensor-core prefill kernel take them
   int64_t uniform_base = -1, uniform_seq = 0;
   int64_t ldq = 0;  // floats between consecutive rows of q (0: dense, nh*d)
+  float scale = 0.f;  // score factor of the tensor-core prefill kernel (0: 1/sqrt(d))
 };
 int launch_attention(const AttnArgs& a, cudaStream_t s);
 size_t attention_split_scratch_bytes(int64_t rows, int64_t nh, int64_t d, int nsplit);

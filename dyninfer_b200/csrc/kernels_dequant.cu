@@ -50,8 +50,26 @@ int launch_dequant(const WRef& w, float* out, cudaStream_t s) {
   return 0;
 }
 
+// Plain rows whose width is not a multiple of the decoders' four elements.
+__global__ void __launch_bounds__(256)
+gather_plain_kernel(WRef w, const int64_t* __restrict__ row_index, int64_t count, float* __restrict__ out) {
+  const int64_t total = count * w.cols;
+  for (int64_t it = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; it < total; it += (int64_t)gridDim.x * blockDim.x) {
+    int64_t src = row_index[it / w.cols];
+    if (src < 0 || src >= w.rows) src = 0;
+    out[it] = aux_load(w.data, w.enc, src * w.cols + it % w.cols);
+  }
+}
+
 int launch_gather(const WRef& w, const int64_t* tokens, int64_t count, float* out,
                   cudaStream_t s) {
+  if ((w.enc == E_F32 || w.enc == E_F16 || w.enc == E_BF16) && w.cols % 4) {
+    const int64_t blocks = (count * w.cols + 255) / 256;
+    gather_plain_kernel<<<(unsigned)(blocks > 148 * 32 ? 148 * 32 : blocks), 256, 0, s>>>(w, tokens, count, out);
+    count_launch();
+    DYN_CUDA(cudaGetLastError());
+    return 0;
+  }
   DYN_ENC_SWITCH(w.enc, return run_dequant<ENC>(w, tokens, count, out, s));
   return 0;
 }

@@ -7,6 +7,7 @@
 // sums are combined with warp shuffles. Up to MT activation rows share one
 // pass over the weights.
 #include "codec.cuh"
+#include "mixers.cuh"
 
 namespace dyn {
 
@@ -118,6 +119,26 @@ static int run_linear(const WRef& w, const void* x, int64_t m, float* y, const f
   return 0;
 }
 
+static bool plain_type(int enc) { return enc == E_F32 || enc == E_F16 || enc == E_BF16; }
+
+int launch_linear_exact(const WRef& w, const void* x, int x_type, int64_t m, float* y, const float* residual,
+                        cudaStream_t s) {
+  DYN_CHECK(x_type == E_F32 || x_type == E_BF16, "linear: x_type must be f32 or bf16, got %d", x_type);
+  DYN_CHECK(m >= 1, "linear: m must be >= 1");
+  if (m <= 4 && (w.enc == E_BF16 || w.enc == E_F16)) {
+    bool handled = false;
+    if (launch_gemv_plain(w, x, x_type, (int)m, y, residual, s, &handled)) return 1;
+    if (handled) return 0;
+  }
+  if (plain_type(w.enc) && (m > 8 || w.cols % 4)) return launch_gemm_f32(w, x, x_type, m, y, residual, s);
+  if (x_type == E_BF16) {
+    DYN_ENC_SWITCH(w.enc, return (run_linear<ENC, true>(w, x, m, y, residual, s)));
+  } else {
+    DYN_ENC_SWITCH(w.enc, return (run_linear<ENC, false>(w, x, m, y, residual, s)));
+  }
+  return 0;
+}
+
 int launch_linear(const WRef& w, const void* x, int x_type, int64_t m, float* y,
                   const float* residual, cudaStream_t s) {
   DYN_CHECK(x_type == E_F32 || x_type == E_BF16, "linear: x_type must be f32 or bf16, got %d",
@@ -134,6 +155,9 @@ int launch_linear(const WRef& w, const void* x, int x_type, int64_t m, float* y,
     if (launch_dqgemm_tc(w, x, x_type, m, y, residual, s, &handled)) return 1;
     if (handled) return 0;
   }
+  // plain weights of shapes no other kernel takes: rows that are not whole groups of four, or many rows of a
+  // width the tensor-core GEMM refuses
+  if (plain_type(w.enc) && (w.cols % 4 || m > 16)) return launch_gemm_f32(w, x, x_type, m, y, residual, s);
   if (m <= 4 && (w.enc == E_BF16 || w.enc == E_F16)) {
     // plain 2-byte weights (a tied bf16 embedding table as lm_head): streaming kernel
     bool handled = false;

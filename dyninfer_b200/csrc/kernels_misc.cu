@@ -2,6 +2,7 @@
 #include <math.h>
 
 #include "common.cuh"
+#include "mixers.cuh"
 
 namespace dyn {
 
@@ -40,11 +41,11 @@ __device__ __forceinline__ float block_sum(float v, float* smem) {
 // in both forms.
 template <int PER>
 __global__ void __launch_bounds__(256)
-rms_norm_kernel(const float* x, const void* __restrict__ w, int w_type, int64_t width, float eps,
-                float* y) {
+rms_norm_kernel(const float* x, const int64_t* __restrict__ index, const void* __restrict__ w, int w_type, int64_t width,
+                float eps, float* y) {
   __shared__ float red[32];
   pdl_trigger();  // a product launched next may begin fetching its weights
-  const float* xr = x + (int64_t)blockIdx.x * width;
+  const float* xr = x + (index ? index[blockIdx.x] : (int64_t)blockIdx.x) * width;
   float* yr = y + (int64_t)blockIdx.x * width;
   float ss = 0.f;
   if (PER > 0) {
@@ -82,16 +83,21 @@ rms_norm_kernel(const float* x, const void* __restrict__ w, int w_type, int64_t 
 
 int launch_rms_norm(const float* x, const void* w, int w_type, int64_t rows, int64_t width,
                     float eps, float* y, cudaStream_t s) {
+  return launch_rms_norm_indexed(x, nullptr, w, w_type, rows, width, eps, y, s);
+}
+
+int launch_rms_norm_indexed(const float* x, const int64_t* index, const void* w, int w_type, int64_t rows,
+                            int64_t width, float eps, float* y, cudaStream_t s) {
   if (rows == 0) return 0;
   const int threads = width >= 1024 ? 256 : (width >= 256 ? 128 : 32);
   if (width <= 8 * threads) {
-    rms_norm_kernel<8><<<(unsigned)rows, threads, 0, s>>>(x, w, w_type, width, eps, y);
+    rms_norm_kernel<8><<<(unsigned)rows, threads, 0, s>>>(x, index, w, w_type, width, eps, y);
   } else if (width <= 16 * threads) {
-    rms_norm_kernel<16><<<(unsigned)rows, threads, 0, s>>>(x, w, w_type, width, eps, y);
+    rms_norm_kernel<16><<<(unsigned)rows, threads, 0, s>>>(x, index, w, w_type, width, eps, y);
   } else if (width <= 32 * threads) {
-    rms_norm_kernel<32><<<(unsigned)rows, threads, 0, s>>>(x, w, w_type, width, eps, y);
+    rms_norm_kernel<32><<<(unsigned)rows, threads, 0, s>>>(x, index, w, w_type, width, eps, y);
   } else {
-    rms_norm_kernel<0><<<(unsigned)rows, threads, 0, s>>>(x, w, w_type, width, eps, y);
+    rms_norm_kernel<0><<<(unsigned)rows, threads, 0, s>>>(x, index, w, w_type, width, eps, y);
   }
   count_launch();
   DYN_CUDA(cudaGetLastError());

@@ -1,0 +1,401 @@
+// Retention: linear attention with a fixed decay per head, no softmax and no denominator.
+//
+// Decode rows: one cluster per (head, row). A CTA of the cluster owns a slice of the value columns of
+// the head's state: it rotates q and k, updates its part of S in place (one read, one write of the f32
+// state: the kernel is bound by that traffic) and forms its part of o = S^T q; the squared sums of the
+// slices meet through distributed shared memory, so norm and gate are applied in the same launch.
+//
+// Portions: chunks of 64 tokens, all chunks at once.
+//   U_c = sum_{t in c} decay^{last - t} k_t v_t^T        (retention_chunk_state_kernel)
+//   P_c = state before chunk c, by a scan over the U_c     (retention_scan_kernel; leaves the new state)
+//   o_t = sum_{s <= t, s in c} decay^{t-s} (q_t . k_s) v_s + decay^{t+1-first} P_c^T q_t, then norm and
+//   gate                                                   (retention_chunk_out_kernel)
+// All of it in f32 on the vector pipes: scores, decays and states are 32-bit quantities.
+#include <cooperative_groups.h>
+
+#include <algorithm>
+
+#include "mixers.cuh"
+
+namespace cg = cooperative_groups;
+
+namespace dyn {
+namespace {
+
+constexpr int RT_C = 64;      // tokens per chunk
+constexpr int RT_PITCH = RT_C + 4;
+constexpr int RT_SLICE = 32;  // reduction elements staged at a time
+
+// The angle of a position, reduced in double precision: p * f is far from 0 for long contexts.
+__device__ __forceinline__ void sincos_position(int64_t pos, double freq, float* sv, float* cv) {
+  const double turns = (double)pos * freq * 0.15915494309189535;  // 1 / 2 pi
+  const double frac = turns - rint(turns);
+  sincospif((float)(2.0 * frac), sv, cv);
+}
+
+__device__ __forceinline__ void load4(float* dst, const float* src) {  // src 16-byte aligned
+  const float4 v = *reinterpret_cast<const float4*>(src);
+  dst[0] = v.x, dst[1] = v.y, dst[2] = v.z, dst[3] = v.w;
+}
+
+__device__ __forceinline__ float silu_of(float z) { return z / (1.0f + expf(-z)); }
+
+// ---- decode: independent rows ----------------------------------------------------------------
+__global__ void __launch_bounds__(256) retention_step_kernel(RetentionArgs a, const int64_t* row_pos,
+                                                             const int64_t* row_seq, int64_t pos0, int64_t seq0,
+                                                             int64_t row0) {
+  extern __shared__ float rs_smem[];
+  __shared__ float part_ss, red_ss[8];
+  const cg::cluster_group cl = cg::this_cluster();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int D = a.dim, E = a.vdim, nsplit = gridDim.x;
+  const int h = blockIdx.y;
+  const int64_t r = row0 + blockIdx.z;
+  const int per = (E + nsplit - 1) / nsplit, e0 = min((int)blockIdx.x * per, E), ne = min(per, E - e0);
+  float* qs = rs_smem;           // [D]
+  float* ks = qs + D;            // [D]
+  float* red = ks + D;           // [8][per]
+  float* os = red + 8 * per;     // [per]
+  const int64_t pos = row_pos ? row_pos[r] : pos0, seq = row_seq ? row_seq[r] : seq0;
+  const float decay = a.decay[h], kscale = 1.0f / sqrtf((float)D);
+  const float* q = a.q.ptr + r * a.q.ld + (int64_t)h * D;
+  const float* k = a.k.ptr + r * a.k.ld + (int64_t)h * D;
+  const float* v = a.v.ptr + r * a.v.ld + (int64_t)h * E + e0;
+  pdl_trigger();
+  const int half = a.rot_dims / 2;
+  for (int i = tid; i < D; i += 256) {
+    if (i < half) {
+      float sv, cv;
+      sincos_position(pos, a.freq[i], &sv, &cv);
+      const float q0 = q[i], q1 = q[i + half], k0 = k[i], k1 = k[i + half];
+      qs[i] = q0 * cv - q1 * sv, qs[i + half] = q1 * cv + q0 * sv;
+      ks[i] = (k0 * cv - k1 * sv) * kscale, ks[i + half] = (k1 * cv + k0 * sv) * kscale;
+    } else if (i >= 2 * half) {
+      qs[i] = q[i], ks[i] = k[i] * kscale;
+    }
+  }
+  __syncthreads();
+  float* S = a.state + ((seq * a.heads + h) * D) * (int64_t)E + e0;
+  for (int c = lane; c < ne; c += 32) {
+    const float vv = v[c];
+    float acc = 0.f;
+    for (int d0 = warp; d0 < D; d0 += 64) {  // eight rows of the state in flight per thread
+      float s[8];
+#pragma unroll
+      for (int j = 0; j < 8; j++) s[j] = (d0 + 8 * j < D && pos > 0) ? S[(int64_t)(d0 + 8 * j) * E + c] : 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; j++) {
+        const int d = d0 + 8 * j;
+        if (d < D) {
+          const float n = fmaf(decay, s[j], ks[d] * vv);
+          S[(int64_t)d * E + c] = n;
+          acc = fmaf(n, qs[d], acc);
+        }
+      }
+    }
+    red[warp * per + c] = acc;
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < ne; c += 256) {
+    float o = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; w++) o += red[w * per + c];
+    os[c] = o;
+    ss = fmaf(o, o, ss);
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) red_ss[warp] = ss;
+  __syncthreads();
+  if (tid == 0) {
+    float t = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; w++) t += red_ss[w];
+    part_ss = t;
+  }
+  cl.sync();
+  float total = 0.f;
+  for (int i = 0; i < nsplit; i++) total += *cl.map_shared_rank(&part_ss, i);
+  cl.sync();  // nobody leaves while another CTA still reads its sum
+  const float inv = 1.0f / sqrtf(total / (float)E + a.eps);
+  const float* g = a.g.ptr + r * a.g.ld + (int64_t)h * E + e0;
+  float* out = a.out + r * (int64_t)a.heads * E + (int64_t)h * E + e0;
+  for (int c = tid; c < ne; c += 256) out[c] = os[c] * inv * silu_of(g[c]);
+}
+
+int step_rows(const RetentionArgs& a, const int64_t* pos, const int64_t* seq, int64_t pos0, int64_t seq0, int64_t row0,
+              int64_t rows, cudaStream_t st) {
+  int nsplit = 1;
+  while (nsplit < 8 && a.vdim / (nsplit * 2) >= 32) nsplit *= 2;
+  const int per = (a.vdim + nsplit - 1) / nsplit;
+  const size_t smem = (size_t)(2 * a.dim + 9 * per) * 4;
+  DYN_CHECK(smem <= 48 * 1024, "retention: head of %d x %d is too large", a.dim, a.vdim);
+  for (int64_t r0 = 0; r0 < rows; r0 += 65535) {
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = dim3((unsigned)nsplit, (unsigned)a.heads, (unsigned)std::min<int64_t>(65535, rows - r0));
+    cfg.blockDim = dim3(256);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr{};
+    attr.id = cudaLaunchAttributeClusterDimension;
+    attr.val.clusterDim.x = (unsigned)nsplit, attr.val.clusterDim.y = 1, attr.val.clusterDim.z = 1;
+    cfg.attrs = &attr, cfg.numAttrs = 1;
+    DYN_CUDA(cudaLaunchKernelEx(&cfg, retention_step_kernel, a, pos, seq, pos0, seq0, row0 + r0));
+    count_launch();
+  }
+  return 0;
+}
+
+// ---- portions ---------------------------------------------------------------------------------
+// q and k of a portion rotated in place (k also scaled): thread = (row, head, pair or passed dim).
+__global__ void __launch_bounds__(256) retention_rotate_kernel(RetentionArgs a, int64_t rows, int64_t base) {
+  const int half = a.rot_dims / 2, per = a.dim - half;  // pairs, then the dims that pass
+  const int64_t total = rows * a.heads * per;
+  const float kscale = 1.0f / sqrtf((float)a.dim);
+  for (int64_t it = blockIdx.x * 256ll + threadIdx.x; it < total; it += (int64_t)gridDim.x * 256) {
+    const int i = (int)(it % per);
+    const int64_t rh = it / per, h = rh % a.heads, r = rh / a.heads;
+    float* q = a.q.ptr + r * a.q.ld + h * a.dim;
+    float* k = a.k.ptr + r * a.k.ld + h * a.dim;
+    if (i < half) {
+      float sv, cv;
+      sincos_position(base + r, a.freq[i], &sv, &cv);
+      const float q0 = q[i], q1 = q[i + half], k0 = k[i], k1 = k[i + half];
+      q[i] = q0 * cv - q1 * sv, q[i + half] = q1 * cv + q0 * sv;
+      k[i] = (k0 * cv - k1 * sv) * kscale, k[i + half] = (k1 * cv + k0 * sv) * kscale;
+    } else {
+      k[i + half] *= kscale;
+    }
+  }
+}
+
+// U[c][h][d][e], one 64 x 64 tile of (d, e) per CTA.
+__global__ void __launch_bounds__(64) retention_chunk_state_kernel(RetentionArgs a, int64_t rows) {
+  __shared__ __align__(16) float ks[RT_C][64], vs[RT_C][64];
+  const int tid = threadIdx.x, tx = tid & 7, ty = tid >> 3;
+  const int D = a.dim, E = a.vdim, et = (E + 63) / 64;
+  const int64_t c = blockIdx.x, t0 = c * RT_C;
+  const int h = blockIdx.y, d0 = (int)(blockIdx.z / et) * 64, e0 = (int)(blockIdx.z % et) * 64;
+  const int n = (int)min((int64_t)RT_C, rows - t0);
+  const float decay = a.decay[h];
+  for (int t = 0; t < n; t++) {
+    const float wt = powf(decay, (float)(n - 1 - t));
+    const float* kr = a.k.ptr + (t0 + t) * a.k.ld + (int64_t)h * D + d0;
+    const float* vr = a.v.ptr + (t0 + t) * a.v.ld + (int64_t)h * E + e0;
+    ks[t][tid] = d0 + tid < D ? kr[tid] * wt : 0.f;
+    vs[t][tid] = e0 + tid < E ? vr[tid] : 0.f;
+  }
+  __syncthreads();
+  float acc[8][8] = {};
+  for (int t = 0; t < n; t++) {
+    float kv[8], vv[8];
+    load4(kv, &ks[t][4 * ty]);
+    load4(kv + 4, &ks[t][32 + 4 * ty]);
+    load4(vv, &vs[t][4 * tx]);
+    load4(vv + 4, &vs[t][32 + 4 * tx]);
+#pragma unroll
+    for (int i = 0; i < 8; i++)
+#pragma unroll
+      for (int j = 0; j < 8; j++) acc[i][j] = fmaf(kv[i], vv[j], acc[i][j]);
+  }
+  float* U = a.scratch + ((c * a.heads + h) * D) * (int64_t)E;
+#pragma unroll
+  for (int i = 0; i < 8; i++) {
+    const int d = d0 + (i < 4 ? 4 * ty + i : 28 + 4 * ty + i);
+    if (d >= D) continue;
+#pragma unroll
+    for (int j = 0; j < 8; j++) {
+      const int e = e0 + (j < 4 ? 4 * tx + j : 28 + 4 * tx + j);
+      if (e < E) U[(int64_t)d * E + e] = acc[i][j];
+    }
+  }
+}
+
+// U[c] -> state before chunk c; the slot's state -> state after the portion.
+__global__ void __launch_bounds__(256) retention_scan_kernel(RetentionArgs a, int64_t rows, int64_t base, int64_t slot) {
+  const int64_t per = (int64_t)a.dim * a.vdim, plane = a.heads * per;
+  const int64_t idx = blockIdx.x * 256ll + threadIdx.x;
+  if (idx >= plane) return;
+  const float decay = a.decay[idx / per];
+  const float full = powf(decay, (float)RT_C);
+  float* st = a.state + slot * plane + idx;
+  float S = base > 0 ? *st : 0.f;
+  const int64_t nc = (rows + RT_C - 1) / RT_C;
+  for (int64_t c0 = 0; c0 < nc; c0 += 8) {
+    float u[8];
+#pragma unroll
+    for (int j = 0; j < 8; j++) u[j] = c0 + j < nc ? a.scratch[(c0 + j) * plane + idx] : 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; j++) {
+      const int64_t c = c0 + j;
+      if (c >= nc) break;
+      a.scratch[c * plane + idx] = S;
+      const int64_t n = min((int64_t)RT_C, rows - c * RT_C);
+      S = fmaf(n == RT_C ? full : powf(decay, (float)n), S, u[j]);
+    }
+  }
+  *st = S;
+}
+
+// One (chunk, head) per CTA: scores, products with the values and with the state before the chunk,
+// norm and gate. EC = 64-column groups of the value dim.
+template <int EC>
+__global__ void __launch_bounds__(256) retention_chunk_out_kernel(RetentionArgs a, int64_t rows, int64_t base) {
+  extern __shared__ __align__(16) float ro_smem[];
+  constexpr int BP = EC * 64 + 4;
+  float(*Qt)[RT_PITCH] = reinterpret_cast<float(*)[RT_PITCH]>(ro_smem);                       // [slice][t]
+  float(*Kt)[RT_PITCH] = Qt + RT_SLICE;                                                        // [slice][s]
+  float(*At)[RT_PITCH] = Kt + RT_SLICE;                                                        // [s][t]
+  float(*Bs)[BP] = reinterpret_cast<float(*)[BP]>(At + RT_C);                                 // [slice][e]
+  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  const int D = a.dim, E = a.vdim;
+  const int64_t c = blockIdx.x, t0 = c * RT_C;
+  const int h = blockIdx.y;
+  const int n = (int)min((int64_t)RT_C, rows - t0);
+  const float decay = a.decay[h];
+  const float* qp = a.q.ptr + t0 * a.q.ld + (int64_t)h * D;
+  const float* kp = a.k.ptr + t0 * a.k.ld + (int64_t)h * D;
+  const float* vp = a.v.ptr + t0 * a.v.ld + (int64_t)h * E;
+  // ---- scores of the chunk, decayed and causal
+  {
+    float s[4][4] = {};
+    for (int d0 = 0; d0 < D; d0 += RT_SLICE) {
+#pragma unroll
+      for (int j = 0; j < RT_C * RT_SLICE / 256; j++) {
+        const int i = tid + 256 * j, t = i / RT_SLICE, d = i % RT_SLICE;
+        const bool live = t < n && d0 + d < D;
+        Qt[d][t] = live ? qp[t * a.q.ld + d0 + d] : 0.f;
+        Kt[d][t] = live ? kp[t * a.k.ld + d0 + d] : 0.f;
+      }
+      __syncthreads();
+#pragma unroll 8
+      for (int d = 0; d < RT_SLICE; d++) {
+        float qv[4], kv[4];
+        load4(qv, &Qt[d][4 * ty]);
+        load4(kv, &Kt[d][4 * tx]);
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+#pragma unroll
+          for (int j = 0; j < 4; j++) s[i][j] = fmaf(qv[i], kv[j], s[i][j]);
+      }
+      __syncthreads();
+    }
+#pragma unroll
+    for (int j = 0; j < 4; j++)
+#pragma unroll
+      for (int i = 0; i < 4; i++) {
+        const int t = 4 * ty + i, u = 4 * tx + j;
+        At[u][t] = u <= t ? s[i][j] * powf(decay, (float)(t - u)) : 0.f;
+      }
+  }
+  float o[4][EC * 4] = {};
+  auto accumulate = [&](float (*L)[RT_PITCH]) {
+#pragma unroll 8
+    for (int k = 0; k < RT_SLICE; k++) {
+      float av[4];
+      load4(av, &L[k][4 * ty]);
+#pragma unroll
+      for (int g = 0; g < EC; g++) {
+        float bv[4];
+        load4(bv, &Bs[k][64 * g + 4 * tx]);
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+#pragma unroll
+          for (int j = 0; j < 4; j++) o[i][4 * g + j] = fmaf(av[i], bv[j], o[i][4 * g + j]);
+      }
+    }
+  };
+  // ---- scores x values
+  for (int s0 = 0; s0 < n; s0 += RT_SLICE) {
+    for (int i = tid; i < RT_SLICE * EC * 64; i += 256) {
+      const int k = i / (EC * 64), e = i % (EC * 64);
+      Bs[k][e] = s0 + k < n && e < E ? vp[(s0 + k) * a.v.ld + e] : 0.f;
+    }
+    __syncthreads();  // also covers the scores' stores before the first use
+    accumulate(At + s0);
+    __syncthreads();
+  }
+  // ---- the state before the chunk
+  if (c > 0 || base > 0) {
+    const float* P = a.scratch + ((c * a.heads + h) * D) * (int64_t)E;
+    for (int d0 = 0; d0 < D; d0 += RT_SLICE) {
+#pragma unroll
+      for (int j = 0; j < RT_C * RT_SLICE / 256; j++) {
+        const int i = tid + 256 * j, t = i / RT_SLICE, d = i % RT_SLICE;
+        Qt[d][t] = t < n && d0 + d < D ? qp[t * a.q.ld + d0 + d] * powf(decay, (float)(t + 1)) : 0.f;
+      }
+      for (int i = tid; i < RT_SLICE * EC * 64; i += 256) {
+        const int k = i / (EC * 64), e = i % (EC * 64);
+        Bs[k][e] = d0 + k < D && e < E ? P[(int64_t)(d0 + k) * E + e] : 0.f;
+      }
+      __syncthreads();
+      accumulate(Qt);
+      __syncthreads();
+    }
+  }
+  // ---- norm over the head's value dims (columns past E hold zeros), gate
+#pragma unroll
+  for (int i = 0; i < 4; i++) {
+    const int t = 4 * ty + i;
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < EC * 4; j++) ss = fmaf(o[i][j], o[i][j], ss);
+#pragma unroll
+    for (int m = 8; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    if (t >= n) continue;
+    const float inv = 1.0f / sqrtf(ss / (float)E + a.eps);
+    const float* g = a.g.ptr + (t0 + t) * a.g.ld + (int64_t)h * E;
+    float* out = a.out + (t0 + t) * (int64_t)a.heads * E + (int64_t)h * E;
+#pragma unroll
+    for (int j = 0; j < EC * 4; j++) {
+      const int e = 64 * (j / 4) + 4 * tx + j % 4;
+      if (e < E) out[e] = o[i][j] * inv * silu_of(g[e]);
+    }
+  }
+}
+
+template <int EC>
+int chunk_out(const RetentionArgs& a, int64_t rows, int64_t base, cudaStream_t st) {
+  const int smem = (int)((2 * RT_SLICE + RT_C) * RT_PITCH + RT_SLICE * (EC * 64 + 4)) * 4;
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(retention_chunk_out_kernel<EC>), smem)) return 1;
+  retention_chunk_out_kernel<EC><<<dim3((unsigned)((rows + RT_C - 1) / RT_C), (unsigned)a.heads), 256, smem, st>>>(a, rows, base);
+  count_launch();
+  return 0;
+}
+
+bool chunked_shape(const RetentionArgs& a) { return a.vdim <= 256; }
+
+}  // namespace
+
+size_t retention_scratch_floats(const RetentionArgs& a, int64_t rows) {
+  return chunked_shape(a) ? (size_t)((rows + RT_C - 1) / RT_C) * a.heads * a.dim * a.vdim : 0;
+}
+
+int launch_retention(const RetentionArgs& a, const StepRows& r, cudaStream_t st) {
+  if (r.rows == 0) return 0;
+  if (r.base < 0) return step_rows(a, r.pos, r.seq, 0, 0, 0, r.rows, st);
+  if (r.rows == 1) return step_rows(a, nullptr, nullptr, r.base, r.slot, 0, 1, st);
+  if (!chunked_shape(a)) {  // wide value heads: token by token
+    for (int64_t i = 0; i < r.rows; i++)
+      if (step_rows(a, nullptr, nullptr, r.base + i, r.slot, i, 1, st)) return 1;
+    return 0;
+  }
+  const unsigned nc = (unsigned)((r.rows + RT_C - 1) / RT_C);
+  {
+    const int64_t total = r.rows * a.heads * (a.dim - a.rot_dims / 2);
+    retention_rotate_kernel<<<(unsigned)std::min<int64_t>((total + 255) / 256, 148 * 16), 256, 0, st>>>(a, r.rows, r.base);
+    const unsigned tiles = (unsigned)(((a.dim + 63) / 64) * ((a.vdim + 63) / 64));
+    retention_chunk_state_kernel<<<dim3(nc, (unsigned)a.heads, tiles), 64, 0, st>>>(a, r.rows);
+    const int64_t plane = (int64_t)a.heads * a.dim * a.vdim;
+    retention_scan_kernel<<<(unsigned)((plane + 255) / 256), 256, 0, st>>>(a, r.rows, r.base, r.slot);
+    count_launch(3);
+  }
+  const int ec = (a.vdim + 63) / 64;
+  if (ec == 1 ? chunk_out<1>(a, r.rows, r.base, st) : ec == 2 ? chunk_out<2>(a, r.rows, r.base, st)
+                                                            : chunk_out<4>(a, r.rows, r.base, st))
+    return 1;
+  DYN_CUDA(cudaGetLastError());
+  return 0;
+}
+
+}  // namespace dyn

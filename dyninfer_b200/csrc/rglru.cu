@@ -1,0 +1,267 @@
+// Gated linear recurrence behind a short causal convolution: two input branches x (recurrent) and y
+// (gate), block-diagonal recurrence and input gates, a diagonal f32 state per channel.
+//
+// The convolution's inputs live in a ring of `taps` rows per slot, position p in row p mod taps, so a
+// decode step writes its own row while other CTAs still read the rows before it. Positions before the
+// sequence start count as zeros and are never read.
+//
+// Decode rows: one launch per layer. A CTA takes 32 outputs of one gate block: it forms the block's
+// convolution outputs (a few multiplies, repeated by the block's CTAs), then a warp per output reads
+// the two gate rows and updates the state.
+// Portions: convolution -> gates (a tiled block-diagonal product whose epilogue leaves a_t and the
+// increment b_t) -> scan. The scan handles 512 tokens x 32 channels per CTA and pass: a warp composes
+// the maps S -> A S + B of its 16 tokens, the 32 segment maps are chained through shared memory, and
+// each warp replays its tokens from its start state.
+#include <algorithm>
+
+#include "mixers.cuh"
+
+namespace dyn {
+namespace {
+
+__device__ __forceinline__ float vec_at(const Vec& v, int64_t i) { return aux_load(v.ptr, v.type, i); }
+__device__ __forceinline__ float sigmoid_of(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus_of(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float gelu_tanh_of(float z) {
+  return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+// gate sums -> (a, sqrt(1 - a^2) i u); 1 - a^2 from the logarithm, without cancellation near a = 1
+__device__ __forceinline__ void recurrence_terms(float rz, float iz, float u, float c, float lam, float* a, float* b) {
+  const float la = -c * sigmoid_of(rz) * softplus_of(lam);
+  *a = expf(la);
+  *b = sqrtf(-expm1f(2.0f * la)) * sigmoid_of(iz) * u;
+}
+
+// ---- decode rows -----------------------------------------------------------------------------
+constexpr int RG_OUT = 32;
+
+// dot(w[row][0..n), u) over the warp; consecutive lanes read consecutive 8-element pieces when they can
+template <bool WIDE>
+__device__ __forceinline__ void two_dots(const RglruArgs& a, int64_t row, int n, const float* u, int lane, float* r, float* i) {
+  float sr = 0.f, si = 0.f;
+  if (WIDE) {  // bf16 rows of a multiple of 8, 16-byte aligned
+    const uint4* wr = reinterpret_cast<const uint4*>(a.ra.ptr + row * n * 2);
+    const uint4* wi = reinterpret_cast<const uint4*>(a.ri.ptr + row * n * 2);
+    for (int p = lane; p < n / 8; p += 32) {
+      const uint4 x = wr[p], y = wi[p];
+      const uint32_t xw[4] = {x.x, x.y, x.z, x.w}, yw[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const float u0 = u[8 * p + 2 * e], u1 = u[8 * p + 2 * e + 1];
+        sr = fmaf(__uint_as_float(xw[e] << 16), u0, sr), sr = fmaf(__uint_as_float(xw[e] & 0xffff0000u), u1, sr);
+        si = fmaf(__uint_as_float(yw[e] << 16), u0, si), si = fmaf(__uint_as_float(yw[e] & 0xffff0000u), u1, si);
+      }
+    }
+  } else {
+    for (int k = lane; k < n; k += 32) {
+      sr = fmaf(vec_at(a.ra, row * n + k), u[k], sr);
+      si = fmaf(vec_at(a.ri, row * n + k), u[k], si);
+    }
+  }
+  *r = warp_sum(sr), *i = warp_sum(si);
+}
+
+template <bool WIDE>
+__global__ void __launch_bounds__(256) rglru_step_kernel(RglruArgs a, const int64_t* row_pos, const int64_t* row_seq,
+                                                         int64_t pos0, int64_t seq0, int64_t row0) {
+  extern __shared__ float u_s[];  // [width / blocks]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int n = a.width / a.blocks, slices = (n + RG_OUT - 1) / RG_OUT;
+  const int blk = blockIdx.x / slices, slice = blockIdx.x % slices;
+  const int64_t r = row0 + blockIdx.y;
+  const int64_t pos = row_pos ? row_pos[r] : pos0, seq = row_seq ? row_seq[r] : seq0;
+  float* ring = a.ring + seq * (int64_t)a.taps * a.width;
+  const float* x = a.x.ptr + r * a.x.ld;
+  pdl_trigger();
+  for (int c = tid; c < n; c += 256) {
+    const int64_t ch = (int64_t)blk * n + c;
+    const float xin = x[ch] + vec_at(a.bx, ch);
+    float u = vec_at(a.conv, ch * a.taps + a.taps - 1) * xin;
+    for (int j = 1; j < a.taps; j++)
+      if (pos >= j) u = fmaf(vec_at(a.conv, ch * a.taps + a.taps - 1 - j), ring[((pos - j) % a.taps) * a.width + ch], u);
+    u_s[c] = u + vec_at(a.bc, ch);
+    if (slice == 0) ring[(pos % a.taps) * a.width + ch] = xin;
+  }
+  __syncthreads();
+  for (int o = slice * RG_OUT + warp; o < min(n, (slice + 1) * RG_OUT); o += 8) {
+    const int64_t ch = (int64_t)blk * n + o;
+    float rz, iz;
+    two_dots<WIDE>(a, ch, n, u_s, lane, &rz, &iz);
+    if (lane == 0) {
+      float av, bv;
+      recurrence_terms(rz + vec_at(a.bra, ch), iz + vec_at(a.bri, ch), u_s[o], a.c, vec_at(a.lam, ch), &av, &bv);
+      float* S = a.state + seq * a.width + ch;
+      const float s = pos > 0 ? fmaf(av, *S, bv) : bv;
+      *S = s;
+      a.out[r * a.width + ch] = s * gelu_tanh_of(a.y.ptr[r * a.y.ld + ch] + vec_at(a.by, ch));
+    }
+  }
+}
+
+bool wide_rows(const RglruArgs& a) {
+  const int n = a.width / a.blocks;
+  auto ok = [&](const Vec& v) { return v.type == E_BF16 && (reinterpret_cast<uintptr_t>(v.ptr) & 15) == 0; };
+  return n % 8 == 0 && ok(a.ra) && ok(a.ri);
+}
+
+int step_rows(const RglruArgs& a, const int64_t* pos, const int64_t* seq, int64_t pos0, int64_t seq0, int64_t row0,
+              int64_t rows, cudaStream_t st) {
+  const int n = a.width / a.blocks, slices = (n + RG_OUT - 1) / RG_OUT;
+  const size_t smem = (size_t)n * 4;
+  DYN_CHECK(smem <= 48 * 1024, "rglru: a gate block of %d channels is too large", n);
+  for (int64_t r0 = 0; r0 < rows; r0 += 65535) {
+    const dim3 grid((unsigned)(a.blocks * slices), (unsigned)std::min<int64_t>(65535, rows - r0));
+    if (wide_rows(a))
+      rglru_step_kernel<true><<<grid, 256, smem, st>>>(a, pos, seq, pos0, seq0, row0 + r0);
+    else
+      rglru_step_kernel<false><<<grid, 256, smem, st>>>(a, pos, seq, pos0, seq0, row0 + r0);
+    count_launch();
+  }
+  DYN_CUDA(cudaGetLastError());
+  return 0;
+}
+
+// ---- portions ---------------------------------------------------------------------------------
+// u[t][ch]; inputs from before the portion come from the ring.
+__global__ void __launch_bounds__(256) rglru_conv_kernel(RglruArgs a, int64_t rows, int64_t base, int64_t slot, float* __restrict__ u) {
+  const int ch = blockIdx.x * 256 + threadIdx.x;
+  if (ch >= a.width) return;
+  const float* ring = a.ring + slot * (int64_t)a.taps * a.width;
+  const float bx = vec_at(a.bx, ch), bc = vec_at(a.bc, ch);
+  const int64_t t = blockIdx.y;
+  float acc = 0.f;
+  for (int j = 0; j < a.taps; j++) {
+    const float w = vec_at(a.conv, (int64_t)ch * a.taps + a.taps - 1 - j);
+    if (j <= t)
+      acc = fmaf(w, a.x.ptr[(t - j) * a.x.ld + ch] + bx, acc);
+    else if (base + t >= j)
+      acc = fmaf(w, ring[((base + t - j) % a.taps) * a.width + ch], acc);
+  }
+  u[t * a.width + ch] = acc + bc;
+}
+
+// Gates of 128 tokens x 64 outputs of one block, f32: both products share the u tile.
+constexpr int GG_M = 128, GG_N = 64, GG_K = 16;
+__global__ void __launch_bounds__(256)
+rglru_gates_kernel(RglruArgs a, int64_t rows, const float* __restrict__ u, float* __restrict__ av, float* __restrict__ bv) {
+  __shared__ __align__(16) float us[GG_K][GG_M + 4], rs[GG_K][GG_N + 4], is[GG_K][GG_N + 4];
+  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  const int n = a.width / a.blocks, tiles = (n + GG_N - 1) / GG_N;
+  const int blk = blockIdx.x / tiles, o0 = (blockIdx.x % tiles) * GG_N;
+  const int64_t t0 = (int64_t)blockIdx.y * GG_M;
+  float ar[8][4] = {}, ai[8][4] = {};
+  for (int k0 = 0; k0 < n; k0 += GG_K) {
+#pragma unroll
+    for (int j = 0; j < GG_M * GG_K / 256; j++) {
+      const int i = tid + 256 * j, t = i / GG_K, k = i % GG_K;
+      us[k][t] = t0 + t < rows && k0 + k < n ? u[(t0 + t) * a.width + blk * n + k0 + k] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < GG_N * GG_K / 256; j++) {
+      const int i = tid + 256 * j, o = i / GG_K, k = i % GG_K;
+      const bool live = o0 + o < n && k0 + k < n;
+      const int64_t at = ((int64_t)blk * n + o0 + o) * n + k0 + k;
+      rs[k][o] = live ? vec_at(a.ra, at) : 0.f;
+      is[k][o] = live ? vec_at(a.ri, at) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < GG_K; k++) {
+      const float4 x0 = *reinterpret_cast<const float4*>(&us[k][4 * ty]), x1 = *reinterpret_cast<const float4*>(&us[k][64 + 4 * ty]);
+      const float4 r4 = *reinterpret_cast<const float4*>(&rs[k][4 * tx]), i4 = *reinterpret_cast<const float4*>(&is[k][4 * tx]);
+      const float xv[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+      const float rv[4] = {r4.x, r4.y, r4.z, r4.w}, iv[4] = {i4.x, i4.y, i4.z, i4.w};
+#pragma unroll
+      for (int i = 0; i < 8; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) ar[i][j] = fmaf(xv[i], rv[j], ar[i][j]), ai[i][j] = fmaf(xv[i], iv[j], ai[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int j = 0; j < 4; j++) {
+    const int o = o0 + 4 * tx + j;
+    if (o >= n) continue;
+    const int64_t ch = (int64_t)blk * n + o;
+    const float br = vec_at(a.bra, ch), bi = vec_at(a.bri, ch), lam = vec_at(a.lam, ch);
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+      const int64_t t = t0 + (i < 4 ? 4 * ty + i : 60 + 4 * ty + i);
+      if (t >= rows) continue;
+      recurrence_terms(ar[i][j] + br, ai[i][j] + bi, u[t * a.width + ch], a.c, lam, &av[t * a.width + ch], &bv[t * a.width + ch]);
+    }
+  }
+}
+
+constexpr int SC_SEG = 32, SC_LEN = 16, SC_PASS = SC_SEG * SC_LEN;
+__global__ void __launch_bounds__(1024)
+rglru_scan_kernel(RglruArgs a, int64_t rows, int64_t base, int64_t slot, const float* __restrict__ av, const float* __restrict__ bv) {
+  __shared__ float sA[SC_SEG][32], sB[SC_SEG][32];
+  const int lane = threadIdx.x & 31, seg = threadIdx.x >> 5;
+  const int ch = blockIdx.x * 32 + lane;
+  const bool live = ch < a.width;
+  float S0 = live && base > 0 ? a.state[slot * a.width + ch] : 0.f;  // state before the pass
+  const float by = live ? vec_at(a.by, ch) : 0.f;
+  for (int64_t p0 = 0; p0 < rows; p0 += SC_PASS) {
+    const int64_t t0 = p0 + seg * SC_LEN;
+    float x[SC_LEN], y[SC_LEN];
+#pragma unroll
+    for (int i = 0; i < SC_LEN; i++) {
+      const bool in = live && t0 + i < rows;
+      x[i] = in ? av[(t0 + i) * a.width + ch] : 1.f;
+      y[i] = in ? bv[(t0 + i) * a.width + ch] : 0.f;
+    }
+    float A = 1.f, B = 0.f;
+#pragma unroll
+    for (int i = 0; i < SC_LEN; i++) B = fmaf(x[i], B, y[i]), A *= x[i];
+    sA[seg][lane] = A, sB[seg][lane] = B;
+    __syncthreads();
+    float S = S0;
+    for (int w = 0; w < SC_SEG; w++) {
+      const float n = fmaf(sA[w][lane], S0, sB[w][lane]);
+      if (w < seg) S = n;
+      S0 = n;
+    }
+#pragma unroll
+    for (int i = 0; i < SC_LEN; i++) {
+      S = fmaf(x[i], S, y[i]);
+      if (live && t0 + i < rows)
+        a.out[(t0 + i) * a.width + ch] = S * gelu_tanh_of(a.y.ptr[(t0 + i) * a.y.ld + ch] + by);
+    }
+    __syncthreads();
+  }
+  if (!live) return;
+  if (seg == 0) a.state[slot * a.width + ch] = S0;
+  // the portion's last inputs go to the ring for the tokens that follow
+  if (seg < a.taps && seg < rows) {
+    const float bx = vec_at(a.bx, ch);
+    float* ring = a.ring + slot * (int64_t)a.taps * a.width;
+    for (int64_t b = seg; b < a.taps && b < rows; b += SC_SEG) {
+      const int64_t t = rows - 1 - b;
+      ring[((base + t) % a.taps) * a.width + ch] = a.x.ptr[t * a.x.ld + ch] + bx;
+    }
+  }
+}
+
+}  // namespace
+
+size_t rglru_scratch_floats(const RglruArgs& a, int64_t rows) { return (size_t)3 * rows * a.width; }
+
+int launch_rglru(const RglruArgs& a, const StepRows& r, cudaStream_t st) {
+  if (r.rows == 0) return 0;
+  if (r.base < 0) return step_rows(a, r.pos, r.seq, 0, 0, 0, r.rows, st);
+  if (r.rows == 1) return step_rows(a, nullptr, nullptr, r.base, r.slot, 0, 1, st);
+  DYN_CHECK(r.rows <= 65535, "rglru: portion of %lld tokens", (long long)r.rows);
+  float* u = a.scratch;
+  float *av = u + r.rows * a.width, *bv = av + r.rows * a.width;
+  rglru_conv_kernel<<<dim3((unsigned)((a.width + 255) / 256), (unsigned)r.rows), 256, 0, st>>>(a, r.rows, r.base, r.slot, u);
+  const int n = a.width / a.blocks;
+  rglru_gates_kernel<<<dim3((unsigned)(a.blocks * ((n + GG_N - 1) / GG_N)), (unsigned)((r.rows + GG_M - 1) / GG_M)), 256, 0, st>>>(
+      a, r.rows, u, av, bv);
+  rglru_scan_kernel<<<(unsigned)((a.width + 31) / 32), 1024, 0, st>>>(a, r.rows, r.base, r.slot, av, bv);
+  count_launch(3);
+  DYN_CUDA(cudaGetLastError());
+  return 0;
+}
+
+}  // namespace dyn

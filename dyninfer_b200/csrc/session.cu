@@ -18,141 +18,31 @@
 #include "common.cuh"
 #include "decode_mega.cuh"
 #include "json_min.h"
+#include "session.cuh"
 
 namespace dyn {
 void set_launch_counter(uint64_t* p);
-
-struct NormW {
-  const void* ptr = nullptr;
-  int type = E_F32;
-  uint64_t bytes = 0;
-};
-
-struct LayerW {
-  NormW attn_norm, ffn_norm, q_norm, k_norm;
-  WRef q, k, v, o, gate, up, down;
-  // rows of consecutive matrices seen as one (data == nullptr: not laid back to back)
-  WRef qkv;     // [q; k] or [q; k; v]
-  int qkv_parts = 0;
-  WRef gate_up; // [gate; up]
-};
-
-struct ModelCfg {
-  int layers = 0, hidden = 0, inter = 0, heads = 0, kv_heads = 0, head_dim = 0, vocab = 0;
-  float eps = 1e-6f, theta = 10000.f;
-  bool qk_norm = true, rope = true;
-  int batch = 1;
-  int kv2_type = E_BF16;  // element type used when the KV cache is configured with 2 bytes
-  bool persistent = true;  // single-token steps run as the persistent decode kernel
-  // tensor parallelism: heads / kv_heads / inter above are this rank's share; the lm_head holds
-  // lm_rows = vocab / tp_world consecutive rows starting at tp_rank * lm_rows
-  int tp_rank = 0, tp_world = 1, lm_rows = 0;
-};
-
 }  // namespace dyn
 
 using namespace dyn;
 
-struct dyninfer_cuda_session_t {
-  int device = 0;
-  cudaStream_t stream = nullptr;
-  cudaEvent_t tm0 = nullptr, tm1 = nullptr;  // dyninfer_cuda_session_timer
-  ModelCfg cfg;
-  FreqTable freq;
-  // parameters
-  uint8_t* arena = nullptr;
-  uint64_t arena_bytes = 0;
-  uint64_t weight_bytes = 0;         // sum of uploaded range lengths
-  uint64_t decode_weight_bytes = 0;  // linears + lm_head + norm vectors
-  WRef embed, lm_head;
-  NormW out_norm;
-  std::vector<LayerW> layers;
-  // KV pool
-  bool kv_configured = false;
-  size_t page_size = 0, chunk_size = 0, kv_elem = 0, pages = 0;
-  int kv_type = E_F32;
-  uint8_t* kcache = nullptr;  // [layer][seq][nkv][cap][d]
-  uint8_t* vcache = nullptr;
-  size_t kv_bytes_each = 0;
-  // scratch
-  int64_t max_rows = 0;
-  float *hidden = nullptr, *xn = nullptr, *q = nullptr, *k = nullptr, *v = nullptr, *ctx = nullptr,
-        *act = nullptr, *up = nullptr, *logits = nullptr;
-  // many-row steps: the dequant GEMM's activation operand written by the norm / SwiGLU kernels, and the
-  // K-split sums of o / down waiting for the residual + norm kernel
-  __half* xh = nullptr;
-  float *xinv = nullptr, *gpart = nullptr;
-  int64_t xh_rows = 0, xh_cols = 0;
-  size_t gpart_bytes = 0;
-  float *qkv1 = nullptr, *gu1 = nullptr;  // rows of [q | k | v] and of [gate | up] for the fused products
-  int64_t *tokens_dev = nullptr, *row_pos_dev = nullptr, *row_seq_dev = nullptr,
-          *out_token_dev = nullptr, *hist_dev = nullptr, *hist_count_dev = nullptr;
-  size_t hist_cap = 0;
-  void* argmax_scratch = nullptr;
-  float* batch_logits = nullptr;      // [batch, vocab], allocated by the first batched step
-  int64_t* batch_tokens_dev = nullptr; // [batch]
-  float* batch_logits_host = nullptr;  // pinned, allocated when logits are first requested
-  // pinned host staging
-  float* logits_host = nullptr;
-  int64_t* stage_host = nullptr;  // [0]=token [1]=pos [2]=seq [3]=out token, then chunk arrays
-  // persistent decode kernel
-  bool mega = false;
-  int mega_grid = 0, mega_nslot = 0, mega_xs = 0, mega_max_split = 1;
-  size_t mega_smem = 0;
-  MegaLayer* mega_layers = nullptr;
-  int64_t* io_dev = nullptr;  // [0] token [1] position [2] slot [3] produced token [4] error word
-  unsigned long long* prof_dev = nullptr;
-  unsigned long long* trace_dev = nullptr;  // [grid][layers + 1][16] event stamps (DYNINFER_CUDA_TRACE=1)
-  uint8_t* prog_dev = nullptr;  // [grid] program blobs
-  MegaProgLayout mega_lay;
-  float* ll_dev = nullptr;  // hand-off vectors of (value, epoch) pairs, one allocation
-  size_t ll_off[7] = {};    // float offsets: hidden0, hidden1, qkv, ctx, part, act, amax
-  unsigned mega_epoch = 0;  // epochs used so far (each launch takes layers + 2)
-  // graphs
-  cudaGraphExec_t decode_graph = nullptr;  // H2D token/pos + forward + D2H token
-  cudaGraphExec_t loop_graph = nullptr;    // forward + device-side advance
-  std::map<int64_t, std::pair<cudaGraphExec_t, uint64_t>> batch_graphs;  // rows -> batched step (graph, nodes)
-  uint64_t graph_nodes = 0, loop_nodes = 0;
-  cudaEvent_t ev0 = nullptr, ev1 = nullptr;
-  // tensor parallelism (tp_world > 1): communicator, partial-sum scratch, per-rank logits
-  void* tp_comm = nullptr;
-  float* tp_part = nullptr;    // [max_rows, hidden] partial o_proj / down products of ranks > 0
-  float* tp_logits = nullptr;  // [max(1, batch), lm_rows] this rank's slice of the logits
-  float* tp_gather = nullptr;  // [tp_world, batch, lm_rows] gathered slices of a batched step
-  bool tp_warm = false;        // the collectives have run once outside a capture
-  TpPeer peer;                 // peer-memory exchange (used instead of the all-reduce once attached)
-  // scratch of the single-row products (K-slice partial sums), owned here so that a captured step
-  // has no allocation nodes between its kernels
-  void* scratch = nullptr;
-  size_t scratch_bytes = 0;
-  // statistics
-  dyninfer_cuda_allocator_statistics_t stats{};
-  uint64_t launches = 0;
-};
+namespace dyn {
+
+// b's rows continue a's: the two are one matrix
+bool follows_in_arena(const WRef& a, const WRef& b) {
+  return a.enc == b.enc && a.enc != E_MLX_U4 && a.cols == b.cols &&
+         reinterpret_cast<const uint8_t*>(b.data) == reinterpret_cast<const uint8_t*>(a.data) + a.total_bytes();
+}
+
+// A product in the session's arithmetic: the framework's choice of kernel, or f32 throughout.
+int session_linear(Session* s, const WRef& w, const void* x, int x_type, int64_t m, float* y, const float* residual) {
+  return s->cfg.exact ? launch_linear_exact(w, x, x_type, m, y, residual, s->stream)
+                      : launch_linear(w, x, x_type, m, y, residual, s->stream);
+}
+
+}  // namespace dyn
 
 namespace {
-
-typedef dyninfer_cuda_session_t Session;
-
-int dev_alloc(Session* s, void** out, size_t bytes) {
-  DYN_CUDA(cudaMalloc(out, bytes ? bytes : 16));
-  s->stats.device_bytes_allocated += bytes;
-  uint64_t live = s->stats.device_bytes_allocated - s->stats.device_bytes_freed;
-  s->stats.device_bytes_peak = std::max(s->stats.device_bytes_peak, live);
-  return 0;
-}
-void dev_free(Session* s, void* p, size_t bytes) {
-  if (!p) return;
-  cudaFree(p);
-  s->stats.device_bytes_freed += bytes;
-}
-int host_alloc(Session* s, void** out, size_t bytes) {
-  DYN_CUDA(cudaMallocHost(out, bytes ? bytes : 16));
-  s->stats.host_bytes_allocated += bytes;
-  uint64_t live = s->stats.host_bytes_allocated - s->stats.host_bytes_freed;
-  s->stats.host_bytes_peak = std::max(s->stats.host_bytes_peak, live);
-  return 0;
-}
 
 int enc_from_name(const std::string& n) {
   if (n == "plain.f32") return E_F32;
@@ -238,7 +128,7 @@ int bind_linear(const std::map<std::string, ParamDesc>& params, const uint8_t* a
   out->enc = p.enc;
   out->rows = rows;
   out->cols = cols;
-  int unit = std::max(4, enc_block_elems(p.enc));
+  const int unit = enc_block_elems(p.enc) == 1 ? 1 : std::max(4, enc_block_elems(p.enc));
   DYN_CHECK(cols % unit == 0, "parameter `%s`: cols %lld not a multiple of %d", name.c_str(),
             (long long)cols, unit);
   const char* main_comp = p.enc == E_MLX_U4 ? "packed" : "data";
@@ -287,6 +177,37 @@ int bind_norm(const std::map<std::string, ParamDesc>& params, const uint8_t* are
   out->bytes = c->second.length;
   return 0;
 }
+
+// A plain tensor of any rank, read by its element type.
+int bind_plain(const std::map<std::string, ParamDesc>& params, const uint8_t* arena, const std::string& name,
+               const std::vector<int64_t>& shape, NormW* out) {
+  auto it = params.find(name);
+  DYN_CHECK(it != params.end(), "model descriptor lacks parameter `%s`", name.c_str());
+  const ParamDesc& p = it->second;
+  DYN_CHECK(p.enc == E_F32 || p.enc == E_F16 || p.enc == E_BF16, "parameter `%s` must be a plain float type", name.c_str());
+  DYN_CHECK(p.shape == shape, "parameter `%s` has the wrong shape", name.c_str());
+  uint64_t n = 1;
+  for (int64_t d : shape) n *= (uint64_t)d;
+  auto c = p.comps.find("data");
+  DYN_CHECK(c != p.comps.end(), "no byte range given for `weights::%s::data`", name.c_str());
+  DYN_CHECK(c->second.length == n * aux_elem_bytes(p.enc), "parameter `%s` byte length mismatch", name.c_str());
+  out->ptr = arena + c->second.arena_off;
+  out->type = p.enc;
+  out->bytes = c->second.length;
+  return 0;
+}
+
+struct UploadedParams : ParamTable {
+  const std::map<std::string, ParamDesc>& params;
+  const uint8_t* arena;
+  UploadedParams(const std::map<std::string, ParamDesc>& p, const uint8_t* a) : params(p), arena(a) {}
+  int linear(const std::string& name, int64_t rows, int64_t cols, WRef* out) const override {
+    return bind_linear(params, arena, name, rows, cols, out);
+  }
+  int plain(const std::string& name, const std::vector<int64_t>& shape, NormW* out) const override {
+    return bind_plain(params, arena, name, shape, out);
+  }
+};
 
 void destroy_graphs(Session* s) {
   if (s->decode_graph) cudaGraphExecDestroy(s->decode_graph);
@@ -337,10 +258,8 @@ int tp_row_parallel(Session* s, const WRef& w, const float* x, int64_t rows, int
   return tp_all_reduce_sum(s->tp_comm, s->tp_part, s->hidden, n, st);
 }
 
-// Enqueue the whole decoder for `rows` rows whose tokens / positions / slots are
-// already in device memory; logits and argmax come from row `logits_row`.
-int enqueue_forward(Session* s, int64_t rows, int64_t logits_row, bool all_rows = false,
-                    int64_t chunk_start = -1, int64_t chunk_slot = 0) {
+// The layers of a GQA decoder.
+int enqueue_gqa_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t chunk_slot) {
   const ModelCfg& c = s->cfg;
   cudaStream_t st = s->stream;
   const bool tp = c.tp_world > 1;
@@ -348,7 +267,6 @@ int enqueue_forward(Session* s, int64_t rows, int64_t logits_row, bool all_rows 
                 kvd = (int64_t)c.kv_heads * c.head_dim;
   const int64_t cap = (int64_t)(s->pages * s->page_size);
   const size_t layer_stride = (size_t)c.batch * c.kv_heads * cap * c.head_dim * s->kv_elem;
-  if (launch_gather(s->embed, s->tokens_dev, rows, s->hidden, st)) return 1;
   bool normed = false;  // xn already holds this layer's attn_norm rows (fused into the last exchange)
   // One row: the q / k / v and [gate; up] products (local also under tensor parallelism), when their K is
   // split over CTAs, leave the
@@ -356,7 +274,7 @@ int enqueue_forward(Session* s, int64_t rows, int64_t logits_row, bool all_rows 
   // launches fewer per layer (8B mixed: 3.24 -> 2.90 ms per step). The sums wait in the session's scratch,
   // held until that kernel is enqueued. The same for o / down with residual + RMSNorm in one single-block
   // kernel was slower (3.39 ms): their reductions stay separate, multi-block launches.
-  const bool fuse1 = rows == 1;
+  const bool fuse1 = rows == 1 && !c.exact;
   auto linear_deferred = [&](const WRef& w, const float* x, float* y, Deferred* d) -> int {
     DeferScope scope(d);
     if (launch_linear(w, x, E_F32, 1, y, nullptr, st)) return 1;
@@ -370,7 +288,7 @@ int enqueue_forward(Session* s, int64_t rows, int64_t logits_row, bool all_rows 
   // per layer and five passes over the activations fewer, with the same bits as the separate kernels.
   // (one block per row: with few rows -- batched decode steps -- the separate multi-block kernels are faster:
   // 32 rows of the 32B shape 13.5 against 14.4 ms per step)
-  bool fuse_n = rows >= 64 && !tp && s->xh && H <= 8192;
+  bool fuse_n = rows >= 64 && !tp && s->xh && H <= 8192 && !c.exact;
   for (int l = 0; l < c.layers && fuse_n; l++) {
     const LayerW& L = s->layers[l];
     const WRef* ws[8] = {L.qkv_parts >= 2 ? &L.qkv : &L.q, L.qkv_parts >= 2 ? nullptr : &L.k, L.qkv_parts == 3 ? nullptr : &L.v,
@@ -494,13 +412,13 @@ int enqueue_forward(Session* s, int64_t rows, int64_t logits_row, bool all_rows 
     } else if (L.qkv_parts >= 2) {
       qp = s->qkv1, kp = qp + qd;
       ldq = ldk = L.qkv_parts == 3 ? qd + 2 * kvd : qd + kvd;
-      if (launch_linear(L.qkv, s->xn, E_F32, rows, qp, nullptr, st)) return 1;
+      if (session_linear(s, L.qkv, s->xn, E_F32, rows, qp, nullptr)) return 1;
       if (L.qkv_parts == 3) vp = kp + kvd, ldv = ldq;
-      else if (launch_linear(L.v, s->xn, E_F32, rows, vp, nullptr, st)) return 1;
+      else if (session_linear(s, L.v, s->xn, E_F32, rows, vp, nullptr)) return 1;
     } else {
-      if (launch_linear(L.q, s->xn, E_F32, rows, qp, nullptr, st)) return 1;
-      if (launch_linear(L.k, s->xn, E_F32, rows, kp, nullptr, st)) return 1;
-      if (launch_linear(L.v, s->xn, E_F32, rows, vp, nullptr, st)) return 1;
+      if (session_linear(s, L.q, s->xn, E_F32, rows, qp, nullptr)) return 1;
+      if (session_linear(s, L.k, s->xn, E_F32, rows, kp, nullptr)) return 1;
+      if (session_linear(s, L.v, s->xn, E_F32, rows, vp, nullptr)) return 1;
     }
     QkvPrepArgs pa{};
     pa.q = qp, pa.k = kp, pa.v = vp;
@@ -526,14 +444,14 @@ int enqueue_forward(Session* s, int64_t rows, int64_t logits_row, bool all_rows 
     if (launch_attention(aa, st)) return 1;
     bool ffn_normed = false;
     if (tp ? tp_row_parallel(s, L.o, s->ctx, rows, 0, &L.ffn_norm, &ffn_normed, st)
-           : launch_linear(L.o, s->ctx, E_F32, rows, s->hidden, s->hidden, st))
+           : session_linear(s, L.o, s->ctx, E_F32, rows, s->hidden, s->hidden))
       return 1;
     if (!ffn_normed &&
         launch_rms_norm(s->hidden, L.ffn_norm.ptr, L.ffn_norm.type, rows, H, c.eps, s->xn, st))
       return 1;
     // one row: the column-split GEMVs run at ~3x the fused scalar kernel's bandwidth, which more than
     // pays for the separate activation launch
-    const bool fast_gemv = (rows == 1 && gemv_cs_workspace_bytes(L.gate, 1) && gemv_cs_workspace_bytes(L.up, 1)) ||
+    const bool fast_gemv = c.exact || (rows == 1 && gemv_cs_workspace_bytes(L.gate, 1) && gemv_cs_workspace_bytes(L.up, 1)) ||
                            (rows <= 4 && gemv_mma_workspace_bytes(L.gate, E_F32, (int)rows) &&
                             gemv_mma_workspace_bytes(L.up, E_F32, (int)rows));
     if (fuse1 && L.gate_up.data && gemv_cs_workspace_bytes(L.gate_up, 1) != 0) {
@@ -544,20 +462,41 @@ int enqueue_forward(Session* s, int64_t rows, int64_t logits_row, bool all_rows 
       thread_scratch_release_all();
     } else if (L.gate_up.data && (rows == 1 ? gemv_cs_workspace_bytes(L.gate_up, 1) != 0 : rows > 4 || fast_gemv)) {
       // [gate; up] as one product into rows of [gate | up], then the activation
-      if (launch_linear(L.gate_up, s->xn, E_F32, rows, s->gu1, nullptr, st)) return 1;
+      if (session_linear(s, L.gate_up, s->xn, E_F32, rows, s->gu1, nullptr)) return 1;
       if (launch_silu_mul_rows(s->gu1, rows, c.inter, s->act, st)) return 1;
     } else if (L.gate.enc == L.up.enc && rows <= 4 && !fast_gemv) {
       if (launch_linear_swiglu(L.gate, L.up, s->xn, rows, s->act, st)) return 1;
     } else {
       // many rows (tensor-core GEMM) or mixed encodings: two products, then the activation
-      if (launch_linear(L.gate, s->xn, E_F32, rows, s->act, nullptr, st)) return 1;
-      if (launch_linear(L.up, s->xn, E_F32, rows, s->up, nullptr, st)) return 1;
+      if (session_linear(s, L.gate, s->xn, E_F32, rows, s->act, nullptr)) return 1;
+      if (session_linear(s, L.up, s->xn, E_F32, rows, s->up, nullptr)) return 1;
       if (launch_silu_mul(s->act, s->up, rows * c.inter, s->act, st)) return 1;
     }
     normed = false;
     if (tp ? tp_row_parallel(s, L.down, s->act, rows, 1,
                              l + 1 < c.layers ? &s->layers[l + 1].attn_norm : nullptr, &normed, st)
-           : launch_linear(L.down, s->act, E_F32, rows, s->hidden, s->hidden, st))
+           : session_linear(s, L.down, s->act, E_F32, rows, s->hidden, s->hidden))
+      return 1;
+  }
+  return 0;
+}
+
+// Enqueue the whole decoder for `rows` rows whose tokens / positions / slots are
+// already in device memory; logits and argmax come from row `logits_row`, or of every row
+// (`all_rows`: a batched step), or logits alone of the `wanted` rows listed in want_index_dev.
+int enqueue_forward(Session* s, int64_t rows, int64_t logits_row, bool all_rows = false,
+                    int64_t chunk_start = -1, int64_t chunk_slot = 0, int64_t wanted = 0) {
+  const ModelCfg& c = s->cfg;
+  cudaStream_t st = s->stream;
+  const bool tp = c.tp_world > 1;
+  const int64_t H = c.hidden;
+  if (launch_gather(s->embed, s->tokens_dev, rows, s->hidden, st)) return 1;
+  if (c.mixers.empty() ? enqueue_gqa_layers(s, rows, chunk_start, chunk_slot)
+                       : enqueue_mixer_layers(s, rows, chunk_start, chunk_slot))
+    return 1;
+  if (wanted) {
+    if (launch_rms_norm_indexed(s->hidden, s->want_index_dev, s->out_norm.ptr, s->out_norm.type, wanted, H, c.eps, s->xn, st) ||
+        session_linear(s, s->lm_head, s->xn, E_F32, wanted, s->want_logits, nullptr))
       return 1;
   }
   if (all_rows) {
@@ -570,7 +509,7 @@ int enqueue_forward(Session* s, int64_t rows, int64_t logits_row, bool all_rows 
       if (tp_all_gather(s->tp_comm, s->tp_logits, s->tp_gather, (size_t)rows * c.lm_rows, st)) return 1;
       return launch_argmax_rows_sharded(s->tp_gather, rows, c.lm_rows, c.tp_world, s->batch_tokens_dev, st);
     }
-    if (launch_linear(s->lm_head, s->xn, E_F32, rows, s->batch_logits, nullptr, st)) return 1;
+    if (session_linear(s, s->lm_head, s->xn, E_F32, rows, s->batch_logits, nullptr)) return 1;
     if (launch_argmax_rows(s->batch_logits, rows, c.vocab, s->batch_tokens_dev, st)) return 1;
     return 0;
   }
@@ -582,11 +521,10 @@ int enqueue_forward(Session* s, int64_t rows, int64_t logits_row, bool all_rows 
     // one row: the gathered slices are the logits in vocabulary order
     if (launch_linear(s->lm_head, s->xn, E_F32, 1, s->tp_logits, nullptr, st)) return 1;
     if (tp_all_gather(s->tp_comm, s->tp_logits, s->logits, (size_t)c.lm_rows, st)) return 1;
-  } else if (launch_linear(s->lm_head, s->xn, E_F32, 1, s->logits, nullptr, st)) {
+  } else if (session_linear(s, s->lm_head, s->xn, E_F32, 1, s->logits, nullptr)) {
     return 1;
   }
   if (launch_argmax(s->logits, c.vocab, s->out_token_dev, s->argmax_scratch, st)) return 1;
-  (void)kvd;
   return 0;
 }
 
@@ -758,6 +696,20 @@ int tp_check_error(Session* s) {
   return 1;
 }
 
+// The position a slot reaches with a step. While the step runs, and for good if it fails, the slot counts
+// as unusable: recurrent state that was only partly updated cannot be continued.
+struct SlotStep {
+  Session* s;
+  size_t slot;
+  int64_t to;
+  SlotStep(Session* session, int64_t at, int64_t next) : s(session), slot((size_t)at), to(next) {
+    if (slot < s->slot_pos.size()) s->slot_pos[slot] = -1;
+  }
+  void done() {
+    if (slot < s->slot_pos.size()) s->slot_pos[slot] = to;
+  }
+};
+
 struct CounterScope {  // routes count_launch() and product scratch to this session for one call
   explicit CounterScope(Session* s) {
     set_launch_counter(&s->launches);
@@ -829,22 +781,32 @@ int dyninfer_cuda_session_create_with_file_params(
               dk.c_str());
     cfg.persistent = dk == "persistent";
   }
+  {
+    const std::string cm = desc.string("compute", "serve");
+    DYN_CHECK(cm == "serve" || cm == "f32", "compute `%s` unknown (serve | f32)", cm.c_str());
+    cfg.exact = cm == "f32";
+    if (cfg.exact) cfg.persistent = false;  // the persistent kernel multiplies split 16-bit operands
+  }
+  if (parse_mixers(desc, &cfg)) return 1;
+  if (!cfg.mixers.empty()) cfg.persistent = false;
   cfg.tp_world = (int)desc.number("tp_world", 1);
   cfg.tp_rank = (int)desc.number("tp_rank", 0);
   DYN_CHECK(cfg.tp_world >= 1 && cfg.tp_rank >= 0 && cfg.tp_rank < cfg.tp_world,
             "tensor-parallel rank %d outside [0, %d)", cfg.tp_rank, cfg.tp_world);
   if (cfg.tp_world > 1) cfg.persistent = false;  // the single-GPU persistent kernel has no exchange step
-  DYN_CHECK(cfg.layers > 0 && cfg.hidden > 0 && cfg.inter > 0 && cfg.heads > 0 &&
-                cfg.kv_heads > 0 && cfg.head_dim > 0 && cfg.vocab > 0 && cfg.batch > 0,
+  const bool mixers = !cfg.mixers.empty();
+  DYN_CHECK(!mixers || cfg.tp_world == 1, "a decoder with mixers has no tensor-parallel form");
+  DYN_CHECK(cfg.layers > 0 && cfg.hidden > 0 && cfg.vocab > 0 && cfg.batch > 0 &&
+                (mixers || (cfg.inter > 0 && cfg.heads > 0 && cfg.kv_heads > 0 && cfg.head_dim > 0)),
             "model descriptor lacks geometry (layers/hidden/intermediate/heads/kv_heads/head_dim/vocab)");
-  DYN_CHECK(cfg.heads % cfg.kv_heads == 0, "heads %d is not a multiple of kv_heads %d", cfg.heads,
+  DYN_CHECK(mixers || cfg.heads % cfg.kv_heads == 0, "heads %d is not a multiple of kv_heads %d", cfg.heads,
             cfg.kv_heads);
   cfg.lm_rows = (int)desc.number("lm_head_rows", cfg.vocab);
   DYN_CHECK(cfg.lm_rows > 0 && (int64_t)cfg.lm_rows * cfg.tp_world == cfg.vocab,
             "lm_head_rows %d x tp_world %d does not equal the vocabulary %d", cfg.lm_rows, cfg.tp_world,
             cfg.vocab);
-  DYN_CHECK(cfg.head_dim % 2 == 0 && cfg.head_dim <= 256, "head_dim %d unsupported", cfg.head_dim);
-  DYN_CHECK(cfg.hidden % 4 == 0 && cfg.inter % 4 == 0, "hidden and intermediate must be multiples of 4");
+  DYN_CHECK(mixers || (cfg.head_dim % 2 == 0 && cfg.head_dim <= 256), "head_dim %d unsupported", cfg.head_dim);
+  DYN_CHECK(mixers || (cfg.hidden % 4 == 0 && cfg.inter % 4 == 0), "hidden and intermediate must be multiples of 4");
 
   // parameters: descriptor entries joined with their byte ranges
   std::map<std::string, ParamDesc> pd;
@@ -998,11 +960,12 @@ int dyninfer_cuda_session_create_with_file_params(
         placed.insert(run[i]);
       }
     };
-    for (int l = 0; l < cfg.layers; l++) {
+    for (int l = 0; l < cfg.layers && !mixers; l++) {
       const std::string b = "blk." + std::to_string(l) + ".";
       place_run({b + "attn_q.weight", b + "attn_k.weight", b + "attn_v.weight"});
       place_run({b + "ffn_gate.weight", b + "ffn_up.weight"});
     }
+    for (const auto& run : mixers ? mixer_place_runs(cfg) : std::vector<std::vector<std::string>>()) place_run(run);
     for (auto& p : pd)
       for (auto& c : p.second.comps) {
         if (placed.count(&c.second)) continue;
@@ -1041,7 +1004,7 @@ int dyninfer_cuda_session_create_with_file_params(
   cudaEventCreate(&s->ev0);
   cudaEventCreate(&s->ev1);
   if (!device_error_word()) return fail();  // allocated before any launch or stream capture
-  fill_freq_table(&s->freq, cfg.head_dim, cfg.theta);
+  if (!mixers) fill_freq_table(&s->freq, cfg.head_dim, cfg.theta);
   if (dev_alloc(s, (void**)&s->arena, arena_bytes)) return fail();
   s->arena_bytes = arena_bytes;
   if (cudaMemset(s->arena, 0, arena_bytes) != cudaSuccess) {
@@ -1083,9 +1046,10 @@ int dyninfer_cuda_session_create_with_file_params(
     s->lm_head = s->embed;  // tied: same bytes (crates/dyninfer-architecture/src/naming.rs:70-96)
   }
   if (bind_norm(pd, s->arena, "output_norm.weight", H, true, &s->out_norm)) return fail();
-  s->layers.resize(cfg.layers);
   uint64_t dwb = s->lm_head.total_bytes() + s->out_norm.bytes;
-  for (int l = 0; l < cfg.layers; l++) {
+  if (mixers && bind_mixers(s, UploadedParams(pd, s->arena), &dwb)) return fail();
+  s->layers.resize(mixers ? 0 : cfg.layers);
+  for (int l = 0; l < cfg.layers && !mixers; l++) {
     LayerW& L = s->layers[l];
     std::string p = "blk." + std::to_string(l) + ".";
     if (bind_norm(pd, s->arena, p + "attn_norm.weight", H, true, &L.attn_norm) ||
@@ -1101,17 +1065,13 @@ int dyninfer_cuda_session_create_with_file_params(
         bind_linear(pd, s->arena, p + "ffn_down.weight", H, I, &L.down))
       return fail();
     {
-      auto follows = [](const WRef& a, const WRef& b) {
-        return a.enc == b.enc && a.enc != E_MLX_U4 && a.cols == b.cols &&
-               reinterpret_cast<const uint8_t*>(b.data) == reinterpret_cast<const uint8_t*>(a.data) + a.total_bytes();
-      };
-      if (follows(L.q, L.k)) {
+      if (follows_in_arena(L.q, L.k)) {
         L.qkv = L.q;
         L.qkv.rows = L.q.rows + L.k.rows;
         L.qkv_parts = 2;
-        if (follows(L.k, L.v)) L.qkv.rows += L.v.rows, L.qkv_parts = 3;
+        if (follows_in_arena(L.k, L.v)) L.qkv.rows += L.v.rows, L.qkv_parts = 3;
       }
-      if (follows(L.gate, L.up)) {
+      if (follows_in_arena(L.gate, L.up)) {
         L.gate_up = L.gate;
         L.gate_up.rows = L.gate.rows + L.up.rows;
       }
@@ -1131,6 +1091,11 @@ int dyninfer_cuda_session_create_with_file_params(
       for (int m = 1; m <= 8; m++) need = std::max(need, gemv_mma_workspace_bytes(w, E_F32, m));
     };
     grow(s->lm_head);
+    for (const MixerLayer& L : s->mix) {
+      for (const WRef& w : L.in) grow(w);
+      for (const WRef* w : {&L.o, &L.gate, &L.up, &L.gate_up, &L.down})
+        if (w->data) grow(*w);
+    }
     for (const LayerW& L : s->layers) {
       const WRef* ws[7] = {&L.q, &L.k, &L.v, &L.o, &L.gate, &L.up, &L.down};
       for (const WRef* wp : ws) grow(*wp);
@@ -1139,7 +1104,8 @@ int dyninfer_cuda_session_create_with_file_params(
     }
     if (need) {
       need = need * 3 + 1024;  // up to three products' K-slice sums wait for the kernel that adds them
-      for (int64_t r : {(int64_t)1, (int64_t)std::max(1, cfg.batch)}) {  // decode attention's slice results
+      for (int64_t r : {(int64_t)1, (int64_t)std::max(1, cfg.batch)}) {
+        if (mixers) break;  // decode attention's slice results
         const int64_t per = std::max<int64_t>(1, std::min<int64_t>(32, 592 / (r * cfg.heads)));
         need = std::max(need, attention_split_scratch_bytes(r, cfg.heads, cfg.head_dim, (int)per));
       }
@@ -1215,11 +1181,13 @@ void dyninfer_cuda_session_destroy(dyninfer_cuda_session_t* s) {
                  s->logits, s->tokens_dev, s->row_pos_dev, s->row_seq_dev, s->out_token_dev,
                  s->hist_dev, s->hist_count_dev, s->argmax_scratch, s->mega_layers, s->io_dev,
                  s->prof_dev, s->trace_dev, s->prog_dev, s->ll_dev, s->batch_logits, s->batch_tokens_dev, s->tp_part, s->tp_logits,
-                 s->tp_gather, s->scratch, s->qkv1, s->gu1, s->xh, s->xinv, s->gpart};
+                 s->tp_gather, s->scratch, s->qkv1, s->gu1, s->xh, s->xinv, s->gpart,
+                 s->lcache, s->state, s->mix_scratch, s->tables, s->want_logits, s->want_index_dev};
   for (void* p : dev)
     if (p) cudaFree(p);
   if (s->logits_host) cudaFreeHost(s->logits_host);
   if (s->batch_logits_host) cudaFreeHost(s->batch_logits_host);
+  if (s->want_logits_host) cudaFreeHost(s->want_logits_host);
   if (s->stage_host) cudaFreeHost(s->stage_host);
   if (s->tm0) cudaEventDestroy(s->tm0);
   if (s->tm1) cudaEventDestroy(s->tm1);
@@ -1263,7 +1231,9 @@ int dyninfer_cuda_session_configure_paged_kv(dyninfer_cuda_session_t* s, size_t 
   const ModelCfg& c = s->cfg;
   const int64_t rows = std::max<int64_t>((int64_t)chunk_size, c.batch);
   const int64_t qd = (int64_t)c.heads * c.head_dim, kvd = (int64_t)c.kv_heads * c.head_dim;
-  if (!s->kv_configured) {
+  if (!s->kv_configured && !c.mixers.empty()) {
+    if (configure_mixers(s, rows)) return 1;
+  } else if (!s->kv_configured) {
     if (dev_alloc(s, (void**)&s->hidden, (size_t)rows * c.hidden * 4) ||
         dev_alloc(s, (void**)&s->xn, (size_t)rows * c.hidden * 4) ||
         dev_alloc(s, (void**)&s->ctx, (size_t)rows * qd * 4) ||
@@ -1348,6 +1318,12 @@ int dyninfer_cuda_session_ensure_kv_pages(dyninfer_cuda_session_t* s, size_t pag
   CounterScope scope(s);
   DYN_CUDA(cudaSetDevice(s->device));
   const ModelCfg& c = s->cfg;
+  if (!c.mixers.empty()) {
+    if (ensure_mixer_pages(s, page_count)) return 1;
+    s->pages = page_count;
+    destroy_graphs(s);
+    return 0;
+  }
   const size_t planes = (size_t)c.layers * c.batch * c.kv_heads;
   const size_t new_row = page_count * s->page_size * c.head_dim * s->kv_elem;  // bytes per plane
   const size_t old_row = s->pages * s->page_size * c.head_dim * s->kv_elem;
@@ -1382,6 +1358,7 @@ int dyninfer_cuda_session_reset_paged_kv(dyninfer_cuda_session_t* s) {
   DYN_CHECK(s->kv_configured, "paged KV is not configured");
   if (!s->pages) return 0;
   DYN_CUDA(cudaSetDevice(s->device));
+  if (!s->cfg.mixers.empty()) return reset_mixers(s);
   // zero-fill in place, the pool is kept (wrapper.c:1273-1303)
   DYN_CUDA(cudaMemsetAsync(s->kcache, 0, s->kv_bytes_each, s->stream));
   DYN_CUDA(cudaMemsetAsync(s->vcache, 0, s->kv_bytes_each, s->stream));
@@ -1393,7 +1370,7 @@ size_t dyninfer_cuda_session_kv_page_count(const dyninfer_cuda_session_t* s) {
   return s ? s->pages : 0;
 }
 size_t dyninfer_cuda_session_kv_allocated_bytes(const dyninfer_cuda_session_t* s) {
-  return s ? 2 * s->kv_bytes_each : 0;
+  return !s ? 0 : s->cfg.mixers.empty() ? 2 * s->kv_bytes_each : s->lcache_bytes + s->state_floats * 4;
 }
 
 int dyninfer_cuda_session_allocator_statistics(const dyninfer_cuda_session_t* s,
@@ -1489,8 +1466,10 @@ int dyninfer_cuda_session_invoke_paged_chunk_slot(dyninfer_cuda_session_t* s, co
   for (int64_t i = 0; i < rows; i++)
     DYN_CHECK(tokens[i] >= 0 && tokens[i] < s->cfg.vocab, "token id %lld at %lld outside [0, %d)",
               (long long)tokens[i], (long long)i, s->cfg.vocab);
+  if (mixer_check_position(s, slot, start_pos)) return 1;
   CounterScope scope(s);
   DYN_CUDA(cudaSetDevice(s->device));
+  SlotStep moved(s, slot, start_pos + rows);
   if (rows == 1 && s->mega) {
     s->stage_host[0] = tokens[0];
     s->stage_host[1] = start_pos;
@@ -1532,6 +1511,7 @@ int dyninfer_cuda_session_invoke_paged_chunk_slot(dyninfer_cuda_session_t* s, co
   if (tp_check_error(s)) return 1;
   if (check_device_error("session step")) return 1;
   if (rows == 1 && s->mega && mega_check_error(s, s->stage_host[4])) return 1;
+  moved.done();
   if (out_token) *out_token = s->stage_host[3];
   if (want_logits) {
     *out_logits = s->logits_host;  // session scratch, borrowed until the next invoke
@@ -1565,6 +1545,7 @@ int dyninfer_cuda_session_decode_batch(dyninfer_cuda_session_t* s, const int64_t
     DYN_CHECK(slots[i] >= 0 && slots[i] < s->cfg.batch && !used[(size_t)slots[i]],
               "slot %lld at %lld is out of range or used twice in one step", (long long)slots[i], (long long)i);
     used[(size_t)slots[i]] = 1;
+    if (mixer_check_position(s, slots[i], positions[i])) return 1;
   }
   if (rows == 1 && !want_logits) {  // a single sequence: the single-token fast path serves any slot
     if (out_logits) *out_logits = nullptr;
@@ -1573,6 +1554,8 @@ int dyninfer_cuda_session_decode_batch(dyninfer_cuda_session_t* s, const int64_t
   }
   CounterScope scope(s);
   DYN_CUDA(cudaSetDevice(s->device));
+  std::vector<SlotStep> moved;
+  for (int64_t i = 0; i < rows; i++) moved.emplace_back(s, slots[i], positions[i] + 1);
   if (!s->batch_logits) {
     if (dev_alloc(s, (void**)&s->batch_logits, (size_t)s->cfg.batch * s->cfg.vocab * 4) ||
         dev_alloc(s, (void**)&s->batch_tokens_dev, (size_t)s->cfg.batch * 8) ||
@@ -1615,8 +1598,82 @@ int dyninfer_cuda_session_decode_batch(dyninfer_cuda_session_t* s, const int64_t
   DYN_CUDA(cudaStreamSynchronize(s->stream));
   if (tp_check_error(s)) return 1;
   if (check_device_error("session step")) return 1;
+  for (SlotStep& m : moved) m.done();
   for (int64_t i = 0; i < rows; i++) out_tokens[i] = st[i];
   if (out_logits) *out_logits = want_logits ? s->batch_logits_host : nullptr;  // borrowed until the next call
+  return 0;
+}
+
+// A portion with the logits of any of its rows: tokens [0, count) of slot `slot` from position start_pos.
+int dyninfer_cuda_session_invoke_portion(dyninfer_cuda_session_t* s, const int64_t* tokens, size_t count, int64_t start_pos,
+                                         int64_t slot, const int64_t* want, size_t want_count, float** out_logits,
+                                         int64_t* out_token) {
+  DYN_CHECK(s != nullptr, "session is NULL");
+  DYN_CHECK(s->kv_configured && s->pages > 0, "paged KV is not configured or has no pages");
+  DYN_CHECK(tokens != nullptr && count >= 1 && count <= s->chunk_size, "portion of %zu tokens outside [1, %zu]", count,
+            s->chunk_size);
+  DYN_CHECK(want_count == 0 || (want && out_logits), "wanted rows need `want` and `out_logits`");
+  DYN_CHECK(want_count <= count, "%zu rows wanted of a portion of %zu", want_count, count);
+  for (size_t i = 0; i < want_count; i++)
+    DYN_CHECK(want[i] >= 0 && (size_t)want[i] < count, "wanted row %lld outside [0, %zu)", (long long)want[i], count);
+  if (out_logits) *out_logits = nullptr;
+  DYN_CHECK(s->cfg.tp_world == 1 || want_count == 0, "wanted rows of a tensor-parallel session are not supported");
+  if (count == 1) {  // the single-token step of any slot
+    size_t n = 0;
+    float* lg = nullptr;
+    if (dyninfer_cuda_session_invoke_paged_chunk_slot(s, tokens, 1, 0, start_pos, slot, &lg, &n, out_token,
+                                                      want_count ? 1 : 0))
+      return 1;
+    if (out_logits) *out_logits = lg;
+    return 0;
+  }
+  DYN_CHECK(slot >= 0 && slot < s->cfg.batch, "slot %lld outside [0, %d) (the descriptor's \"batch\")",
+            (long long)slot, s->cfg.batch);
+  const int64_t rows = (int64_t)count, cap = (int64_t)(s->pages * s->page_size), wanted = (int64_t)want_count;
+  DYN_CHECK(start_pos >= 0 && start_pos + rows <= cap, "positions [%lld, %lld) exceed the KV capacity %lld",
+            (long long)start_pos, (long long)(start_pos + rows), (long long)cap);
+  for (int64_t i = 0; i < rows; i++)
+    DYN_CHECK(tokens[i] >= 0 && tokens[i] < s->cfg.vocab, "token id %lld at %lld outside [0, %d)",
+              (long long)tokens[i], (long long)i, s->cfg.vocab);
+  if (mixer_check_position(s, slot, start_pos)) return 1;
+  CounterScope scope(s);
+  DYN_CUDA(cudaSetDevice(s->device));
+  SlotStep moved(s, slot, start_pos + rows);
+  if (wanted > s->want_cap) {
+    const size_t old = (size_t)s->want_cap * s->cfg.vocab * 4, bytes = want_count * s->cfg.vocab * 4;
+    dev_free(s, s->want_logits, old);
+    dev_free(s, s->want_index_dev, (size_t)s->want_cap * 8);
+    if (s->want_logits_host) {
+      cudaFreeHost(s->want_logits_host);
+      s->stats.host_bytes_freed += old;
+    }
+    s->want_logits = s->want_logits_host = nullptr, s->want_index_dev = nullptr, s->want_cap = 0;
+    if (dev_alloc(s, (void**)&s->want_logits, bytes) || dev_alloc(s, (void**)&s->want_index_dev, want_count * 8) ||
+        host_alloc(s, (void**)&s->want_logits_host, bytes))
+      return 1;
+    s->want_cap = wanted;
+  }
+  int64_t* st = s->stage_host + 8;
+  for (int64_t i = 0; i < rows; i++) {
+    st[i] = tokens[i];
+    st[rows + i] = start_pos + i;
+    st[2 * rows + i] = slot;
+  }
+  DYN_CUDA(cudaMemcpyAsync(s->tokens_dev, st, rows * 8, cudaMemcpyHostToDevice, s->stream));
+  DYN_CUDA(cudaMemcpyAsync(s->row_pos_dev, st + rows, rows * 8, cudaMemcpyHostToDevice, s->stream));
+  DYN_CUDA(cudaMemcpyAsync(s->row_seq_dev, st + 2 * rows, rows * 8, cudaMemcpyHostToDevice, s->stream));
+  if (wanted) DYN_CUDA(cudaMemcpyAsync(s->want_index_dev, want, wanted * 8, cudaMemcpyHostToDevice, s->stream));
+  if (enqueue_forward(s, rows, rows - 1, false, start_pos, slot, wanted)) return 1;
+  DYN_CUDA(cudaMemcpyAsync(s->stage_host + 3, s->out_token_dev, 8, cudaMemcpyDeviceToHost, s->stream));
+  if (wanted)
+    DYN_CUDA(cudaMemcpyAsync(s->want_logits_host, s->want_logits, want_count * s->cfg.vocab * 4, cudaMemcpyDeviceToHost,
+                             s->stream));
+  DYN_CUDA(cudaStreamSynchronize(s->stream));
+  if (tp_check_error(s)) return 1;
+  if (check_device_error("session step")) return 1;
+  moved.done();
+  if (out_token) *out_token = s->stage_host[3];
+  if (wanted) *out_logits = s->want_logits_host;  // borrowed until the next call
   return 0;
 }
 
@@ -1704,6 +1761,7 @@ int dyninfer_cuda_session_decode_loop(dyninfer_cuda_session_t* s, int64_t first_
             (long long)(start_pos + (int64_t)steps), (long long)cap);
   if (out_device_ms) *out_device_ms = 0.f;
   if (steps == 0) return 0;
+  if (mixer_check_position(s, 0, start_pos)) return 1;
   CounterScope scope(s);
   DYN_CUDA(cudaSetDevice(s->device));
   if (ensure_hist(s, steps)) return 1;
@@ -1731,6 +1789,7 @@ int dyninfer_cuda_session_decode_loop(dyninfer_cuda_session_t* s, int64_t first_
       DYN_CUDA(cudaMemcpy(out_tokens, s->hist_dev, steps * 8, cudaMemcpyDeviceToHost));
     return 0;
   }
+  SlotStep moved(s, 0, start_pos + (int64_t)steps);
   if (!s->loop_graph && capture(s, true, &s->loop_graph, &s->loop_nodes)) return 1;
   s->stage_host[0] = first_token;
   s->stage_host[1] = start_pos;
@@ -1746,6 +1805,7 @@ int dyninfer_cuda_session_decode_loop(dyninfer_cuda_session_t* s, int64_t first_
   DYN_CUDA(cudaStreamSynchronize(s->stream));
   if (tp_check_error(s)) return 1;
   if (check_device_error("session step")) return 1;
+  moved.done();
   if (out_device_ms) DYN_CUDA(cudaEventElapsedTime(out_device_ms, s->ev0, s->ev1));
   if (out_tokens)
     DYN_CUDA(cudaMemcpy(out_tokens, s->hist_dev, steps * 8, cudaMemcpyDeviceToHost));

@@ -1,0 +1,425 @@
+// Decoders whose layers are listed one by one, each with a mixer of its own kind (retention, gated
+// linear recurrence, latent attention) and an optional gated feed-forward: descriptor entries, binding
+// of parameters, caches and states, and the layers of a step.
+//
+// A layer may run with another layer's parameters; its cache and state are always its own. The steps,
+// graphs, batching and ABI around the layers are the session's (session.cu).
+#include <math.h>
+
+#include "json_min.h"
+#include "session.cuh"
+
+namespace dyn {
+
+int parse_mixers(const Json& desc, ModelCfg* cfg) {
+  const Json* list = desc.get("mixers");
+  if (!list) return 0;
+  DYN_CHECK(list->kind == Json::Arr && (int)list->arr.size() == cfg->layers && cfg->layers > 0,
+            "descriptor `mixers` must list all %d layers", cfg->layers);
+  for (int l = 0; l < cfg->layers; l++) {
+    const Json& j = list->arr[l];
+    MixerCfg m;
+    const std::string kind = j.string("type", "");
+    auto num = [&](const char* k) { return (int)j.number(k, 0); };
+    m.tensors = (int)j.number("tensors", l);
+    m.ff = num("ff");
+    m.heads = num("heads"), m.dim = num("dim"), m.vdim = num("vdim");
+    DYN_CHECK(m.tensors >= 0 && m.tensors < cfg->layers && m.ff >= 0, "layer %d: bad `tensors` or `ff`", l);
+    if (kind == "retention") {
+      m.kind = MIX_RETENTION;
+      m.rot_dims = num("rot_dims"), m.rot_base = j.number("rot_base", 0);
+      const Json* d = j.get("decay");
+      DYN_CHECK(d && d->kind == Json::Arr && (int)d->arr.size() == m.heads, "layer %d: one decay per head", l);
+      for (auto& v : d->arr) m.decay.push_back(v.num);
+      DYN_CHECK(m.heads > 0 && m.dim > 0 && m.vdim > 0, "layer %d: retention sizes", l);
+      DYN_CHECK(m.rot_dims >= 0 && m.rot_dims <= m.dim && m.rot_dims % 2 == 0 && (m.rot_dims == 0 || m.rot_base > 0),
+                "layer %d: rotation of %d dims in heads of %d", l, m.rot_dims, m.dim);
+    } else if (kind == "rglru") {
+      m.kind = MIX_RGLRU;
+      m.width = num("width"), m.blocks = num("blocks"), m.taps = num("taps");
+      DYN_CHECK(m.width > 0 && m.blocks > 0 && m.taps > 0 && m.width % m.blocks == 0,
+                "layer %d: recurrence of width %d, %d gate blocks, %d taps", l, m.width, m.blocks, m.taps);
+    } else if (kind == "latent_attention") {
+      m.kind = MIX_LATENT;
+      m.rank = num("rank"), m.scale = (float)j.number("scale", 0);
+      DYN_CHECK(m.heads > 0 && m.dim > 0 && m.vdim > 0 && m.rank > 0 && m.rank <= 1024, "layer %d: latent attention sizes", l);
+    } else {
+      DYN_CHECK(false, "E_KERNEL_COVERAGE: layer %d has a mixer without a cuda kernel: `%s`", l, kind.c_str());
+    }
+    cfg->mixers.push_back(m);
+  }
+  for (int l = 0; l < cfg->layers; l++)
+    DYN_CHECK(cfg->mixers[cfg->mixers[l].tensors].kind == cfg->mixers[l].kind &&
+                  cfg->mixers[cfg->mixers[l].tensors].tensors == cfg->mixers[l].tensors,
+              "layer %d runs with the parameters of layer %d, which has other ones", l, cfg->mixers[l].tensors);
+  return 0;
+}
+
+static std::string layer_name(int l) { return "blk." + std::to_string(l) + "."; }
+
+static std::vector<std::string> input_names(const MixerCfg& m, int l) {
+  const std::string b = layer_name(l);
+  switch (m.kind) {
+    case MIX_RETENTION: return {b + "attn_q.weight", b + "attn_k.weight", b + "attn_v.weight", b + "attn_gate.weight"};
+    case MIX_RGLRU: return {b + "rec_y.weight", b + "rec_x.weight"};
+    default: return {b + "attn_q.weight", b + "attn_kv_down.weight", b + "attn_gate.weight"};
+  }
+}
+
+std::vector<std::vector<std::string>> mixer_place_runs(const ModelCfg& cfg) {
+  std::vector<std::vector<std::string>> runs;
+  for (int l = 0; l < cfg.layers; l++) {
+    const MixerCfg& m = cfg.mixers[l];
+    if (m.tensors != l) continue;
+    const std::string b = layer_name(l);
+    runs.push_back(input_names(m, l));
+    if (m.kind == MIX_LATENT) runs.push_back({b + "attn_k_up.weight", b + "attn_v_up.weight"});
+    if (m.ff) runs.push_back({b + "ffn_gate.weight", b + "ffn_up.weight"});
+  }
+  return runs;
+}
+
+int bind_mixers(Session* s, const ParamTable& t, uint64_t* decode_bytes) {
+  const ModelCfg& c = s->cfg;
+  const int64_t H = c.hidden;
+  s->mix.resize(c.layers);
+  size_t floats = 0;
+  std::vector<size_t> decay_at(c.layers), freq_at(c.layers);
+  for (int l = 0; l < c.layers; l++) {
+    const MixerCfg& m = c.mixers[l];
+    if (m.tensors != l || m.kind != MIX_RETENTION) continue;
+    freq_at[l] = floats, floats += (size_t)m.rot_dims / 2 * 2;  // doubles first, on even offsets
+    floats = (floats + 1) / 2 * 2;
+    decay_at[l] = floats, floats += (m.heads + 1) / 2 * 2;
+  }
+  if (dev_alloc(s, (void**)&s->tables, floats * 4)) return 1;
+  for (int l = 0; l < c.layers; l++) {
+    MixerLayer& L = s->mix[l];
+    const MixerCfg& m = c.mixers[l];
+    L.c = m;
+    if (m.tensors != l) continue;
+    const std::string b = layer_name(l);
+    std::vector<int64_t> in_rows;
+    int64_t out_cols = 0;
+    if (m.kind == MIX_RETENTION) {
+      const int64_t qd = (int64_t)m.heads * m.dim, vd = (int64_t)m.heads * m.vdim;
+      in_rows = {qd, qd, vd, vd}, out_cols = vd;
+      std::vector<double> f(m.rot_dims / 2);
+      for (size_t i = 0; i < f.size(); i++) f[i] = pow(m.rot_base, -2.0 * (double)i / m.rot_dims);
+      std::vector<float> d(m.decay.begin(), m.decay.end());
+      L.freq = reinterpret_cast<double*>(s->tables + freq_at[l]), L.decay = s->tables + decay_at[l];
+      if (!f.empty()) DYN_CUDA(cudaMemcpy(L.freq, f.data(), f.size() * 8, cudaMemcpyHostToDevice));
+      DYN_CUDA(cudaMemcpy(L.decay, d.data(), d.size() * 4, cudaMemcpyHostToDevice));
+    } else if (m.kind == MIX_RGLRU) {
+      in_rows = {m.width, m.width}, out_cols = m.width;
+      const int64_t n = m.width / m.blocks;
+      if (t.plain(b + "rec_y.bias", {m.width}, &L.by) || t.plain(b + "rec_x.bias", {m.width}, &L.bx) ||
+          t.plain(b + "rec_conv.weight", {m.width, m.taps}, &L.conv) || t.plain(b + "rec_conv.bias", {m.width}, &L.bc) ||
+          t.plain(b + "rec_a_gate.weight", {m.blocks, n, n}, &L.ra) || t.plain(b + "rec_a_gate.bias", {m.blocks, n}, &L.bra) ||
+          t.plain(b + "rec_i_gate.weight", {m.blocks, n, n}, &L.ri) || t.plain(b + "rec_i_gate.bias", {m.blocks, n}, &L.bri) ||
+          t.plain(b + "rec_lambda", {m.width}, &L.lam))
+        return 1;
+    } else {
+      const int64_t qd = (int64_t)m.heads * m.dim, vd = (int64_t)m.heads * m.vdim;
+      in_rows = {qd, m.rank, vd}, out_cols = vd;
+      if (t.plain(b + "attn_kv_norm.weight", {m.rank}, &L.lat_norm) ||
+          t.linear(b + "attn_k_up.weight", qd, m.rank, &L.uk) || t.linear(b + "attn_v_up.weight", vd, m.rank, &L.uv))
+        return 1;
+      for (const WRef* w : {&L.uk, &L.uv})
+        DYN_CHECK(w->enc == E_F32 || w->enc == E_F16 || w->enc == E_BF16, "layer %d: latent up-projections must be a plain type", l);
+      if (follows_in_arena(L.uk, L.uv)) L.ukv = L.uk, L.ukv.rows += L.uv.rows;
+    }
+    const auto names = input_names(m, l);
+    L.parts = (int)names.size();
+    WRef prev;
+    for (int p = 0; p < L.parts; p++) {
+      WRef w;
+      if (t.linear(names[p], in_rows[p], H, &w)) return 1;
+      if (p && follows_in_arena(prev, w)) {
+        L.part_col[p] = L.in.back().rows;
+        L.in.back().rows += w.rows;
+      } else {
+        L.part_col[p] = 0;
+        L.in.push_back(w);
+      }
+      L.part_in[p] = (int)L.in.size() - 1;
+      prev = w;
+    }
+    if (t.plain(b + "attn_norm.weight", {H}, &L.norm1) ||
+        t.linear(b + (m.kind == MIX_RGLRU ? "rec_output.weight" : "attn_output.weight"), H, out_cols, &L.o))
+      return 1;
+    if (m.ff) {
+      if (t.plain(b + "ffn_norm.weight", {H}, &L.norm2) || t.linear(b + "ffn_gate.weight", m.ff, H, &L.gate) ||
+          t.linear(b + "ffn_up.weight", m.ff, H, &L.up) || t.linear(b + "ffn_down.weight", H, m.ff, &L.down))
+        return 1;
+      if (follows_in_arena(L.gate, L.up)) L.gate_up = L.gate, L.gate_up.rows += L.up.rows;
+    }
+  }
+  // layers that run with another layer's parameters; state regions
+  size_t off = 0;
+  for (int l = 0; l < c.layers; l++) {
+    const MixerCfg& m = c.mixers[l];
+    if (m.tensors != l) {
+      s->mix[l] = s->mix[m.tensors];
+      s->mix[l].c = m;
+      DYN_CHECK(c.mixers[m.tensors].heads == m.heads && c.mixers[m.tensors].dim == m.dim && c.mixers[m.tensors].vdim == m.vdim &&
+                    c.mixers[m.tensors].width == m.width && c.mixers[m.tensors].blocks == m.blocks &&
+                    c.mixers[m.tensors].taps == m.taps && c.mixers[m.tensors].rank == m.rank &&
+                    c.mixers[m.tensors].rot_dims == m.rot_dims && c.mixers[m.tensors].ff == m.ff,
+                "layer %d runs with the parameters of layer %d but has other sizes", l, m.tensors);
+    }
+    MixerLayer& L = s->mix[l];
+    L.state_floats = m.kind == MIX_RETENTION ? (size_t)m.heads * m.dim * m.vdim : m.kind == MIX_RGLRU ? (size_t)m.width : 0;
+    L.ring_floats = m.kind == MIX_RGLRU ? (size_t)m.taps * m.width : 0;
+    auto region = [&](size_t per_slot) {
+      const size_t at = off;
+      off += ((size_t)c.batch * per_slot + 63) / 64 * 64;
+      return at;
+    };
+    L.state_off = region(L.state_floats);
+    L.ring_off = region(L.ring_floats);
+    for (const WRef& w : L.in) *decode_bytes += w.total_bytes();
+    for (const WRef* w : {&L.o, &L.gate, &L.up, &L.down, &L.uk, &L.uv})
+      if (w->data) *decode_bytes += w->total_bytes();
+    for (const NormW* w : {&L.norm1, &L.norm2, &L.by, &L.bx, &L.conv, &L.bc, &L.ra, &L.bra, &L.ri, &L.bri, &L.lam, &L.lat_norm})
+      *decode_bytes += w->bytes;
+  }
+  s->state_floats = off;
+  s->slot_pos.assign((size_t)c.batch, 0);
+  return 0;
+}
+
+size_t mixer_cache_elements(const ModelCfg& cfg) {
+  size_t n = 0;
+  for (const MixerCfg& m : cfg.mixers) n += m.kind == MIX_LATENT ? m.rank : 0;
+  return n;
+}
+
+static Vec vec(const NormW& w) {
+  Vec v;
+  v.ptr = reinterpret_cast<const uint8_t*>(w.ptr), v.type = w.type;
+  return v;
+}
+
+static int64_t input_width(const MixerLayer& L) {
+  int64_t n = 0;
+  for (const WRef& w : L.in) n += w.rows;
+  return n;
+}
+
+// Where part p of the layer's input products lies when the products of `rows` rows are written to `buf`
+// one after the other.
+static Rows part_rows(const MixerLayer& L, float* buf, int64_t rows, int p) {
+  for (int i = 0; i < L.part_in[p]; i++) buf += rows * L.in[i].rows;
+  Rows r;
+  r.ptr = buf + L.part_col[p], r.ld = L.in[L.part_in[p]].rows;
+  return r;
+}
+
+static uint8_t* latent_plane(Session* s, int layer, int64_t cap) {
+  size_t elems = 0;
+  for (int l = 0; l < layer; l++)
+    if (s->mix[l].c.kind == MIX_LATENT) elems += (size_t)s->cfg.batch * cap * s->mix[l].c.rank;
+  return s->lcache + elems * s->kv_elem;
+}
+
+static RetentionArgs retention_args(Session* s, const MixerLayer& L, int64_t rows) {
+  RetentionArgs a;
+  a.q = part_rows(L, s->qkv1, rows, 0), a.k = part_rows(L, s->qkv1, rows, 1);
+  a.v = part_rows(L, s->qkv1, rows, 2), a.g = part_rows(L, s->qkv1, rows, 3);
+  a.heads = L.c.heads, a.dim = L.c.dim, a.vdim = L.c.vdim, a.rot_dims = L.c.rot_dims;
+  a.freq = L.freq, a.decay = L.decay;
+  a.state = s->state + L.state_off, a.out = s->ctx, a.scratch = s->mix_scratch, a.eps = s->cfg.eps;
+  return a;
+}
+
+static RglruArgs rglru_args(Session* s, const MixerLayer& L, int64_t rows) {
+  RglruArgs a;
+  a.y = part_rows(L, s->qkv1, rows, 0), a.x = part_rows(L, s->qkv1, rows, 1);
+  a.width = L.c.width, a.blocks = L.c.blocks, a.taps = L.c.taps;
+  a.by = vec(L.by), a.bx = vec(L.bx), a.conv = vec(L.conv), a.bc = vec(L.bc), a.ra = vec(L.ra), a.bra = vec(L.bra);
+  a.ri = vec(L.ri), a.bri = vec(L.bri), a.lam = vec(L.lam);
+  a.state = s->state + L.state_off, a.ring = s->state + L.ring_off;
+  a.out = s->ctx, a.scratch = s->mix_scratch, a.exact = s->cfg.exact;
+  return a;
+}
+
+static LatentArgs latent_args(Session* s, const MixerLayer& L, int layer, int64_t rows, int64_t cap) {
+  LatentArgs a;
+  a.q = part_rows(L, s->qkv1, rows, 0), a.d = part_rows(L, s->qkv1, rows, 1), a.g = part_rows(L, s->qkv1, rows, 2);
+  a.heads = L.c.heads, a.dim = L.c.dim, a.vdim = L.c.vdim, a.rank = L.c.rank;
+  a.scale = L.c.scale, a.eps = s->cfg.eps, a.norm = vec(L.lat_norm);
+  a.uk = L.uk, a.uv = L.uv, a.ukv = L.ukv;
+  a.cache = latent_plane(s, layer, cap), a.kv_type = s->kv_type, a.cap = cap;
+  a.out = s->ctx, a.scratch = s->mix_scratch, a.exact = s->cfg.exact, a.max_rows = s->max_rows;
+  return a;
+}
+
+static int grow_mix_scratch(Session* s, int64_t rows, int64_t cap) {
+  size_t need = 0;
+  for (int l = 0; l < s->cfg.layers; l++) {
+    const MixerLayer& L = s->mix[l];
+    if (L.c.kind == MIX_RETENTION) need = std::max(need, retention_scratch_floats(retention_args(s, L, rows), rows));
+    else if (L.c.kind == MIX_RGLRU) need = std::max(need, rglru_scratch_floats(rglru_args(s, L, rows), rows));
+    else need = std::max(need, latent_scratch_floats(latent_args(s, L, l, rows, cap), rows));
+  }
+  if (need <= s->mix_scratch_floats) return 0;
+  dev_free(s, s->mix_scratch, s->mix_scratch_floats * 4);
+  s->mix_scratch = nullptr, s->mix_scratch_floats = 0;
+  if (dev_alloc(s, (void**)&s->mix_scratch, need * 4)) return 1;
+  s->mix_scratch_floats = need;
+  return 0;
+}
+
+// Activation scratch and the recurrent state, at the first configuration.
+int configure_mixers(Session* s, int64_t rows) {
+  const ModelCfg& c = s->cfg;
+  int64_t proj = 0, ctx = 0, ff = 0;
+  for (const MixerLayer& L : s->mix) {
+    proj = std::max(proj, input_width(L));
+    ctx = std::max(ctx, L.o.cols);
+    ff = std::max<int64_t>(ff, L.c.ff);
+  }
+  const int64_t wide = std::max({(int64_t)c.hidden, ctx, ff}), alloc = rows + rows / 2 + 64;
+  if (dev_alloc(s, (void**)&s->hidden, (size_t)rows * c.hidden * 4) ||
+      dev_alloc(s, (void**)&s->xn, (size_t)rows * c.hidden * 4) ||
+      dev_alloc(s, (void**)&s->ctx, (size_t)rows * ctx * 4) ||
+      dev_alloc(s, (void**)&s->act, (size_t)rows * std::max<int64_t>(1, ff) * 4) ||
+      (!c.exact && rows >= 64 &&
+       (dev_alloc(s, (void**)&s->xh, (size_t)alloc * wide * 2) || dev_alloc(s, (void**)&s->xinv, (size_t)alloc * 4) ||
+        dev_alloc(s, (void**)&s->gpart, (size_t)8 * rows * c.hidden * 4))) ||
+      dev_alloc(s, (void**)&s->qkv1, (size_t)rows * proj * 4) ||
+      dev_alloc(s, (void**)&s->gu1, (size_t)rows * 2 * std::max<int64_t>(1, ff) * 4) ||
+      dev_alloc(s, (void**)&s->tokens_dev, (size_t)rows * 8) || dev_alloc(s, (void**)&s->row_pos_dev, (size_t)rows * 8) ||
+      dev_alloc(s, (void**)&s->row_seq_dev, (size_t)rows * 8) ||
+      host_alloc(s, (void**)&s->stage_host, (size_t)(8 + 3 * rows) * 8) ||
+      dev_alloc(s, (void**)&s->state, s->state_floats * 4))
+    return 1;
+  if (s->xh) s->xh_rows = alloc, s->xh_cols = wide, s->gpart_bytes = (size_t)8 * rows * c.hidden * 4;
+  s->max_rows = rows;
+  DYN_CUDA(cudaMemset(s->state, 0, s->state_floats * 4));
+  return 0;
+}
+
+int ensure_mixer_pages(Session* s, size_t page_count) {
+  const ModelCfg& c = s->cfg;
+  const int64_t cap = (int64_t)(page_count * s->page_size), old = (int64_t)(s->pages * s->page_size);
+  const size_t bytes = mixer_cache_elements(c) * c.batch * (size_t)cap * s->kv_elem;
+  uint8_t* fresh = nullptr;
+  if (bytes) {
+    if (dev_alloc(s, (void**)&fresh, bytes)) return 1;
+    DYN_CUDA(cudaMemsetAsync(fresh, 0, bytes, s->stream));
+    if (s->pages) {  // keep what is cached: every layer's slots are planes of their own
+      size_t from = 0, to = 0;
+      for (const MixerLayer& L : s->mix) {
+        if (L.c.kind != MIX_LATENT) continue;
+        const size_t src = (size_t)old * L.c.rank * s->kv_elem, dst = (size_t)cap * L.c.rank * s->kv_elem;
+        DYN_CUDA(cudaMemcpy2DAsync(fresh + to, dst, s->lcache + from, src, src, (size_t)c.batch, cudaMemcpyDeviceToDevice, s->stream));
+        from += src * c.batch, to += dst * c.batch;
+      }
+    }
+    DYN_CUDA(cudaStreamSynchronize(s->stream));
+    dev_free(s, s->lcache, s->lcache_bytes);
+    s->lcache = fresh, s->lcache_bytes = bytes;
+  }
+  return grow_mix_scratch(s, s->max_rows, cap);
+}
+
+int reset_mixers(Session* s) {
+  if (s->lcache) DYN_CUDA(cudaMemsetAsync(s->lcache, 0, s->lcache_bytes, s->stream));
+  if (s->state_floats) DYN_CUDA(cudaMemsetAsync(s->state, 0, s->state_floats * 4, s->stream));
+  DYN_CUDA(cudaStreamSynchronize(s->stream));
+  std::fill(s->slot_pos.begin(), s->slot_pos.end(), 0);
+  return 0;
+}
+
+int mixer_check_position(Session* s, int64_t slot, int64_t start) {
+  if (s->cfg.mixers.empty() || start == 0) return 0;
+  const int64_t at = s->slot_pos[(size_t)slot];
+  DYN_CHECK(at >= 0, "slot %lld: its last step failed, the sequence must start over at position 0", (long long)slot);
+  DYN_CHECK(start == at, "slot %lld is at position %lld: recurrent state cannot continue at %lld", (long long)slot,
+            (long long)at, (long long)start);
+  return 0;
+}
+
+int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t chunk_slot) {
+  const ModelCfg& c = s->cfg;
+  cudaStream_t st = s->stream;
+  const int64_t H = c.hidden, cap = (int64_t)(s->pages * s->page_size);
+  StepRows step;
+  step.rows = rows, step.pos = s->row_pos_dev, step.seq = s->row_seq_dev;
+  step.base = chunk_start, step.slot = chunk_slot;
+  // Many rows whose products all go to the dequant GEMM: the norm kernels write its operand themselves and
+  // the K-split sums of the output and down projections are added inside the norm that follows.
+  bool fuse = !c.exact && rows >= 64 && s->xh && H <= 8192;
+  for (const MixerLayer& L : s->mix) {
+    auto takes = [&](const WRef& w) {
+      return !w.data || (dqgemm_tc_takes(w, rows) && dqgemm_tc_padded_rows(w, rows) <= s->xh_rows);
+    };
+    for (const WRef& w : L.in) fuse = fuse && takes(w);
+    for (const WRef* w : {&L.o, &L.gate, &L.up, &L.down}) fuse = fuse && takes(*w);
+  }
+  int pending = 0;  // K-split sums in gpart that `hidden` still lacks
+  auto norm = [&](const NormW& w) -> int {
+    if (!fuse) return launch_rms_norm(s->hidden, w.ptr, w.type, rows, H, c.eps, s->xn, st);
+    const int splits = pending;
+    pending = 0;
+    return splits > 1 ? launch_norm_prepare(nullptr, s->gpart, splits, s->hidden, s->hidden, w.ptr, w.type, rows, H, c.eps,
+                                            s->xh, s->xinv, st)
+                      : launch_norm_prepare(s->hidden, nullptr, 0, nullptr, nullptr, w.ptr, w.type, rows, H, c.eps, s->xh,
+                                            s->xinv, st);
+  };
+  auto gemm = [&](const WRef& w, const float* x, float* y, const float* residual, bool defer) -> int {
+    TgIo io;
+    if (!x) io.xh = s->xh, io.inv_s = s->xinv, io.rows_alloc = s->xh_rows;  // the prepared operand
+    if (defer) io.partial = s->gpart, io.partial_bytes = s->gpart_bytes;
+    bool handled = false;
+    if (launch_dqgemm_tc(w, x, E_F32, rows, y, residual, st, &handled, &io)) return 1;
+    DYN_CHECK(handled, "dequant GEMM refused a product it had accepted");
+    if (defer) pending = io.splits;
+    return 0;
+  };
+  // a product of the normalised rows
+  auto from_norm = [&](const WRef& w, float* y) -> int {
+    return fuse ? gemm(w, nullptr, y, nullptr, false) : session_linear(s, w, s->xn, E_F32, rows, y, nullptr);
+  };
+  // hidden += W x; `last`: no norm of this function follows to add deferred sums
+  auto to_hidden = [&](const WRef& w, const float* x, bool prepared, bool last) -> int {
+    return fuse ? gemm(w, prepared ? nullptr : x, s->hidden, s->hidden, !last)
+                : session_linear(s, w, x, E_F32, rows, s->hidden, s->hidden);
+  };
+  for (int l = 0; l < c.layers; l++) {
+    const MixerLayer& L = s->mix[l];
+    const bool final_layer = l + 1 == c.layers;
+    if (norm(L.norm1)) return 1;
+    float* y = s->qkv1;
+    for (const WRef& w : L.in) {
+      if (from_norm(w, y)) return 1;
+      y += rows * w.rows;
+    }
+    int rc;
+    switch (L.c.kind) {
+      case MIX_RETENTION: rc = launch_retention(retention_args(s, L, rows), step, st); break;
+      case MIX_RGLRU: rc = launch_rglru(rglru_args(s, L, rows), step, st); break;
+      default: rc = launch_latent_attention(latent_args(s, L, l, rows, cap), step, st);
+    }
+    if (rc || to_hidden(L.o, s->ctx, false, final_layer && !L.c.ff)) return 1;
+    if (!L.c.ff) continue;
+    if (norm(L.norm2)) return 1;
+    bool prepared = false;
+    if (L.gate_up.data) {
+      if (from_norm(L.gate_up, s->gu1)) return 1;
+      prepared = fuse;
+      if (fuse ? launch_silu_prepare(s->gu1, rows, L.c.ff, s->xh, s->xinv, st)
+               : launch_silu_mul_rows(s->gu1, rows, L.c.ff, s->act, st))
+        return 1;
+    } else {
+      float* up = s->gu1 + rows * L.c.ff;
+      if (from_norm(L.gate, s->gu1) || from_norm(L.up, up) || launch_silu_mul(s->gu1, up, rows * L.c.ff, s->act, st)) return 1;
+    }
+    if (to_hidden(L.down, s->act, prepared, final_layer)) return 1;
+  }
+  return 0;
+}
+
+}  // namespace dyn

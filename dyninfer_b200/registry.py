@@ -15,7 +15,9 @@ from dataclasses import dataclass, field
 
 OPERATIONS = ("Input", "Embedding", "Linear", "RmsNorm", "PerHeadRmsNorm", "Rope", "KvCacheWrite",
               "KvCacheRead", "Attention", "ShortConv", "Silu", "Multiply", "Residual",
-              "OutputProjection")
+              "OutputProjection",
+              # mixers beyond the reference's GQA attention
+              "Retention", "GatedRecurrence", "LatentAttention", "OutputGate")
 MODES = ("prefill", "decode")
 
 
@@ -144,7 +146,7 @@ CUDA_SM100 = TargetConstraint(("cuda",), ("sm_100a", "sm_100"), ())
 # (encoding, elements per block along the input axis)
 CUDA_ENCODINGS = (("gguf.q4_0", 32), ("gguf.q4_1", 32), ("gguf.q8_0", 32), ("gguf.q6_k", 256),
                   ("gguf.q4_k", 256), ("gguf.q5_k", 256), ("gguf.iq4_xs", 256),
-                  ("mlx.affine.u4", 64), ("plain.bf16", 4), ("plain.f16", 4), ("plain.f32", 4))
+                  ("mlx.affine.u4", 64), ("plain.bf16", 1), ("plain.f16", 1), ("plain.f32", 1))
 
 
 def register_cuda_candidates(reg: KernelRegistry) -> KernelRegistry:
@@ -162,7 +164,11 @@ def register_cuda_candidates(reg: KernelRegistry) -> KernelRegistry:
                     ("Rope", "rope.cuda_sm100.f32"), ("KvCacheWrite", "kv_cache.write.cuda_sm100"),
                     ("KvCacheRead", "kv_cache.read.cuda_sm100"),
                     ("Attention", "attention.gqa.cuda_sm100"), ("Silu", "silu.cuda_sm100.f32"),
-                    ("Multiply", "multiply.cuda_sm100.f32"), ("Residual", "residual.cuda_sm100.f32")):
+                    ("Multiply", "multiply.cuda_sm100.f32"), ("Residual", "residual.cuda_sm100.f32"),
+                    ("ShortConv", "short_conv.cuda_sm100.f32"), ("Retention", "retention.cuda_sm100.f32"),
+                    ("GatedRecurrence", "rglru.cuda_sm100.f32"),
+                    ("LatentAttention", "attention.latent.cuda_sm100"),
+                    ("OutputGate", "output_gate.cuda_sm100.f32")):
         reg.register(KernelCandidate(id=kid, operation=op, encoding=None, target=CUDA_SM100,
                                      deterministic_score=200, lowering=kid))
     return reg
@@ -186,6 +192,41 @@ def default_registry() -> KernelRegistry:
     return register_cuda_candidates(register_builtin_semantic_candidates(KernelRegistry()))
 
 
+def _mixer_operations(config: dict, par):
+    """The layers of a decoder whose configuration lists a mixer per layer. Layers that run with another
+    layer's parameters ask for the same products again."""
+    ops = []
+    for l, m in enumerate(config["mixers"]):
+        p, t = f"blk.{l}.", f"blk.{m['tensors']}."
+
+        def linear(*names):
+            return [(p + n, "Linear", *par(t + n + ".weight")) for n in names]
+
+        ops.append((p + "attn_norm", "RmsNorm", None, None))
+        if m["type"] == "retention":
+            ops += linear("attn_q", "attn_k", "attn_v", "attn_gate")
+            if m["rot_dims"]:
+                ops += [(p + "rope_q", "Rope", None, None), (p + "rope_k", "Rope", None, None)]
+            ops += [(p + "retention", "Retention", None, None), (p + "head_norm", "PerHeadRmsNorm", None, None),
+                    (p + "output_gate", "OutputGate", None, None), *linear("attn_output")]
+        elif m["type"] == "rglru":
+            ops += [*linear("rec_y", "rec_x"), (p + "rec_conv", "ShortConv", None, None),
+                    (p + "recurrence", "GatedRecurrence", None, None),
+                    (p + "output_gate", "OutputGate", None, None), *linear("rec_output")]
+        else:
+            ops += [*linear("attn_q", "attn_kv_down", "attn_gate"), (p + "attn_kv_norm", "RmsNorm", None, None),
+                    (p + "kv_write_latent", "KvCacheWrite", None, None), *linear("attn_k_up", "attn_v_up"),
+                    (p + "kv_read_latent", "KvCacheRead", None, None),
+                    (p + "attention", "LatentAttention", None, None),
+                    (p + "output_gate", "OutputGate", None, None), *linear("attn_output")]
+        ops.append((p + "mixer_residual", "Residual", None, None))
+        if m["ff"]:
+            ops += [(p + "ffn_norm", "RmsNorm", None, None), *linear("ffn_gate", "ffn_up"),
+                    (p + "ffn_silu", "Silu", None, None), (p + "ffn_mul", "Multiply", None, None),
+                    *linear("ffn_down"), (p + "ffn_residual", "Residual", None, None)]
+    return ops
+
+
 def decoder_operations(config: dict, parameters: dict):
     """(operation id, kind, encoding, logical shape) for every op of the decoder graph in the
     order fixed by crates/dyninfer-architecture/src/builder.rs:491-614,664-718.
@@ -196,7 +237,9 @@ def decoder_operations(config: dict, parameters: dict):
 
     ops = [("input.tokens", "Input", None, None),
            ("embed", "Embedding", *par("token_embd.weight"))]
-    for l in range(config["layers"]):
+    if config.get("mixers"):
+        ops += _mixer_operations(config, par)
+    for l in range(0 if config.get("mixers") else config["layers"]):
         p = f"blk.{l}."
         ops.append((p + "attn_norm", "RmsNorm", None, None))
         for s in ("attn_q", "attn_k", "attn_v"):

@@ -111,7 +111,7 @@ class CudaSession:
             kv_heads = desc["kv_heads"]
         else:
             desc = ck.model_descriptor(model.catalog, kv_dtype=self.kv_dtype, decode_kernel=model.decode_kernel,
-                                       batch=max(1, int(config.batch_size)))
+                                       batch=max(1, int(config.batch_size)), compute=model.compute)
             ranges = [(p.external_key, p.source_file_index, p.offset, p.length) for p in model.plan.parameters]
         self._keys = [r[0].encode() for r in ranges]
         params = (_lib.FileParam * len(self._keys))(
@@ -239,6 +239,47 @@ class CudaSession:
         self.position_ += 1
         return lg, nxt
 
+    def _portion(self, tokens, want, start: int, slot: int):
+        """Runs `tokens` of one sequence from position `start`; logits of the rows in `want`, and the argmax
+        of the last row. Longer portions go through the native session in pieces of the chunk size."""
+        tokens = np.ascontiguousarray(tokens, dtype=np.int64)
+        want = [int(w) for w in want]
+        if not tokens.size:
+            raise DynInferError("a portion requires a non-empty token list")
+        if start + tokens.size > self._max_seq():
+            raise DynInferError(f"position {start + tokens.size} exceeds session/KV limit {self._max_seq()}")
+        if any(not 0 <= w < tokens.size for w in want):
+            raise DynInferError(f"wanted rows outside the portion of {tokens.size} tokens")
+        self._ensure_pages()
+        i64p = C.POINTER(C.c_int64)
+        vocab = self.metadata["vocabulary_size"]
+        out = np.empty((len(want), vocab), dtype=np.float32)
+        tok = C.c_int64(-1)
+        for lo in range(0, tokens.size, self.model.chunk_size):
+            piece = tokens[lo:lo + self.model.chunk_size]
+            rows = sorted({w - lo for w in want if lo <= w < lo + piece.size})
+            idx = np.array(rows, dtype=np.int64)
+            ptr = C.POINTER(C.c_float)()
+            check(lib().dyninfer_cuda_session_invoke_portion(
+                self._h, piece.ctypes.data_as(i64p), piece.size, start + lo, slot,
+                idx.ctypes.data_as(i64p) if rows else None, len(rows), C.byref(ptr), C.byref(tok)))
+            if rows:
+                got = np.ctypeslib.as_array(ptr, shape=(len(rows), vocab))
+                at = {r: i for i, r in enumerate(rows)}
+                for i, w in enumerate(want):
+                    if w - lo in at:
+                        out[i] = got[at[w - lo]]
+        return out, int(tok.value)
+
+    def extend(self, tokens, want=()) -> np.ndarray:
+        """Runs `tokens` from the current position on; logits [len(want), vocab] of the rows `want` of this
+        portion. Prompts may be fed in portions cut anywhere."""
+        self._require_batch_1()
+        logits, _ = self._portion(tokens, want, self.position_, 0)
+        self.history.extend(int(t) for t in tokens)
+        self.position_ += len(tokens)
+        return logits
+
     # -- ModelSession
     def prefill(self, tokens) -> Logits:
         lg, _ = self._prefill(tokens, True)
@@ -272,11 +313,11 @@ class CudaSession:
 
     def kv_cache_metrics(self) -> KvCacheMetrics:
         cfg = self.model.catalog.config
-        per_token = cfg["layers"] * cfg["kv_heads"] * cfg["head_dim"] * self.kv_elem * 2
+        per_token = self.kv_elem * cfg.get("kv_elements_per_token", cfg["layers"] * cfg["kv_heads"] * cfg["head_dim"] * 2)
         pages = lib().dyninfer_cuda_session_kv_page_count(self._h)
         alloc = lib().dyninfer_cuda_session_kv_allocated_bytes(self._h)
         return KvCacheMetrics(page_count=pages, allocated_bytes=alloc,
-                              capacity_bytes=per_token * self.max_kv, used_bytes=alloc,
+                              capacity_bytes=per_token * self.max_kv + cfg.get("state_bytes_per_slot", 0), used_bytes=alloc,
                               filled_tokens=self.position_, layers=cfg["layers"],
                               kv_heads=cfg["kv_heads"], head_dim=cfg["head_dim"],
                               max_sequence_length=self.max_kv, key_dtype=self.kv_dtype,
@@ -358,7 +399,7 @@ class LoadedModel:
     def __init__(self, catalog: ck.Catalog, plan: ck.ProviderPlan, target: reg.TargetProfile,
                  device_uri: str, coverage: reg.CoverageReport, max_kv: int, kv_dtype: str,
                  chunk_size: int, decode_kernel: str = "persistent", tp: tuple | None = None,
-                 tp_exchange: str = "peer"):
+                 tp_exchange: str = "peer", compute: str = "serve"):
         self.catalog, self.plan, self.target, self.device_uri = catalog, plan, target, device_uri
         # (rank, world) of a tensor-parallel group: one process per GPU, every process loads the
         # same checkpoint and uploads its own slices; torch.distributed must be initialised
@@ -371,6 +412,12 @@ class LoadedModel:
         # "persistent": one cooperative kernel per decoded token; "graph": a captured graph of
         # per-operator kernels (the path multi-row chunks always take)
         self.decode_kernel = decode_kernel
+        # "serve": the kernels and precisions models are served with; "f32": every product in f32
+        if compute not in ("serve", "f32"):
+            raise DynInferError(f"compute `{compute}` unknown (serve | f32)")
+        if self.tp and (compute != "serve" or catalog.config.get("mixers")):
+            raise DynInferError("tensor parallelism covers GQA decoders in serving precision only")
+        self.compute = compute
         c = catalog.config
         self.metadata = {"architecture": c.get("model_type", "qwen3"), "vocabulary_size": c["vocab"],
                          "context_length": c.get("context_length", 0), "pad_token_id": 0}
@@ -422,6 +469,16 @@ class BatchedCudaSession(CudaSession):
                 logits = np.ctypeslib.as_array(ptr, shape=(count.value,)).copy()
         self.positions[slot] = len(tokens)
         return (logits, token) if want_logits else token
+
+    def extend_slot(self, slot: int, tokens, want=(), restart: bool = False) -> np.ndarray:
+        """A portion of the sequence in KV slot `slot` (from position 0 with `restart`, which is how a slot is
+        given to a new sequence); logits of the rows in `want`."""
+        if not 0 <= slot < self.slots:
+            raise DynInferError(f"slot {slot} outside [0, {self.slots})")
+        start = 0 if restart else self.positions[slot]
+        logits, _ = self._portion(tokens, want, start, int(slot))
+        self.positions[slot] = start + len(tokens)
+        return logits
 
     def step(self, tokens: dict, want_logits: bool = False):
         """One decode step: `tokens` maps slot -> token to feed. Returns slot -> next token
@@ -485,13 +542,13 @@ class ModelLoader:
 
     def load(self, path: str, target: str = "cuda", max_kv: int = 2048, kv_dtype: str = "f32",
              chunk_size: int = CHUNK_SIZE, decode_kernel: str = "persistent",
-             tp: tuple | None = None, tp_exchange: str = "peer") -> LoadedModel:
+             tp: tuple | None = None, tp_exchange: str = "peer", compute: str = "serve") -> LoadedModel:
         profile, uri = self.resolve_target(target)
         catalog = self.bind(path)
         coverage = self.kernel_coverage(catalog, profile).require_complete()
         plan = ck.build_runtime_provider_plan(catalog)
         return LoadedModel(catalog, plan, profile, uri, coverage, max_kv, kv_dtype, chunk_size, decode_kernel, tp,
-                           tp_exchange)
+                           tp_exchange, compute)
 
 
 # ----------------------------------------------------------------------- generation

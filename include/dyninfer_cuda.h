@@ -230,6 +230,18 @@ int dyninfer_cuda_session_invoke_paged_chunk_slot(dyninfer_cuda_session_t* sessi
                                                   float** out_logits, size_t* out_count,
                                                   int64_t* out_token, int want_logits);
 
+/* A portion of a sequence with the logits of chosen rows: tokens [0, count), 1 <= count <= chunk size, at
+ * positions start_pos .. of KV slot `slot`; want[0 .. want_count) are distinct row numbers inside the
+ * portion. *out_logits (session scratch, valid until the next call) points at [want_count, vocab] floats in
+ * the order of `want`, NULL when nothing is wanted; *out_token is the argmax of the last row. A sequence may
+ * be cut into portions anywhere. Models with recurrent state continue only where the slot stands: start_pos
+ * is 0 (the slot starts over) or the position after the slot's last step. No counterpart in the
+ * reference, whose chunk call returns one row. */
+int dyninfer_cuda_session_invoke_portion(dyninfer_cuda_session_t* session, const int64_t* tokens,
+                                         size_t count, int64_t start_pos, int64_t slot,
+                                         const int64_t* want, size_t want_count, float** out_logits,
+                                         int64_t* out_token);
+
 /* One decode step for `count` sequences at once (count <= "batch"): row i feeds tokens[i] at
  * positions[i] into slot slots[i] (all slots distinct) and out_tokens[i] receives the first strict
  * maximum of its logits. With want_logits != 0, *out_logits points at [count, vocab] floats of

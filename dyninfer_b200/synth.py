@@ -289,3 +289,63 @@ def write_qwen3_mlx(dirpath: str, cfg: dict, seed: int = 0, group: int = 64,
     with open(os.path.join(dirpath, "config.json"), "w") as f:
         json.dump(hf_cfg, f)
     return dirpath
+
+
+def zupudra_shapes(doc: dict) -> dict:
+    """Tensor name -> shape of a Zupudra configuration (tensors of layers that share another's are absent)."""
+    W = doc["width"]
+    out = {"embed": (doc["vocab"], W), "final.norm": (W,)}
+    for i, layer in enumerate(doc["layers"]):
+        if layer.get("weights_of") is not None:
+            continue
+        m, p, mx = layer["mixer"], f"l{i}.", f"l{i}.mix."
+        out[p + "norm1"] = (W,)
+        if layer["type"] == "retention":
+            qd, vd = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            out.update({mx + "q": (qd, W), mx + "k": (qd, W), mx + "v": (vd, W), mx + "g": (vd, W), mx + "o": (W, vd)})
+        elif layer["type"] == "rglru":
+            n, b = m["width"], m["blocks"]
+            out.update({mx + "y": (n, W), mx + "y.b": (n,), mx + "x": (n, W), mx + "x.b": (n,), mx + "conv": (n, m["conv"]),
+                        mx + "conv.b": (n,), mx + "ra": (b, n // b, n // b), mx + "ra.b": (b, n // b),
+                        mx + "ri": (b, n // b, n // b), mx + "ri.b": (b, n // b), mx + "lam": (n,), mx + "o": (W, n)})
+        else:
+            qd, vd, r = m["heads"] * m["dim"], m["heads"] * m["vdim"], m["kv_rank"]
+            out.update({mx + "q": (qd, W), mx + "dkv": (r, W), mx + "dkv.norm": (r,), mx + "uk": (qd, r), mx + "uv": (vd, r),
+                        mx + "g": (vd, W), mx + "o": (W, vd)})
+        if layer.get("mlp"):
+            ff = layer["mlp"]["ff"]
+            out.update({p + "norm2": (W,), p + "mlp.gate": (ff, W), p + "mlp.up": (ff, W), p + "mlp.down": (W, ff)})
+    return out
+
+
+def zupudra_tensors(doc: dict, seed: int = 0, dtype=np.float32) -> dict:
+    """Seeded random weights: matrices of unit gain, norms and biases around 1 and 0, recurrences that
+    forget over a few to a few hundred tokens."""
+    out = {}
+    for name, shape in zupudra_shapes(doc).items():
+        rng = np.random.default_rng(tensor_seed(seed, name))
+        if name.endswith("norm") or name.endswith(("norm1", "norm2")):
+            w = rng.uniform(0.7, 1.3, size=shape)
+        elif name.endswith(".lam"):
+            w = rng.uniform(-6.0, -1.0, size=shape)
+        elif name.endswith(".b"):
+            w = rng.normal(0.0, 0.3, size=shape)
+        elif name.endswith(".conv"):
+            w = rng.normal(0.0, shape[-1] ** -0.5, size=shape)
+        elif name == "embed":
+            w = rng.normal(0.0, 1.0, size=shape)
+        else:
+            w = rng.normal(0.0, shape[-1] ** -0.5, size=shape)
+        out[name] = w.astype(dtype)
+    return out
+
+
+def write_zupudra(dirpath: str, doc: dict, seed: int = 0, tensors: dict | None = None) -> str:
+    """Seeded Zupudra directory (config.json + bf16 model.safetensors). `tensors` replaces the random weights."""
+    os.makedirs(dirpath, exist_ok=True)
+    t = zupudra_tensors(doc, seed) if tensors is None else tensors
+    ck.write_safetensors(os.path.join(dirpath, "model.safetensors"),
+                         {k: ("BF16", v.shape, f32_to_bf16_bits(np.ascontiguousarray(v, np.float32))) for k, v in t.items()})
+    with open(os.path.join(dirpath, "config.json"), "w") as f:
+        json.dump(dict(doc, architecture="Zupudra"), f)
+    return dirpath

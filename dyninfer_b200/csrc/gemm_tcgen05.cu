@@ -5,9 +5,9 @@
 //   * sixteen warps dequantise (four groups of four, one pipeline stage each): for every 64-wide K chunk
 //     they decode the raw checkpoint blocks of the tile's 128 rows (every quantised encoding with word
 //     fetches issued a step ahead and packed f16 / f32 arithmetic that rounds like the decoders of
-//     codec.cuh; plain f32 / f16 / bf16 weights through those decoders) and round to f16. Q4_0, Q4_1,
-//     Q8_0, MLX-U4, Q4_K, Q5_K and IQ4_XS write the A operand into tensor memory (tcgen05.st, thread =
-//     weight row, column = two consecutive K elements); Q6_K and the plain types store it in shared
+//     codec.cuh; plain f32 weights through those decoders) and round to f16. Q4_0, Q4_1,
+//     Q8_0, MLX-U4, Q4_K, Q5_K, IQ4_XS and plain f16 / bf16 write the A operand into tensor memory (tcgen05.st, thread =
+//     weight row, column = two consecutive K elements); Q6_K and plain f32 store it in shared
 //     memory in the canonical K-major 128-byte-swizzled layout (8-row groups of 1024 bytes, 16-byte
 //     chunk c of row r at position c ^ (r & 7));
 //   * one thread of another warp fetches the matching activation chunk (f16, prepared once per call, or
@@ -53,8 +53,9 @@ __host__ __device__ constexpr int tg_conversion_index(int warp) { return warp; }
 // cycle, more than the chunk's 512 tensor-pipe cycles.
 __host__ __device__ constexpr bool tg_a_in_tmem(int enc) {
   return enc == E_Q4_0 || enc == E_Q4_1 || enc == E_Q8_0 || enc == E_MLX_U4 || enc == E_Q4_K || enc == E_Q5_K ||
-         enc == E_IQ4_XS;
+         enc == E_IQ4_XS || enc == E_BF16 || enc == E_F16;
 }
+__host__ __device__ constexpr bool tg_plain16(int enc) { return enc == E_BF16 || enc == E_F16; }
 __host__ __device__ constexpr bool tg_kquant(int enc) { return enc == E_Q4_K || enc == E_Q5_K || enc == E_IQ4_XS; }
 constexpr int TG_TMEM_A_COL = 256;        // first column of the A ring (32 columns per slot) behind the accumulator
 constexpr int TG_RAW_WORDS = 32 * 21;     // per-warp staging of raw row words (Q5_K: 20 words per row and chunk, odd stride)
@@ -365,6 +366,55 @@ dqgemm_tc_kernel(const TgArgs a, const __grid_constant__ CUtensorMap xmap) {
         tc_fence_before();
       };
       tg_produce_chunks<WPR, 1>(grp, nk, nslot, smem, stage_bytes, empty_bar, full_bar, &s_abort, lane, fetch, convert);
+    } else if constexpr (AT && tg_plain16(ENC)) {
+      // Plain 16-bit weights, thread = row as below, in two halves of 32 weights (64 bytes of a row). A half
+      // is fetched with 16-byte loads, four lanes per row and eight rows per load, turned to f16 on the way
+      // (bf16: through f32, the decoder's value rounded once) and passed to "thread = row" through the per-warp scratch:
+      // rows of four 16-byte pieces, piece p of row r at p ^ ((r >> 1) & 3), conflict-free both ways.
+      static_assert(32 * 16 <= TG_RAW_WORDS, "per-warp scratch");
+      const int quarter = warp & 3;
+      uint32_t* raw = reinterpret_cast<uint32_t*>(smem + (size_t)nslot * stage_bytes) + warp * TG_RAW_WORDS;
+      const int64_t last = N - 1 - (n0 + quarter * 32);  // rows past the matrix repeat its last row (never stored)
+      const int rsub = lane >> 2, piece = lane & 3;
+      auto fetch = [&](int kc, int sub, uint32_t (&q)[16]) {
+        const uint8_t* cb = a.w.data + ((int64_t)(kbase + kc) * TG_BK + sub * 32) * 2 + piece * 16;
+#pragma unroll
+        for (int it = 0; it < 4; it++) {
+          const int r = it * 8 + rsub;
+          const uint4 v = *reinterpret_cast<const uint4*>(cb + (n0 + quarter * 32 + (r < last ? r : last)) * K * 2);
+          q[4 * it] = v.x, q[4 * it + 1] = v.y, q[4 * it + 2] = v.z, q[4 * it + 3] = v.w;
+        }
+      };
+      auto convert = [&](int kc, int sub, uint32_t (&q)[16], uint8_t*) {
+        auto f16_pair = [](uint32_t u) {
+          if constexpr (ENC == E_F16) return u;
+          const __half2 h = __floats2half2_rn(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u));
+          return *reinterpret_cast<const uint32_t*>(&h);
+        };
+#pragma unroll
+        for (int it = 0; it < 4; it++) {
+          const int r = it * 8 + rsub;
+          *reinterpret_cast<uint4*>(raw + r * 16 + ((piece ^ ((r >> 1) & 3)) << 2)) =
+              make_uint4(f16_pair(q[4 * it]), f16_pair(q[4 * it + 1]), f16_pair(q[4 * it + 2]), f16_pair(q[4 * it + 3]));
+        }
+        __syncwarp();
+        uint32_t out[16];
+#pragma unroll
+        for (int p = 0; p < 4; p++) {
+          const uint4 v = *reinterpret_cast<const uint4*>(raw + lane * 16 + ((p ^ ((lane >> 1) & 3)) << 2));
+          out[4 * p] = v.x, out[4 * p + 1] = v.y, out[4 * p + 2] = v.z, out[4 * p + 3] = v.w;
+        }
+        const uint32_t taddr = tmem_d + ((uint32_t)(quarter * 32) << 16) + TG_TMEM_A_COL + (uint32_t)(kc & (nslot - 1)) * 32u;
+        asm volatile(
+            "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};"
+            ::"r"(taddr + 16u * sub), "r"(out[0]), "r"(out[1]), "r"(out[2]), "r"(out[3]), "r"(out[4]), "r"(out[5]), "r"(out[6]),
+              "r"(out[7]), "r"(out[8]), "r"(out[9]), "r"(out[10]), "r"(out[11]), "r"(out[12]), "r"(out[13]), "r"(out[14]), "r"(out[15])
+            : "memory");
+        __syncwarp();  // the scratch is read; the next half may overwrite it
+        asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+        tc_fence_before();
+      };
+      tg_produce_chunks<16, 2>(grp, nk, nslot, smem, stage_bytes, empty_bar, full_bar, &s_abort, lane, fetch, convert);
     } else if constexpr (AT) {
       // A operand in tensor memory. A warp converts the 32 rows of its lane quarter: thread = row, the
       // chunk's 64 weights of a row = 32 packed columns (column c = weights 2c, 2c + 1), written with one
@@ -736,6 +786,7 @@ bool tg_shape_ok(const WRef& w, int64_t M) {
   if ((w.enc == E_Q4_0 || w.enc == E_Q4_1 || w.enc == E_Q8_0 || w.enc == E_MLX_U4 || tg_kquant(w.enc)) && (addr & 3))
     return false;
   if (w.enc == E_Q6_K && (addr & 1)) return false;
+  if (tg_plain16(w.enc) && (addr & 15)) return false;
   return M >= 1 && w.rows >= 1 && w.cols >= TG_BK && w.cols % (enc_block_elems(w.enc) == 256 ? 256 : TG_BK) == 0;
 }
 

@@ -25,6 +25,7 @@ namespace {
 constexpr int RT_C = 64;      // tokens per chunk
 constexpr int RT_PITCH = RT_C + 4;
 constexpr int RT_SLICE = 32;  // reduction elements staged at a time
+constexpr int RT_PRE = 16;    // state rows a decode thread fetches ahead
 
 // The angle of a position, reduced in double precision: p * f is far from 0 for long contexts.
 __device__ __forceinline__ void sincos_position(int64_t pos, double freq, float* sv, float* cv) {
@@ -56,12 +57,19 @@ __global__ void __launch_bounds__(256) retention_step_kernel(RetentionArgs a, co
   float* ks = qs + D;            // [D]
   float* red = ks + D;           // [8][per]
   float* os = red + 8 * per;     // [per]
+  pdl_trigger();
   const int64_t pos = row_pos ? row_pos[r] : pos0, seq = row_seq ? row_seq[r] : seq0;
+  // the state was written one token ago, with ordinary launches in between, so its first 128 rows are fetched
+  // before the kernel waits for this token's products
+  float* S = a.state + ((seq * a.heads + h) * D) * (int64_t)E + e0;
+  float pre[RT_PRE];
+#pragma unroll
+  for (int j = 0; j < RT_PRE; j++) pre[j] = warp + 8 * j < D && lane < ne && pos > 0 ? S[(int64_t)(warp + 8 * j) * E + lane] : 0.f;
+  pdl_wait();
   const float decay = a.decay[h], kscale = 1.0f / sqrtf((float)D);
   const float* q = a.q.ptr + r * a.q.ld + (int64_t)h * D;
   const float* k = a.k.ptr + r * a.k.ld + (int64_t)h * D;
   const float* v = a.v.ptr + r * a.v.ld + (int64_t)h * E + e0;
-  pdl_trigger();
   const int half = a.rot_dims / 2;
   for (int i = tid; i < D; i += 256) {
     if (i < half) {
@@ -75,11 +83,23 @@ __global__ void __launch_bounds__(256) retention_step_kernel(RetentionArgs a, co
     }
   }
   __syncthreads();
-  float* S = a.state + ((seq * a.heads + h) * D) * (int64_t)E + e0;
   for (int c = lane; c < ne; c += 32) {
     const float vv = v[c];
     float acc = 0.f;
-    for (int d0 = warp; d0 < D; d0 += 64) {  // eight rows of the state in flight per thread
+    int first = warp;
+    if (c == lane) {
+#pragma unroll
+      for (int j = 0; j < RT_PRE; j++) {
+        const int d = warp + 8 * j;
+        if (d < D) {
+          const float n = fmaf(decay, pre[j], ks[d] * vv);
+          S[(int64_t)d * E + c] = n;
+          acc = fmaf(n, qs[d], acc);
+        }
+      }
+      first += 8 * RT_PRE;
+    }
+    for (int d0 = first; d0 < D; d0 += 64) {  // eight rows of the state in flight per thread
       float s[8];
 #pragma unroll
       for (int j = 0; j < 8; j++) s[j] = (d0 + 8 * j < D && pos > 0) ? S[(int64_t)(d0 + 8 * j) * E + c] : 0.f;
@@ -136,10 +156,13 @@ int step_rows(const RetentionArgs& a, const int64_t* pos, const int64_t* seq, in
     cfg.blockDim = dim3(256);
     cfg.dynamicSmemBytes = smem;
     cfg.stream = st;
-    cudaLaunchAttribute attr{};
-    attr.id = cudaLaunchAttributeClusterDimension;
-    attr.val.clusterDim.x = (unsigned)nsplit, attr.val.clusterDim.y = 1, attr.val.clusterDim.z = 1;
-    cfg.attrs = &attr, cfg.numAttrs = 1;
+    cudaLaunchAttribute attr[2] = {};
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = (unsigned)nsplit, attr[0].val.clusterDim.y = 1, attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    // a portion run token by token has no ordinary launch between its states: no early start there
+    cfg.attrs = attr, cfg.numAttrs = pos && pdl_enabled() ? 2 : 1;
     DYN_CUDA(cudaLaunchKernelEx(&cfg, retention_step_kernel, a, pos, seq, pos0, seq0, row0 + r0));
     count_launch();
   }

@@ -5,7 +5,7 @@
 // decode step writes its own row while other CTAs still read the rows before it. Positions before the
 // sequence start count as zeros and are never read.
 //
-// Decode rows: one launch per layer. A CTA takes 32 outputs of one gate block: it forms the block's
+// Decode rows: one launch per layer. A CTA takes 16 outputs of one gate block: it forms the block's
 // convolution outputs (a few multiplies, repeated by the block's CTAs), then a warp per output reads
 // the two gate rows and updates the state.
 // Portions: convolution -> gates (a tiled block-diagonal product whose epilogue leaves a_t and the
@@ -33,60 +33,75 @@ __device__ __forceinline__ void recurrence_terms(float rz, float iz, float u, fl
 }
 
 // ---- decode rows -----------------------------------------------------------------------------
-constexpr int RG_OUT = 32;
+constexpr int RG_OUT = 16, RG_PER_WARP = RG_OUT / 8;
 
-// dot(w[row][0..n), u) over the warp; consecutive lanes read consecutive 8-element pieces when they can
-template <bool WIDE>
-__device__ __forceinline__ void two_dots(const RglruArgs& a, int64_t row, int n, const float* u, int lane, float* r, float* i) {
-  float sr = 0.f, si = 0.f;
-  if (WIDE) {  // bf16 rows of a multiple of 8, 16-byte aligned
-    const uint4* wr = reinterpret_cast<const uint4*>(a.ra.ptr + row * n * 2);
-    const uint4* wi = reinterpret_cast<const uint4*>(a.ri.ptr + row * n * 2);
-    for (int p = lane; p < n / 8; p += 32) {
-      const uint4 x = wr[p], y = wi[p];
-      const uint32_t xw[4] = {x.x, x.y, x.z, x.w}, yw[4] = {y.x, y.y, y.z, y.w};
+__device__ __forceinline__ float dot8(const uint4& w, const float* u) {
+  const uint32_t x[4] = {w.x, w.y, w.z, w.w};
+  float s = 0.f;
 #pragma unroll
-      for (int e = 0; e < 4; e++) {
-        const float u0 = u[8 * p + 2 * e], u1 = u[8 * p + 2 * e + 1];
-        sr = fmaf(__uint_as_float(xw[e] << 16), u0, sr), sr = fmaf(__uint_as_float(xw[e] & 0xffff0000u), u1, sr);
-        si = fmaf(__uint_as_float(yw[e] << 16), u0, si), si = fmaf(__uint_as_float(yw[e] & 0xffff0000u), u1, si);
-      }
-    }
-  } else {
-    for (int k = lane; k < n; k += 32) {
-      sr = fmaf(vec_at(a.ra, row * n + k), u[k], sr);
-      si = fmaf(vec_at(a.ri, row * n + k), u[k], si);
-    }
-  }
-  *r = warp_sum(sr), *i = warp_sum(si);
+  for (int e = 0; e < 4; e++)
+    s = fmaf(__uint_as_float(x[e] << 16), u[2 * e], s), s = fmaf(__uint_as_float(x[e] & 0xffff0000u), u[2 * e + 1], s);
+  return s;
 }
 
+// WIDE: bf16 gate rows of whole 16-byte pieces; a warp's first piece per lane of its four gate rows is fetched
+// before the kernel waits for the products.
 template <bool WIDE>
 __global__ void __launch_bounds__(256) rglru_step_kernel(RglruArgs a, const int64_t* row_pos, const int64_t* row_seq,
                                                          int64_t pos0, int64_t seq0, int64_t row0) {
-  extern __shared__ float u_s[];  // [width / blocks]
+  extern __shared__ __align__(16) float u_s[];  // [width / blocks]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int n = a.width / a.blocks, slices = (n + RG_OUT - 1) / RG_OUT;
   const int blk = blockIdx.x / slices, slice = blockIdx.x % slices;
   const int64_t r = row0 + blockIdx.y;
+  const int pieces = n / 8;
+  pdl_trigger();
+  uint4 wr[RG_PER_WARP], wi[RG_PER_WARP];
+  if (WIDE) {
+#pragma unroll
+    for (int i = 0; i < RG_PER_WARP; i++) {
+      const int o = slice * RG_OUT + warp + 8 * i;
+      const int64_t at = (int64_t)blk * n + o;
+      if (o < n && lane < pieces) {
+        wr[i] = reinterpret_cast<const uint4*>(a.ra.ptr + at * n * 2)[lane];
+        wi[i] = reinterpret_cast<const uint4*>(a.ri.ptr + at * n * 2)[lane];
+      }
+    }
+  }
+  pdl_wait();
   const int64_t pos = row_pos ? row_pos[r] : pos0, seq = row_seq ? row_seq[r] : seq0;
   float* ring = a.ring + seq * (int64_t)a.taps * a.width;
   const float* x = a.x.ptr + r * a.x.ld;
-  pdl_trigger();
   for (int c = tid; c < n; c += 256) {
     const int64_t ch = (int64_t)blk * n + c;
     const float xin = x[ch] + vec_at(a.bx, ch);
     float u = vec_at(a.conv, ch * a.taps + a.taps - 1) * xin;
+#pragma unroll 4
     for (int j = 1; j < a.taps; j++)
       if (pos >= j) u = fmaf(vec_at(a.conv, ch * a.taps + a.taps - 1 - j), ring[((pos - j) % a.taps) * a.width + ch], u);
     u_s[c] = u + vec_at(a.bc, ch);
     if (slice == 0) ring[(pos % a.taps) * a.width + ch] = xin;
   }
   __syncthreads();
-  for (int o = slice * RG_OUT + warp; o < min(n, (slice + 1) * RG_OUT); o += 8) {
+#pragma unroll
+  for (int i = 0; i < RG_PER_WARP; i++) {
+    const int o = slice * RG_OUT + warp + 8 * i;
+    if (o >= n) break;
     const int64_t ch = (int64_t)blk * n + o;
-    float rz, iz;
-    two_dots<WIDE>(a, ch, n, u_s, lane, &rz, &iz);
+    float rz = 0.f, iz = 0.f;
+    if (WIDE) {
+      if (lane < pieces) rz = dot8(wr[i], u_s + 8 * lane), iz = dot8(wi[i], u_s + 8 * lane);
+      for (int p = lane + 32; p < pieces; p += 32) {
+        rz += dot8(reinterpret_cast<const uint4*>(a.ra.ptr + ch * n * 2)[p], u_s + 8 * p);
+        iz += dot8(reinterpret_cast<const uint4*>(a.ri.ptr + ch * n * 2)[p], u_s + 8 * p);
+      }
+    } else {
+      for (int k = lane; k < n; k += 32) {
+        rz = fmaf(vec_at(a.ra, ch * n + k), u_s[k], rz);
+        iz = fmaf(vec_at(a.ri, ch * n + k), u_s[k], iz);
+      }
+    }
+    rz = warp_sum(rz), iz = warp_sum(iz);
     if (lane == 0) {
       float av, bv;
       recurrence_terms(rz + vec_at(a.bra, ch), iz + vec_at(a.bri, ch), u_s[o], a.c, vec_at(a.lam, ch), &av, &bv);
@@ -112,9 +127,9 @@ int step_rows(const RglruArgs& a, const int64_t* pos, const int64_t* seq, int64_
   for (int64_t r0 = 0; r0 < rows; r0 += 65535) {
     const dim3 grid((unsigned)(a.blocks * slices), (unsigned)std::min<int64_t>(65535, rows - r0));
     if (wide_rows(a))
-      rglru_step_kernel<true><<<grid, 256, smem, st>>>(a, pos, seq, pos0, seq0, row0 + r0);
+      DYN_CUDA(launch_pdl(rglru_step_kernel<true>, grid, dim3(256), smem, st, a, pos, seq, pos0, seq0, row0 + r0));
     else
-      rglru_step_kernel<false><<<grid, 256, smem, st>>>(a, pos, seq, pos0, seq0, row0 + r0);
+      DYN_CUDA(launch_pdl(rglru_step_kernel<false>, grid, dim3(256), smem, st, a, pos, seq, pos0, seq0, row0 + r0));
     count_launch();
   }
   DYN_CUDA(cudaGetLastError());

@@ -359,8 +359,25 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
     for (const WRef& w : L.in) fuse = fuse && takes(w);
     for (const WRef* w : {&L.o, &L.gate, &L.up, &L.down}) fuse = fuse && takes(*w);
   }
+  // A few rows of 16-bit weights: the streaming GEMV forms its normalised / gated input itself.
+  bool stream = rows <= 4;
+  for (const MixerLayer& L : s->mix) {
+    for (const WRef& w : L.in) stream = stream && gemv_plain_takes(w, rows);
+    if (L.c.ff) stream = stream && L.gate_up.data && gemv_plain_takes(L.gate_up, rows) && gemv_plain_takes(L.down, rows);
+  }
+  GemvInput formed;
+  auto streamed = [&](const WRef& w, const float* x, float* y, const float* residual) -> int {
+    bool handled = false;
+    if (launch_gemv_plain(w, x, E_F32, (int)rows, y, residual, st, &handled, formed)) return 1;
+    DYN_CHECK(handled, "streaming GEMV refused a product it had accepted");
+    return 0;
+  };
   int pending = 0;  // K-split sums in gpart that `hidden` still lacks
   auto norm = [&](const NormW& w) -> int {
+    if (stream) {
+      formed.mode = GEMV_NORM, formed.norm_w = w.ptr, formed.norm_type = w.type, formed.eps = c.eps;
+      return 0;
+    }
     if (!fuse) return launch_rms_norm(s->hidden, w.ptr, w.type, rows, H, c.eps, s->xn, st);
     const int splits = pending;
     pending = 0;
@@ -381,6 +398,7 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
   };
   // a product of the normalised rows
   auto from_norm = [&](const WRef& w, float* y) -> int {
+    if (stream) return streamed(w, s->hidden, y, nullptr);
     return fuse ? gemm(w, nullptr, y, nullptr, false) : session_linear(s, w, s->xn, E_F32, rows, y, nullptr);
   };
   // hidden += W x; `last`: no norm of this function follows to add deferred sums
@@ -407,6 +425,12 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
     if (!L.c.ff) continue;
     if (norm(L.norm2)) return 1;
     bool prepared = false;
+    if (stream) {
+      if (from_norm(L.gate_up, s->gu1)) return 1;
+      formed.mode = GEMV_SWIGLU;
+      if (streamed(L.down, s->gu1, s->hidden, s->hidden)) return 1;
+      continue;
+    }
     if (L.gate_up.data) {
       if (from_norm(L.gate_up, s->gu1)) return 1;
       prepared = fuse;

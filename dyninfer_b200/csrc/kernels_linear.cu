@@ -6,6 +6,8 @@
 // weight is the exact f32 value the reference dequantises to, and the partial
 // sums are combined with warp shuffles. Up to MT activation rows share one
 // pass over the weights.
+#include <algorithm>
+
 #include "codec.cuh"
 #include "mixers.cuh"
 
@@ -150,7 +152,20 @@ int launch_linear(const WRef& w, const void* x, int x_type, int64_t m, float* y,
   // passes: the GEMM's dequantisation cost does not shrink with the row count)
   const bool cheap_producer = w.enc == E_Q4_0 || w.enc == E_Q4_1 || w.enc == E_Q8_0 || w.enc == E_Q6_K ||
                               w.enc == E_Q4_K || w.enc == E_Q5_K || w.enc == E_IQ4_XS || w.enc == E_MLX_U4;
-  if (m > 16 || (cheap_producer && m > (x_type == E_BF16 ? 8 : 4))) {
+  if (m > 4 && m <= 8 && gemv_plain_takes(w, 4)) {
+    // plain 16-bit weights: two streaming passes of up to four rows cost less than the GEMM's fixed part
+    const size_t xe = x_type == E_BF16 ? 2 : 4;
+    for (int64_t m0 = 0; m0 < m; m0 += 4) {
+      bool handled = false;
+      if (launch_gemv_plain(w, reinterpret_cast<const uint8_t*>(x) + (size_t)m0 * w.cols * xe, x_type,
+                            (int)std::min<int64_t>(4, m - m0), y + m0 * w.rows,
+                            residual ? residual + m0 * w.rows : nullptr, s, &handled))
+        return 1;
+      DYN_CHECK(handled, "streaming GEMV refused a product it had accepted");
+    }
+    return 0;
+  }
+  if (m > 16 || ((w.enc == E_BF16 || w.enc == E_F16) && m > 8) || (cheap_producer && m > (x_type == E_BF16 ? 8 : 4))) {
     bool handled = false;
     if (launch_dqgemm_tc(w, x, x_type, m, y, residual, s, &handled)) return 1;
     if (handled) return 0;

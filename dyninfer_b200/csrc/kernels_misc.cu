@@ -218,7 +218,9 @@ int launch_norm_prepare(const float* x, const float* partial, int splits, const 
   return 0;
 }
 
-__global__ void __launch_bounds__(256)
+// PER > 0: the row fits PER elements per thread, computed once and kept in registers.
+template <int PER>
+__global__ void __launch_bounds__(512)
 silu_prepare_kernel(const float* __restrict__ gu, int64_t I, __half* __restrict__ xh, float* __restrict__ inv_s) {
   __shared__ float red[32];
   const int64_t row = blockIdx.x;
@@ -227,17 +229,39 @@ silu_prepare_kernel(const float* __restrict__ gu, int64_t I, __half* __restrict_
     const float gv = g[i];
     return (gv / (1.0f + expf(-gv))) * g[I + i];
   };
-  float mx = 0.f;
-  for (int64_t i = threadIdx.x; i < I; i += blockDim.x) mx = fmaxf(mx, fabsf(val(i)));
-  float sc, is;
-  f16_row_scale(mx, red, &sc, &is);
+  float mx = 0.f, sc, is;
+  if constexpr (PER > 0) {
+    float v[PER];
+#pragma unroll
+    for (int k = 0; k < PER; k++) {
+      const int64_t i = threadIdx.x + (int64_t)k * blockDim.x;
+      v[k] = i < I ? val(i) : 0.f;
+      mx = fmaxf(mx, fabsf(v[k]));
+    }
+    f16_row_scale(mx, red, &sc, &is);
+#pragma unroll
+    for (int k = 0; k < PER; k++) {
+      const int64_t i = threadIdx.x + (int64_t)k * blockDim.x;
+      if (i < I) xh[row * I + i] = __float2half_rn(v[k] * sc);
+    }
+  } else {
+    for (int64_t i = threadIdx.x; i < I; i += blockDim.x) mx = fmaxf(mx, fabsf(val(i)));
+    f16_row_scale(mx, red, &sc, &is);
+    for (int64_t i = threadIdx.x; i < I; i += blockDim.x) xh[row * I + i] = __float2half_rn(val(i) * sc);
+  }
   if (threadIdx.x == 0) inv_s[row] = is;
-  for (int64_t i = threadIdx.x; i < I; i += blockDim.x) xh[row * I + i] = __float2half_rn(val(i) * sc);
 }
 
 int launch_silu_prepare(const float* gate_up, int64_t rows, int64_t inter, __half* xh, float* inv_s, cudaStream_t s) {
   if (rows == 0 || inter == 0) return 0;
-  silu_prepare_kernel<<<(unsigned)rows, 256, 0, s>>>(gate_up, inter, xh, inv_s);
+  if (inter <= 8 * 512)
+    silu_prepare_kernel<8><<<(unsigned)rows, 512, 0, s>>>(gate_up, inter, xh, inv_s);
+  else if (inter <= 16 * 512)
+    silu_prepare_kernel<16><<<(unsigned)rows, 512, 0, s>>>(gate_up, inter, xh, inv_s);
+  else if (inter <= 24 * 512)
+    silu_prepare_kernel<24><<<(unsigned)rows, 512, 0, s>>>(gate_up, inter, xh, inv_s);
+  else
+    silu_prepare_kernel<0><<<(unsigned)rows, 512, 0, s>>>(gate_up, inter, xh, inv_s);
   count_launch();
   DYN_CUDA(cudaGetLastError());
   return 0;

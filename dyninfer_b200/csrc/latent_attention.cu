@@ -508,10 +508,13 @@ int run_absorbed(const LatentArgs& a, const StepRows& s, cudaStream_t st) {
 
 // ---- expanded keys and values ---------------------------------------------------------------------
 constexpr int EX_D = 128;  // head width of the prefill attention
+constexpr int EX_SPLITS = 4;  // K-split sums of the up-projection kept for the expansion to add
 
-// y rows [k heads | v heads] of tokens t0.. -> K, V planes [head][cap][128] bf16, zero padded
+// y rows [k heads | v heads] of tokens t0.. -> K, V planes [head][cap][128] bf16, zero padded. With splits > 1
+// the rows still lie as that many K-split sums `zstride` floats apart.
 __global__ void __launch_bounds__(256)
-latent_expand_kernel(const float* __restrict__ k, int64_t ldk, const float* __restrict__ v, int64_t ldv, int heads, int dim, int vdim,
+latent_expand_kernel(const float* __restrict__ k, int64_t ldk, const float* __restrict__ v, int64_t ldv, int splits, int64_t zstride,
+                     int heads, int dim, int vdim,
                      int64_t t0, int64_t tokens, int64_t cap, __nv_bfloat162* __restrict__ kx, __nv_bfloat162* __restrict__ vx) {
   const int64_t total = tokens * heads * (EX_D / 2);
   for (int64_t it = blockIdx.x * 256ll + threadIdx.x; it < total; it += (int64_t)gridDim.x * 256) {
@@ -520,8 +523,15 @@ latent_expand_kernel(const float* __restrict__ k, int64_t ldk, const float* __re
     const float* kr = k + t * ldk + h * dim;
     const float* vr = v + t * ldv + h * vdim;
     const int64_t at = ((h * cap + t0 + t) * EX_D + c) / 2;
-    kx[at] = __floats2bfloat162_rn(c < dim ? kr[c] : 0.f, c + 1 < dim ? kr[c + 1] : 0.f);
-    vx[at] = __floats2bfloat162_rn(c < vdim ? vr[c] : 0.f, c + 1 < vdim ? vr[c + 1] : 0.f);
+    float k0 = 0.f, k1 = 0.f, v0 = 0.f, v1 = 0.f;
+    for (int z = 0; z < splits; z++, kr += zstride, vr += zstride) {
+      if (c < dim) k0 += kr[c];
+      if (c + 1 < dim) k1 += kr[c + 1];
+      if (c < vdim) v0 += vr[c];
+      if (c + 1 < vdim) v1 += vr[c + 1];
+    }
+    kx[at] = __floats2bfloat162_rn(k0, k1);
+    vx[at] = __floats2bfloat162_rn(v0, v1);
   }
 }
 
@@ -572,15 +582,23 @@ int run_expanded(const LatentArgs& a, const StepRows& s, cudaStream_t st) {
   const int64_t kd = H * a.dim, vd = H * a.vdim;
   __nv_bfloat16* kx = reinterpret_cast<__nv_bfloat16*>(a.scratch);
   __nv_bfloat16* vx = kx + H * a.cap * EX_D;
-  float* y = reinterpret_cast<float*>(vx + H * a.cap * EX_D);  // [max_rows, kd + vd]
-  float* qp = y + a.max_rows * (kd + vd);                      // [rows, H * 128]
+  float* y = reinterpret_cast<float*>(vx + H * a.cap * EX_D);  // [EX_SPLITS][max_rows, kd + vd]
+  float* qp = y + EX_SPLITS * a.max_rows * (kd + vd);          // [rows, H * 128]
   float* ctx = qp + a.max_rows * H * EX_D;
   const __nv_bfloat16* lat = reinterpret_cast<const __nv_bfloat16*>(a.cache) + s.slot * a.cap * a.rank;
   for (int64_t t0 = 0; t0 < end; t0 += a.max_rows) {
     const int64_t n = std::min(a.max_rows, end - t0);
     const float *k = y, *v = y + kd;
     int64_t ldk = kd + vd, ldv = kd + vd;
-    if (a.ukv.data) {
+    int splits = 1;
+    if (a.ukv.data && n > 16 && dqgemm_tc_takes(a.ukv, n)) {
+      TgIo io;
+      io.partial = y, io.partial_bytes = (size_t)EX_SPLITS * a.max_rows * (kd + vd) * 4;
+      bool handled = false;
+      if (launch_dqgemm_tc(a.ukv, lat + t0 * a.rank, E_BF16, n, y, nullptr, st, &handled, &io)) return 1;
+      DYN_CHECK(handled, "dequant GEMM refused a product it had accepted");
+      splits = std::max(1, io.splits);
+    } else if (a.ukv.data) {
       if (launch_linear(a.ukv, lat + t0 * a.rank, E_BF16, n, y, nullptr, st)) return 1;
     } else {
       v = y + n * kd, ldk = kd, ldv = vd;
@@ -588,7 +606,7 @@ int run_expanded(const LatentArgs& a, const StepRows& s, cudaStream_t st) {
           launch_linear(a.uv, lat + t0 * a.rank, E_BF16, n, y + n * kd, nullptr, st))
         return 1;
     }
-    latent_expand_kernel<<<ew_grid(n * H * (EX_D / 2)), 256, 0, st>>>(k, ldk, v, ldv, a.heads, a.dim, a.vdim, t0, n, a.cap,
+    latent_expand_kernel<<<ew_grid(n * H * (EX_D / 2)), 256, 0, st>>>(k, ldk, v, ldv, splits, n * (kd + vd), a.heads, a.dim, a.vdim, t0, n, a.cap,
                                                                       reinterpret_cast<__nv_bfloat162*>(kx),
                                                                       reinterpret_cast<__nv_bfloat162*>(vx));
     count_launch();
@@ -620,7 +638,7 @@ size_t latent_scratch_floats(const LatentArgs& a, int64_t rows) {
     need = std::max(need, (size_t)r * a.heads * (a.rank + (size_t)slices(a, r) * (a.rank + 4)) + 4);
   if (expands(a) && rows >= EXPAND_MIN_ROWS)
     need = std::max(need, (size_t)a.heads * a.cap * EX_D +
-                              (size_t)a.max_rows * a.heads * (a.dim + a.vdim + 2 * EX_D) + 64);
+                              (size_t)a.max_rows * a.heads * (EX_SPLITS * (a.dim + a.vdim) + 2 * EX_D) + 64);
   return need;
 }
 

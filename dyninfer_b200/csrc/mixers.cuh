@@ -41,6 +41,7 @@ struct RetentionArgs {
   float* out = nullptr;           // [rows, heads * vdim]
   float* scratch = nullptr;       // retention_scratch_floats
   float eps = 0.f;
+  bool exact = false;             // f32 products only
 };
 size_t retention_scratch_floats(const RetentionArgs& a, int64_t rows);
 int launch_retention(const RetentionArgs& a, const StepRows& r, cudaStream_t st);

@@ -9,9 +9,9 @@
 // convolution outputs (a few multiplies, repeated by the block's CTAs), then a warp per output reads
 // the two gate rows and updates the state.
 // Portions: convolution -> gates (a tiled block-diagonal product whose epilogue leaves a_t and the
-// increment b_t) -> scan. The scan handles 512 tokens x 32 channels per CTA and pass: a warp composes
-// the maps S -> A S + B of its 16 tokens, the 32 segment maps are chained through shared memory, and
-// each warp replays its tokens from its start state.
+// increment b_t) -> scan. The scan handles 512 tokens x 16 channels per CTA and pass: a thread composes
+// the maps S -> A S + B of its 8 tokens, the 64 segment maps are chained through shared memory, and
+// each thread replays its tokens from its start state.
 #include <algorithm>
 
 #include "mixers.cuh"
@@ -137,22 +137,122 @@ int step_rows(const RglruArgs& a, const int64_t* pos, const int64_t* seq, int64_
 }
 
 // ---- portions ---------------------------------------------------------------------------------
-// u[t][ch]; inputs from before the portion come from the ring.
-__global__ void __launch_bounds__(256) rglru_conv_kernel(RglruArgs a, int64_t rows, int64_t base, int64_t slot, float* __restrict__ u) {
-  const int ch = blockIdx.x * 256 + threadIdx.x;
+// u[t][ch]; inputs from before the portion come from the ring. A thread takes one channel and CV_T tokens; with
+// TAPS > 0 the window of inputs stays in registers.
+constexpr int CV_T = 16;
+template <int TAPS>
+__global__ void __launch_bounds__(128) rglru_conv_kernel(RglruArgs a, int64_t rows, int64_t base, int64_t slot, float* __restrict__ u) {
+  const int ch = blockIdx.x * 128 + threadIdx.x;
   if (ch >= a.width) return;
   const float* ring = a.ring + slot * (int64_t)a.taps * a.width;
   const float bx = vec_at(a.bx, ch), bc = vec_at(a.bc, ch);
-  const int64_t t = blockIdx.y;
-  float acc = 0.f;
-  for (int j = 0; j < a.taps; j++) {
-    const float w = vec_at(a.conv, (int64_t)ch * a.taps + a.taps - 1 - j);
-    if (j <= t)
-      acc = fmaf(w, a.x.ptr[(t - j) * a.x.ld + ch] + bx, acc);
-    else if (base + t >= j)
-      acc = fmaf(w, ring[((base + t - j) % a.taps) * a.width + ch], acc);
+  const int64_t t0 = (int64_t)blockIdx.y * CV_T;
+  auto input = [&](int64_t t) {  // of token base + t, t possibly before the portion
+    if (t >= 0) return t < rows ? a.x.ptr[t * a.x.ld + ch] + bx : 0.f;
+    return base + t >= 0 ? ring[((base + t) % a.taps) * a.width + ch] : 0.f;
+  };
+  if constexpr (TAPS > 0) {
+    float w[TAPS], in[CV_T + TAPS - 1];
+#pragma unroll
+    for (int j = 0; j < TAPS; j++) w[j] = vec_at(a.conv, (int64_t)ch * TAPS + j);
+#pragma unroll
+    for (int j = 0; j < CV_T + TAPS - 1; j++) in[j] = input(t0 + j - (TAPS - 1));
+#pragma unroll
+    for (int i = 0; i < CV_T; i++) {
+      float acc = 0.f;
+#pragma unroll
+      for (int j = TAPS - 1; j >= 0; j--) acc = fmaf(w[j], in[i + j], acc);
+      if (t0 + i < rows) u[(t0 + i) * a.width + ch] = acc + bc;
+    }
+  } else {
+    for (int i = 0; i < CV_T && t0 + i < rows; i++) {
+      float acc = 0.f;
+      for (int j = 0; j < a.taps; j++)
+        acc = fmaf(vec_at(a.conv, (int64_t)ch * a.taps + a.taps - 1 - j), input(t0 + i - j), acc);
+      u[(t0 + i) * a.width + ch] = acc + bc;
+    }
   }
-  u[t * a.width + ch] = acc + bc;
+}
+
+// Gates on the tensor cores for bf16 weights: 64 tokens x 64 outputs of one block per CTA, both products. The f32
+// inputs enter as three bf16 terms (hi + mid + lo hold all 24 bits), the weights as stored, so every product
+// is exact and the sums are f32: these are gates of a recurrence, not 16-bit activations. Warp w takes 16 tokens
+// (w mod 4) of one of the two matrices (w / 4).
+constexpr int GT_T = 64, GT_K = 64, GT_P = GT_K + 8;
+constexpr int GT_SMEM = (3 * GT_T + 2 * GT_T) * GT_P * 2;
+__global__ void __launch_bounds__(256)
+rglru_gates_tc_kernel(RglruArgs a, int64_t rows, const float* __restrict__ u, float* __restrict__ av, float* __restrict__ bv) {
+  extern __shared__ __align__(16) uint8_t gt_smem[];
+  __nv_bfloat16(*us)[GT_T][GT_P] = reinterpret_cast<__nv_bfloat16(*)[GT_T][GT_P]>(gt_smem);              // [term][token][k]
+  __nv_bfloat16(*ws)[GT_T][GT_P] = reinterpret_cast<__nv_bfloat16(*)[GT_T][GT_P]>(gt_smem + 3 * GT_T * GT_P * 2);  // [matrix][output][k]
+  float(*zs)[GT_T + 4] = reinterpret_cast<float(*)[GT_T + 4]>(gt_smem);                                  // [matrix * 64 + token][output], afterwards
+  static_assert(2 * GT_T * (GT_T + 4) * 4 <= GT_SMEM, "gate sums fit the operand tiles");
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const int n = a.width / a.blocks, tiles = (n + GT_T - 1) / GT_T;
+  const int blk = blockIdx.x / tiles, o0 = (blockIdx.x % tiles) * GT_T;
+  const int64_t t0 = (int64_t)blockIdx.y * GT_T;
+  const int mt = warp & 3, mat = warp >> 2;
+  float acc[8][4] = {};
+  for (int k0 = 0; k0 < n; k0 += GT_K) {
+#pragma unroll
+    for (int j = 0; j < GT_T * GT_K / 4 / 256; j++) {
+      const int i = tid + 256 * j, tok = i / (GT_K / 4), k = (i % (GT_K / 4)) * 4;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);  // n is a multiple of 8: whole quads
+      if (t0 + tok < rows && k0 + k < n) v = *reinterpret_cast<const float4*>(u + (t0 + tok) * a.width + blk * n + k0 + k);
+      const float x[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const __nv_bfloat16 h = __float2bfloat16_rn(x[e]);
+        const float r1 = x[e] - __bfloat162float(h);
+        const __nv_bfloat16 m = __float2bfloat16_rn(r1);
+        us[0][tok][k + e] = h, us[1][tok][k + e] = m, us[2][tok][k + e] = __float2bfloat16_rn(r1 - __bfloat162float(m));
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 2 * GT_T * GT_K / 8 / 256; j++) {
+      const int i = tid + 256 * j, m = i / (GT_T * GT_K / 8), o = (i / (GT_K / 8)) % GT_T, k = (i % (GT_K / 8)) * 8;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (o0 + o < n && k0 + k < n)
+        v = *reinterpret_cast<const uint4*>((m ? a.ri.ptr : a.ra.ptr) + (((int64_t)blk * n + o0 + o) * n + k0 + k) * 2);
+      *reinterpret_cast<uint4*>(&ws[m][o][k]) = v;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < GT_K / 16; kk++) {
+      uint32_t af[3][4];
+#pragma unroll
+      for (int s = 0; s < 3; s++) {
+        const __nv_bfloat16 *p0 = &us[s][16 * mt + g][16 * kk + 2 * t], *p1 = &us[s][16 * mt + g + 8][16 * kk + 2 * t];
+        af[s][0] = *reinterpret_cast<const uint32_t*>(p0), af[s][1] = *reinterpret_cast<const uint32_t*>(p1);
+        af[s][2] = *reinterpret_cast<const uint32_t*>(p0 + 8), af[s][3] = *reinterpret_cast<const uint32_t*>(p1 + 8);
+      }
+#pragma unroll
+      for (int nt = 0; nt < 8; nt++) {
+        const __nv_bfloat16* p = &ws[mat][8 * nt + g][16 * kk + 2 * t];
+        const uint32_t b0 = *reinterpret_cast<const uint32_t*>(p), b1 = *reinterpret_cast<const uint32_t*>(p + 8);
+#pragma unroll
+        for (int s = 2; s >= 0; s--)  // small terms first
+          asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+              : "+f"(acc[nt][0]), "+f"(acc[nt][1]), "+f"(acc[nt][2]), "+f"(acc[nt][3])
+              : "r"(af[s][0]), "r"(af[s][1]), "r"(af[s][2]), "r"(af[s][3]), "r"(b0), "r"(b1));
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int nt = 0; nt < 8; nt++)
+#pragma unroll
+    for (int e = 0; e < 4; e++) zs[mat * GT_T + 16 * mt + g + 8 * (e >> 1)][8 * nt + 2 * t + (e & 1)] = acc[nt][e];
+  __syncthreads();
+  const int o = tid % GT_T;
+  if (o0 + o >= n) return;
+  const int64_t ch = (int64_t)blk * n + o0 + o;
+  const float br = vec_at(a.bra, ch), bi = vec_at(a.bri, ch), lam = vec_at(a.lam, ch);
+#pragma unroll 4
+  for (int tok = tid / GT_T; tok < GT_T && t0 + tok < rows; tok += 256 / GT_T) {
+    const int64_t at = (t0 + tok) * a.width + ch;
+    recurrence_terms(zs[tok][o] + br, zs[GT_T + tok][o] + bi, u[at], a.c, lam, &av[at], &bv[at]);
+  }
 }
 
 // Gates of 128 tokens x 64 outputs of one block, f32: both products share the u tile.
@@ -208,12 +308,12 @@ rglru_gates_kernel(RglruArgs a, int64_t rows, const float* __restrict__ u, float
   }
 }
 
-constexpr int SC_SEG = 32, SC_LEN = 16, SC_PASS = SC_SEG * SC_LEN;
+constexpr int SC_CH = 16, SC_SEG = 64, SC_LEN = 8, SC_PASS = SC_SEG * SC_LEN;
 __global__ void __launch_bounds__(1024)
 rglru_scan_kernel(RglruArgs a, int64_t rows, int64_t base, int64_t slot, const float* __restrict__ av, const float* __restrict__ bv) {
-  __shared__ float sA[SC_SEG][32], sB[SC_SEG][32];
-  const int lane = threadIdx.x & 31, seg = threadIdx.x >> 5;
-  const int ch = blockIdx.x * 32 + lane;
+  __shared__ float sA[SC_SEG][SC_CH], sB[SC_SEG][SC_CH];
+  const int lane = threadIdx.x % SC_CH, seg = threadIdx.x / SC_CH;
+  const int ch = blockIdx.x * SC_CH + lane;
   const bool live = ch < a.width;
   float S0 = live && base > 0 ? a.state[slot * a.width + ch] : 0.f;  // state before the pass
   const float by = live ? vec_at(a.by, ch) : 0.f;
@@ -232,6 +332,7 @@ rglru_scan_kernel(RglruArgs a, int64_t rows, int64_t base, int64_t slot, const f
     sA[seg][lane] = A, sB[seg][lane] = B;
     __syncthreads();
     float S = S0;
+#pragma unroll 8
     for (int w = 0; w < SC_SEG; w++) {
       const float n = fmaf(sA[w][lane], S0, sB[w][lane]);
       if (w < seg) S = n;
@@ -269,11 +370,20 @@ int launch_rglru(const RglruArgs& a, const StepRows& r, cudaStream_t st) {
   DYN_CHECK(r.rows <= 65535, "rglru: portion of %lld tokens", (long long)r.rows);
   float* u = a.scratch;
   float *av = u + r.rows * a.width, *bv = av + r.rows * a.width;
-  rglru_conv_kernel<<<dim3((unsigned)((a.width + 255) / 256), (unsigned)r.rows), 256, 0, st>>>(a, r.rows, r.base, r.slot, u);
+  const dim3 cgrid((unsigned)((a.width + 127) / 128), (unsigned)((r.rows + CV_T - 1) / CV_T));
+  if (a.taps == 4)
+    rglru_conv_kernel<4><<<cgrid, 128, 0, st>>>(a, r.rows, r.base, r.slot, u);
+  else
+    rglru_conv_kernel<0><<<cgrid, 128, 0, st>>>(a, r.rows, r.base, r.slot, u);
   const int n = a.width / a.blocks;
-  rglru_gates_kernel<<<dim3((unsigned)(a.blocks * ((n + GG_N - 1) / GG_N)), (unsigned)((r.rows + GG_M - 1) / GG_M)), 256, 0, st>>>(
+  if (!a.exact && wide_rows(a)) {
+    if (ensure_dynamic_smem(reinterpret_cast<const void*>(rglru_gates_tc_kernel), GT_SMEM)) return 1;
+    rglru_gates_tc_kernel<<<dim3((unsigned)(a.blocks * ((n + GT_T - 1) / GT_T)), (unsigned)((r.rows + GT_T - 1) / GT_T)), 256, GT_SMEM, st>>>(
+        a, r.rows, u, av, bv);
+  } else
+    rglru_gates_kernel<<<dim3((unsigned)(a.blocks * ((n + GG_N - 1) / GG_N)), (unsigned)((r.rows + GG_M - 1) / GG_M)), 256, 0, st>>>(
       a, r.rows, u, av, bv);
-  rglru_scan_kernel<<<(unsigned)((a.width + 31) / 32), 1024, 0, st>>>(a, r.rows, r.base, r.slot, av, bv);
+  rglru_scan_kernel<<<(unsigned)((a.width + SC_CH - 1) / SC_CH), SC_CH * SC_SEG, 0, st>>>(a, r.rows, r.base, r.slot, av, bv);
   count_launch(3);
   DYN_CUDA(cudaGetLastError());
   return 0;

@@ -229,7 +229,7 @@ static RetentionArgs retention_args(Session* s, const MixerLayer& L, int64_t row
   a.v = part_rows(L, s->qkv1, rows, 2), a.g = part_rows(L, s->qkv1, rows, 3);
   a.heads = L.c.heads, a.dim = L.c.dim, a.vdim = L.c.vdim, a.rot_dims = L.c.rot_dims;
   a.freq = L.freq, a.decay = L.decay;
-  a.state = s->state + L.state_off, a.out = s->ctx, a.scratch = s->mix_scratch, a.eps = s->cfg.eps;
+  a.state = s->state + L.state_off, a.out = s->ctx, a.scratch = s->mix_scratch, a.eps = s->cfg.eps, a.exact = s->cfg.exact;
   return a;
 }
 

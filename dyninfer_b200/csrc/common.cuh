@@ -269,18 +269,17 @@ int launch_gemv_cs_q6k(const WRef& w, const void* x, int x_type, float* y, const
 size_t gemv_cs_workspace_bytes(const WRef& w, int M);
 int launch_gemv_cs(const WRef& w, const void* x, int x_type, int M, float* y, const float* residual,
                    uint8_t* ws, cudaStream_t s, bool* handled);
-// How the streaming GEMV of plain weights forms its activation rows from x: as they are, RMSNorm of f32 rows,
-// or silu(gate) * up of f32 rows [gate | up] (2 K values each).
-enum { GEMV_PLAIN = 0, GEMV_NORM = 1, GEMV_SWIGLU = 2 };
-struct GemvInput {
-  int mode = GEMV_PLAIN;
+// What the streaming GEMV of plain weights does besides the product: RMSNorm of its f32 activation rows
+// (norm_w given), and silu(gate) * up of a matrix [gate; up] (pairs: half as many outputs).
+struct GemvForm {
   const void* norm_w = nullptr;
   int norm_type = E_F32;
   float eps = 0.f;
+  int pairs = 0;
 };
 bool gemv_plain_takes(const WRef& w, int64_t M);
 int launch_gemv_plain(const WRef& w, const void* x, int x_type, int M, float* y, const float* residual,
-                      cudaStream_t s, bool* handled, const GemvInput& in = GemvInput());
+                      cudaStream_t s, bool* handled, const GemvForm& form = GemvForm());
 size_t gemv_mma_workspace_bytes(const WRef& w, int x_type, int M);
 int launch_gemv_mma(const WRef& w, const void* x, int x_type, int M, float* y, const float* residual,
                     void* workspace, cudaStream_t s, bool* handled);

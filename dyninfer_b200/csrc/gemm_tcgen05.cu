@@ -820,9 +820,15 @@ __global__ void __launch_bounds__(256)
 tg_split_reduce_kernel(const float* __restrict__ partial, int splits, int64_t count, float* y, const float* residual) {
   const int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x;
   if (i >= count) return;
+  float t[8];  // at most eight splits, all under way together
+#pragma unroll
+  for (int z = 0; z < 8; z++) t[z] = z < splits ? partial[(int64_t)z * count + i] : 0.f;
+  const float r = residual ? residual[i] : 0.f;
   float v = 0.f;
-  for (int z = 0; z < splits; z++) v += partial[(int64_t)z * count + i];
-  if (residual) v += residual[i];
+#pragma unroll
+  for (int z = 0; z < 8; z++)
+    if (z < splits) v += t[z];
+  if (residual) v += r;
   y[i] = v;
 }
 

@@ -153,25 +153,33 @@ norm_prepare_kernel(const float* __restrict__ x, const float* __restrict__ parti
   __shared__ float red[32];
   const int64_t row = blockIdx.x;
   float v[PER], wv[PER];
+  // all elements of one slice are under way together; each element adds its slices in ascending order
+  const float* first = S ? partial + row * width : x + row * width;
 #pragma unroll
   for (int k = 0; k < PER; k++) {
     const int64_t i = threadIdx.x + (int64_t)k * blockDim.x;
-    float t = 0.f;
-    if (i < width) {
-      if (S) {
-        for (int z = 0; z < S; z++) t += partial[((int64_t)z * rows + row) * width + i];
-      } else {
-        t = x[row * width + i];
-      }
-    }
-    v[k] = t;
+    v[k] = i < width ? first[i] : 0.f;
   }
-  if (residual) {
+  for (int z = 1; z < S; z++) {
+    const float* p = partial + ((int64_t)z * rows + row) * width;
+    float t[PER];
 #pragma unroll
     for (int k = 0; k < PER; k++) {
       const int64_t i = threadIdx.x + (int64_t)k * blockDim.x;
-      if (i < width) v[k] += residual[row * width + i];
+      t[k] = i < width ? p[i] : 0.f;
     }
+#pragma unroll
+    for (int k = 0; k < PER; k++) v[k] += t[k];
+  }
+  if (residual) {
+    float t[PER];
+#pragma unroll
+    for (int k = 0; k < PER; k++) {
+      const int64_t i = threadIdx.x + (int64_t)k * blockDim.x;
+      t[k] = i < width ? residual[row * width + i] : 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < PER; k++) v[k] += t[k];
   }
 #pragma unroll
   for (int k = 0; k < PER; k++) {
@@ -231,11 +239,15 @@ silu_prepare_kernel(const float* __restrict__ gu, int64_t I, __half* __restrict_
   };
   float mx = 0.f, sc, is;
   if constexpr (PER > 0) {
-    float v[PER];
+    float v[PER], up[PER];
 #pragma unroll
     for (int k = 0; k < PER; k++) {
       const int64_t i = threadIdx.x + (int64_t)k * blockDim.x;
-      v[k] = i < I ? val(i) : 0.f;
+      v[k] = i < I ? g[i] : 0.f, up[k] = i < I ? g[I + i] : 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < PER; k++) {
+      v[k] = (v[k] / (1.0f + expf(-v[k]))) * up[k];
       mx = fmaxf(mx, fabsf(v[k]));
     }
     f16_row_scale(mx, red, &sc, &is);

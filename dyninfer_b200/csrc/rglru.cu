@@ -319,12 +319,13 @@ rglru_scan_kernel(RglruArgs a, int64_t rows, int64_t base, int64_t slot, const f
   const float by = live ? vec_at(a.by, ch) : 0.f;
   for (int64_t p0 = 0; p0 < rows; p0 += SC_PASS) {
     const int64_t t0 = p0 + seg * SC_LEN;
-    float x[SC_LEN], y[SC_LEN];
+    float x[SC_LEN], y[SC_LEN], gate[SC_LEN];
 #pragma unroll
     for (int i = 0; i < SC_LEN; i++) {
       const bool in = live && t0 + i < rows;
       x[i] = in ? av[(t0 + i) * a.width + ch] : 1.f;
       y[i] = in ? bv[(t0 + i) * a.width + ch] : 0.f;
+      gate[i] = in ? a.y.ptr[(t0 + i) * a.y.ld + ch] : 0.f;
     }
     float A = 1.f, B = 0.f;
 #pragma unroll
@@ -342,7 +343,7 @@ rglru_scan_kernel(RglruArgs a, int64_t rows, int64_t base, int64_t slot, const f
     for (int i = 0; i < SC_LEN; i++) {
       S = fmaf(x[i], S, y[i]);
       if (live && t0 + i < rows)
-        a.out[(t0 + i) * a.width + ch] = S * gelu_tanh_of(a.y.ptr[(t0 + i) * a.y.ld + ch] + by);
+        a.out[(t0 + i) * a.width + ch] = S * gelu_tanh_of(gate[i] + by);
     }
     __syncthreads();
   }

@@ -464,6 +464,13 @@ int enqueue_gqa_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t ch
       // [gate; up] as one product into rows of [gate | up], then the activation
       if (session_linear(s, L.gate_up, s->xn, E_F32, rows, s->gu1, nullptr)) return 1;
       if (launch_silu_mul_rows(s->gu1, rows, c.inter, s->act, st)) return 1;
+    } else if (L.gate_up.data && gemv_plain_takes(L.gate_up, rows)) {
+      // plain 16-bit weights, a few rows: the streaming GEMV takes gate and up rows in pairs
+      GemvForm form;
+      form.pairs = 1;
+      bool handled = false;
+      if (launch_gemv_plain(L.gate_up, s->xn, E_F32, (int)rows, s->act, nullptr, st, &handled, form)) return 1;
+      DYN_CHECK(handled, "streaming GEMV refused a product it had accepted");
     } else if (L.gate.enc == L.up.enc && rows <= 4 && !fast_gemv) {
       if (launch_linear_swiglu(L.gate, L.up, s->xn, rows, s->act, st)) return 1;
     } else {

@@ -359,23 +359,23 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
     for (const WRef& w : L.in) fuse = fuse && takes(w);
     for (const WRef* w : {&L.o, &L.gate, &L.up, &L.down}) fuse = fuse && takes(*w);
   }
-  // A few rows of 16-bit weights: the streaming GEMV forms its normalised / gated input itself.
+  // A few rows of 16-bit weights: the streaming GEMV normalises its input and gates its output itself.
   bool stream = rows <= 4;
   for (const MixerLayer& L : s->mix) {
     for (const WRef& w : L.in) stream = stream && gemv_plain_takes(w, rows);
-    if (L.c.ff) stream = stream && L.gate_up.data && gemv_plain_takes(L.gate_up, rows) && gemv_plain_takes(L.down, rows);
+    if (L.c.ff) stream = stream && L.gate_up.data && gemv_plain_takes(L.gate_up, rows);
   }
-  GemvInput formed;
-  auto streamed = [&](const WRef& w, const float* x, float* y, const float* residual) -> int {
+  GemvForm form;
+  auto streamed = [&](const WRef& w, const float* x, float* y) -> int {
     bool handled = false;
-    if (launch_gemv_plain(w, x, E_F32, (int)rows, y, residual, st, &handled, formed)) return 1;
+    if (launch_gemv_plain(w, x, E_F32, (int)rows, y, nullptr, st, &handled, form)) return 1;
     DYN_CHECK(handled, "streaming GEMV refused a product it had accepted");
     return 0;
   };
   int pending = 0;  // K-split sums in gpart that `hidden` still lacks
   auto norm = [&](const NormW& w) -> int {
     if (stream) {
-      formed.mode = GEMV_NORM, formed.norm_w = w.ptr, formed.norm_type = w.type, formed.eps = c.eps;
+      form.norm_w = w.ptr, form.norm_type = w.type, form.eps = c.eps;
       return 0;
     }
     if (!fuse) return launch_rms_norm(s->hidden, w.ptr, w.type, rows, H, c.eps, s->xn, st);
@@ -398,7 +398,7 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
   };
   // a product of the normalised rows
   auto from_norm = [&](const WRef& w, float* y) -> int {
-    if (stream) return streamed(w, s->hidden, y, nullptr);
+    if (stream) return streamed(w, s->hidden, y);
     return fuse ? gemm(w, nullptr, y, nullptr, false) : session_linear(s, w, s->xn, E_F32, rows, y, nullptr);
   };
   // hidden += W x; `last`: no norm of this function follows to add deferred sums
@@ -426,9 +426,9 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
     if (norm(L.norm2)) return 1;
     bool prepared = false;
     if (stream) {
-      if (from_norm(L.gate_up, s->gu1)) return 1;
-      formed.mode = GEMV_SWIGLU;
-      if (streamed(L.down, s->gu1, s->hidden, s->hidden)) return 1;
+      form.pairs = 1;
+      if (from_norm(L.gate_up, s->act) || to_hidden(L.down, s->act, false, final_layer)) return 1;
+      form.pairs = 0;
       continue;
     }
     if (L.gate_up.data) {

@@ -397,7 +397,8 @@ def main():
         if args.arch_profile:
             arch_bench.profile_case(args.arch_profile, args.arch_size.split(",")[0], args.arch_prompt, 4)
         else:
-            arch_bench.run(args.arch_size.split(","), args.arch_prompt, args.steps, args.warmup, ClockSampler(local_rank))
+            arch_bench.run(args.arch_size.split(","), args.arch_prompt, args.steps, args.warmup,
+                           lambda: ClockSampler(local_rank))
         return
 
     import torch

@@ -32,9 +32,9 @@ SIZES = {"0.4b": (1024, 12, 8, 256, (1024, 4), 3072, 4),
 def zupudra_doc(size: str) -> dict:
     width, layers, heads, rank, (rw, blocks), ff, _ = SIZES[size]
     mlp = {"kind": "dense", "ff": ff}
-    decay = [1.0 - 2.0 ** -(5 + 3 * i / heads) for i in range(heads)]
+    decay = [1.0 - 2.0 ** -(4.5 + 4 * i / heads) for i in range(heads)]
     kinds = [{"type": "retention", "mixer": {"heads": heads, "dim": 128, "vdim": 128, "decay": decay,
-                                             "rot": {"dims": 128, "base": 1e6}}, "mlp": mlp},
+                                             "rot": {"dims": 128, "base": 5e5}}, "mlp": mlp},
              {"type": "rglru", "mixer": {"width": rw, "blocks": blocks, "conv": 4}, "mlp": mlp},
              {"type": "latent_attention", "mixer": {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": rank,
                                                     "scale": 128 ** -0.5}, "mlp": mlp}]
@@ -109,7 +109,7 @@ def run(sizes, prompt_len: int, steps: int, warmup: int, clocks) -> None:
         line = {"metric": "arch_tokens_per_s", "arch": "zupudra", "size": size, "prompt": prompt_len, "steps": steps,
                 "warmup": warmup, "dtype": "bf16 weights and cache", "data": "synthetic", "n_gpus": 1,
                 "l2": "each decode step streams more weight bytes than L2 holds"}
-        with clocks as c:
+        with clocks() as c:
             for kind in ("zupudra", "qwen3"):
                 line[kind] = measure(checkpoint(kind, size), prompt_len, steps, warmup)
         line["clocks"] = c.summary()

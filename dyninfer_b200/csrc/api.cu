@@ -161,13 +161,13 @@ void set_launch_counter(uint64_t* p) { g_counter = p ? p : &g_default_counter; }
 
 static bool aligned(const void* p, size_t a) { return (reinterpret_cast<uintptr_t>(p) % a) == 0; }
 
-int wref_from_api(const dyninfer_cuda_weight_t* w, WRef* out) {
+int wref_from_api(const dyninfer_cuda_weight_t* w, WRef* out, bool any_width) {
   DYN_CHECK(w != nullptr, "weight descriptor is NULL");
   DYN_CHECK(w->encoding >= E_F32 && w->encoding <= E_LAST, "unknown encoding %d", w->encoding);
   DYN_CHECK(w->rows >= 0 && w->cols > 0, "weight shape [%lld, %lld] is invalid",
             (long long)w->rows, (long long)w->cols);
   int unit = enc_block_elems(w->encoding);
-  if (unit < 4) unit = 4;
+  if (unit < 4 && !(any_width && unit == 1)) unit = 4;
   DYN_CHECK(w->cols % unit == 0, "cols %lld is not a multiple of %d for encoding %d",
             (long long)w->cols, unit, w->encoding);
   DYN_CHECK(w->data != nullptr && aligned(w->data, 16), "weight data must be a 16-byte aligned device pointer");
@@ -239,7 +239,7 @@ int dyninfer_cuda_dequant(const dyninfer_cuda_weight_t* w, float* out_dev, void*
 int dyninfer_cuda_embedding_gather(const dyninfer_cuda_weight_t* w, const int64_t* tokens_dev,
                                    int64_t count, float* out_dev, void* stream) {
   WRef r;
-  if (wref_from_api(w, &r)) return 1;
+  if (wref_from_api(w, &r, true)) return 1;
   DYN_CHECK(count >= 0, "count must be >= 0");
   DYN_CHECK(count == 0 || tokens_dev, "tokens is NULL");
   if (count == 0) return 0;
@@ -251,7 +251,7 @@ int dyninfer_cuda_embedding_gather(const dyninfer_cuda_weight_t* w, const int64_
 int dyninfer_cuda_linear(const dyninfer_cuda_weight_t* w, const void* x_dev, int x_type, int64_t m,
                          float* y_dev, void* stream) {
   WRef r;
-  if (wref_from_api(w, &r)) return 1;
+  if (wref_from_api(w, &r, true)) return 1;
   DYN_CHECK(x_dev && aligned(x_dev, 16), "x must be a 16-byte aligned device pointer");
   DYN_CHECK(y_dev != nullptr, "y is NULL");
   if (require_device()) return 1;

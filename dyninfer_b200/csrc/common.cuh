@@ -198,7 +198,7 @@ struct WRef {
   }
 };
 
-int wref_from_api(const dyninfer_cuda_weight_t* w, WRef* out);
+int wref_from_api(const dyninfer_cuda_weight_t* w, WRef* out, bool any_width = false);  // any_width: plain rows of any length
 
 // ---- small device helpers -------------------------------------------------------
 __device__ __forceinline__ uint32_t ld_u16(const uint8_t* p) {

@@ -53,8 +53,9 @@ def mixer_entry(layers: list, i: int) -> dict:
         raise ValueError(f"layer {i}: unknown feed-forward `{mlp['kind']}`")
     e = {"type": kind, "tensors": owner(layers, i), "ff": int(mlp["ff"]) if mlp else 0}
     if kind == "retention":
-        e.update(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), rot_dims=int(m["rot"]["dims"]),
-                 rot_base=float(m["rot"]["base"]), decay=[float(d) for d in m["decay"]])
+        rot = m.get("rot") or {"dims": 0, "base": 0.0}
+        e.update(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), rot_dims=int(rot["dims"]),
+                 rot_base=float(rot["base"]), decay=[float(d) for d in m["decay"]])
     elif kind == "rglru":
         e.update(width=int(m["width"]), blocks=int(m["blocks"]), taps=int(m["conv"]))
     else:

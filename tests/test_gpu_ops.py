@@ -282,3 +282,32 @@ def test_argmax_first_maximum(native_lib, oracle):
     v[9] = -3.0
     assert ops.argmax(torch.from_numpy(v).cuda()) == 9
     assert ops.argmax(torch.tensor([2.0]).cuda()) == 0
+
+
+@pytest.mark.parametrize("enc", ["plain.bf16", "plain.f16"])
+@pytest.mark.parametrize("rows,cols", [(1, 256), (7, 1280), (149, 512), (1500, 2048), (2051, 6144), (9000, 256)])
+def test_streaming_gemv_of_plain_weights(native_lib, oracle, enc, rows, cols):
+    """One to eight rows: outputs dealt over CTAs in uneven blocks, rows cut into spans of K where there are few."""
+    from dyninfer_b200 import ops
+    dw, ow = make_pair(oracle, enc, rows, cols, seed=rows)
+    w = oracle.dequant(ow).astype(np.float64)
+    for m in (1, 2, 3, 4, 5, 8):
+        x = np.random.default_rng(m).standard_normal((m, cols)).astype(np.float32)
+        want = x @ w.T
+        got = ops.linear(dw, torch.from_numpy(x).cuda()).cpu().numpy()
+        assert np.abs(got - want).max() <= 2e-6 * np.abs(x).max() * np.abs(w).max() * cols, m
+
+
+@pytest.mark.parametrize("enc", ["plain.bf16", "plain.f16", "plain.f32"])
+@pytest.mark.parametrize("rows,cols", [(5, 3), (130, 67), (64, 36), (300, 129)])
+def test_plain_weights_of_any_width(native_lib, oracle, enc, rows, cols):
+    from dyninfer_b200 import ops
+    rng = np.random.default_rng(rows)
+    w = rng.standard_normal((rows, cols)).astype(np.float32)
+    raw = {"plain.bf16": synth.f32_to_bf16_bits(w), "plain.f16": w.astype(np.float16), "plain.f32": w}[enc]
+    w = {"plain.bf16": lambda: synth.bf16_bits_to_f32(raw), "plain.f16": lambda: raw.astype(np.float32), "plain.f32": lambda: w}[enc]()
+    dw = ops.DeviceWeight(enc, rows, cols, raw)
+    for m in (1, 4, 9, 70):
+        x = rng.standard_normal((m, cols)).astype(np.float32)
+        got = ops.linear(dw, torch.from_numpy(x).cuda()).cpu().numpy()
+        assert np.abs(got - x.astype(np.float64) @ w.astype(np.float64).T).max() <= 1e-5 * cols, m

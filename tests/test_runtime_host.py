@@ -31,6 +31,7 @@ class RecordingLibrary:
         self.keys = None
         self.fail_next_invoke = None
         self.slot_invokes = []     # (slot, tokens, last, start_pos, want_logits)
+        self.portions = []         # (slot, tokens, start_pos, wanted rows)
         self.batch_steps = []      # ([(slot, token, position)], want_logits)
 
     def dyninfer_cuda_last_error(self):
@@ -108,6 +109,16 @@ class RecordingLibrary:
         if want_logits:
             self._batch_logits = (C.c_float * (n * VOCAB))(*[float(i // VOCAB) for i in range(n * VOCAB)])
             out_logits._obj.contents = self._batch_logits
+        return 0
+
+
+    def dyninfer_cuda_session_invoke_portion(self, h, tokens, n, start, slot, want, n_want, out_logits, out_token):
+        rows = [int(want[i]) for i in range(n_want)]
+        self.portions.append((int(slot), [int(tokens[i]) for i in range(n)], int(start), rows))
+        if n_want:                                  # row r of the portion answers with its absolute position
+            self._portion = (C.c_float * (n_want * VOCAB))(*[float(start + r) for r in rows for _ in range(VOCAB)])
+            out_logits._obj.contents = self._portion
+        out_token._obj.value = self.script(start + n - 1)
         return 0
 
 
@@ -302,3 +313,47 @@ def test_batched_session_places_sequences_in_slots(model, fake):
         assert s.positions == [0, 0, 0, 0]
     with pytest.raises(DynInferError, match="batch_size must be >= 1"):
         model.create_batched_session(SessionConfig(batch_size=0))
+
+
+def test_portions_continue_the_sequence_and_map_wanted_rows(model, fake):
+    ids = [(5 * i + 2) % VOCAB for i in range(1200)]
+    with model.create_session(SessionConfig(max_sequence_length=2048)) as s:
+        got = s.extend(ids[:3], [2, 0])
+        assert fake.portions == [(0, ids[:3], 0, [0, 2])] and got[:, 0].tolist() == [2.0, 0.0]
+        got = s.extend(ids[3:1200], [1196, 0, 511, 512, 511])      # longer than a chunk: pieces of 512, any order of rows
+        assert [(len(t), start, rows) for _, t, start, rows in fake.portions[1:]] == \
+            [(512, 3, [0, 511]), (512, 515, [0]), (173, 1027, [172])]
+        assert got[:, 0].tolist() == [1199.0, 3.0, 514.0, 515.0, 514.0]
+        assert s.position() == 1200 and s.history == ids and s.extend([1], []).shape == (0, VOCAB)
+        for tokens, want, match in (([], [], "non-empty"), ([1], [1], "wanted rows"), ([1] * 900, [], "exceeds session/KV limit")):
+            with pytest.raises(DynInferError, match=match):
+                s.extend(tokens, want)
+        assert s.position() == 1201 and len(fake.portions) == 5
+
+
+def test_slots_of_a_batched_session_take_portions(model, fake):
+    with model.create_batched_session(SessionConfig(max_sequence_length=64, batch_size=2)) as s:
+        s.extend_slot(1, [1, 2, 3], restart=True)
+        s.extend_slot(1, [4, 5])
+        s.step({1: 6})
+        s.extend_slot(1, [7])
+        s.extend_slot(1, [8, 9], restart=True)                       # the slot goes to another sequence
+        assert [(slot, start) for slot, _, start, _ in fake.portions] == [(1, 0), (1, 3), (1, 6), (1, 0)]
+        assert fake.batch_steps == [([(1, 6, 5)], 0)] and s.positions == [0, 2]
+        with pytest.raises(DynInferError, match="slot 2 outside"):
+            s.extend_slot(2, [1])
+
+
+def test_trace_replay_hands_slots_on(model, fake):
+    from dyninfer_b200.trace_run import Replay
+    with model.create_batched_session(SessionConfig(max_sequence_length=64, batch_size=2)) as s:
+        r = Replay(s, 2)
+        assert r.run({"entries": [{"id": "a", "tokens": [1, 2], "want": []}], "end": []}) is None
+        got = r.run({"entries": [{"id": "b", "tokens": [3], "want": [0]}, {"id": "a", "tokens": [4, 5], "want": [1, 0]}], "end": ["a"]})
+        assert got[:, 0].tolist() == [0.0, 3.0, 2.0]
+        r.run({"entries": [{"id": "c", "tokens": [6], "want": []}], "end": ["b", "c"]})
+        r.run({"entries": [{"id": "a", "tokens": [7], "want": []}], "end": []})     # the name may come again, as a new request
+        assert [(slot, start) for slot, _, start, _ in fake.portions] == [(0, 0), (1, 0), (0, 2), (0, 0), (1, 0)]
+        r.run({"entries": [{"id": "d", "tokens": [8], "want": []}], "end": []})
+        with pytest.raises(RuntimeError, match="no free slot"):
+            r.run({"entries": [{"id": "e", "tokens": [8], "want": []}], "end": []})

@@ -413,11 +413,19 @@ __device__ __forceinline__ void split_into(AFrag& f, int i, float x) {
   const Tf32Pair p = tf32_split(x);
   f.hi[i] = p.hi, f.lo[i] = p.lo;
 }
-__device__ __forceinline__ void mma3(float (&c)[4], const AFrag& a, float b0, float b1) {
-  const Tf32Pair p = tf32_split(b0), q = tf32_split(b1);
-  mma_tf32(c, a.lo, p.hi, q.hi);
-  mma_tf32(c, a.hi, p.lo, q.lo);
-  mma_tf32(c, a.hi, p.hi, q.hi);
+// c[nt] += a b[nt] for NT column tiles of one k-step; b(nt, 0 / 1) are the tile's two operand values. Term by term,
+// so that the products of consecutive instructions are independent.
+template <int NT, class B>
+__device__ __forceinline__ void mma3(float (&c)[NT][4], const AFrag& a, B b) {
+  Tf32Pair p[NT], q[NT];
+#pragma unroll
+  for (int nt = 0; nt < NT; nt++) p[nt] = tf32_split(b(nt, 0)), q[nt] = tf32_split(b(nt, 1));
+#pragma unroll
+  for (int nt = 0; nt < NT; nt++) mma_tf32(c[nt], a.lo, p[nt].hi, q[nt].hi);
+#pragma unroll
+  for (int nt = 0; nt < NT; nt++) mma_tf32(c[nt], a.hi, p[nt].lo, q[nt].lo);
+#pragma unroll
+  for (int nt = 0; nt < NT; nt++) mma_tf32(c[nt], a.hi, p[nt].hi, q[nt].hi);
 }
 
 // rows x cols floats (cols <= 128, both 16-byte aligned) into shared memory, zeros to `fill_rows` x 128
@@ -433,8 +441,9 @@ __device__ __forceinline__ void stage_rows(float* dst, int pitch, const float* s
 }
 
 constexpr int TCS_SMEM = RT_C * (TC_BP + 72) * 4;
-// U of one (chunk, head, 64 rows of the state): A = (decayed k)^T, B = v. Warp: 16 rows x half of the columns.
-__global__ void __launch_bounds__(256) retention_chunk_state_tc_kernel(RetentionArgs a, int64_t rows) {
+constexpr int TC_THREADS = 512;  // sixteen warps: four groups of 16 rows x four of 32 columns
+// U of one (chunk, head, 64 rows of the state): A = (decayed k)^T, B = v. Columns past vdim hold zeros.
+__global__ void __launch_bounds__(TC_THREADS) retention_chunk_state_tc_kernel(RetentionArgs a, int64_t rows) {
   extern __shared__ __align__(16) float ts_smem[];
   float* vs = ts_smem;                 // [t][TC_BP]
   float* ks = vs + RT_C * TC_BP;       // [t][72]
@@ -442,8 +451,8 @@ __global__ void __launch_bounds__(256) retention_chunk_state_tc_kernel(Retention
   const int D = a.dim, E = a.vdim, h = blockIdx.y, d0 = blockIdx.z * 64;
   const int64_t c = blockIdx.x, t0 = c * RT_C;
   const int n = (int)min((int64_t)RT_C, rows - t0);
-  stage_rows(vs, TC_BP, a.v.ptr + t0 * a.v.ld + (int64_t)h * E, a.v.ld, n, E, RT_C, tid, 256);
-  for (int i = tid; i < RT_C * 16; i += 256) {
+  stage_rows(vs, TC_BP, a.v.ptr + t0 * a.v.ld + (int64_t)h * E, a.v.ld, n, E, RT_C, tid, TC_THREADS);
+  for (int i = tid; i < RT_C * 16; i += TC_THREADS) {
     const int t = i / 16, d = (i % 16) * 4;
     const bool live = t < n && d0 + d < D;
     const float* src = a.k.ptr + t0 * a.k.ld + (int64_t)h * D;
@@ -452,10 +461,10 @@ __global__ void __launch_bounds__(256) retention_chunk_state_tc_kernel(Retention
                  "r"(live ? 16 : 0) : "memory");
   }
   const float decay = a.decay[h];
-  const int mt = warp & 3, nh = warp >> 2;
+  const int mt = warp & 3, nq = warp >> 2;
   asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory");
   __syncthreads();
-  float acc[8][4] = {};
+  float acc[4][4] = {};
 #pragma unroll
   for (int kk = 0; kk < RT_C / 8; kk++) {
     const int ta = 8 * kk + t4, tb = ta + 4;
@@ -463,16 +472,12 @@ __global__ void __launch_bounds__(256) retention_chunk_state_tc_kernel(Retention
     const float *ka = ks + ta * 72 + 16 * mt + g, *kb = ks + tb * 72 + 16 * mt + g;
     AFrag f;
     split_into(f, 0, ka[0] * wa), split_into(f, 1, ka[8] * wa), split_into(f, 2, kb[0] * wb), split_into(f, 3, kb[8] * wb);
-#pragma unroll
-    for (int nt = 0; nt < 8; nt++) {
-      const int e = nh * 64 + 8 * nt + g;
-      if (nh * 64 + 8 * nt < E) mma3(acc[nt], f, vs[ta * TC_BP + e], vs[tb * TC_BP + e]);
-    }
+    mma3<4>(acc, f, [&](int nt, int half) { return vs[(half ? tb : ta) * TC_BP + nq * 32 + 8 * nt + g]; });
   }
   float* U = a.scratch + ((c * a.heads + h) * D) * (int64_t)E;
 #pragma unroll
-  for (int nt = 0; nt < 8; nt++) {
-    const int e = nh * 64 + 8 * nt + 2 * t4;
+  for (int nt = 0; nt < 4; nt++) {
+    const int e = nq * 32 + 8 * nt + 2 * t4;
     if (e >= E) continue;
 #pragma unroll
     for (int i = 0; i < 2; i++) {
@@ -482,95 +487,91 @@ __global__ void __launch_bounds__(256) retention_chunk_state_tc_kernel(Retention
   }
 }
 
-constexpr int TCO_SMEM = (2 * RT_C * TC_AP + RT_C * TC_BP + TC_D * TC_BP + RT_C * TC_SP + 2 * RT_C) * 4;
-// Outputs of one (chunk, head). Warp: 16 tokens x half of the keys, then x half of the value columns.
-__global__ void __launch_bounds__(256) retention_chunk_out_tc_kernel(RetentionArgs a, int64_t rows, int64_t base) {
+constexpr int TCO_SMEM = (2 * RT_C * TC_AP + RT_C * TC_BP + TC_D * TC_BP + RT_C * TC_SP + 4 * RT_C) * 4;
+// Outputs of one (chunk, head). Warp: 16 tokens x a quarter of the keys, then x a quarter of the value columns.
+__global__ void __launch_bounds__(TC_THREADS) retention_chunk_out_tc_kernel(RetentionArgs a, int64_t rows, int64_t base) {
   extern __shared__ __align__(16) float to_smem[];
   float* qs = to_smem;                 // [t][TC_AP]
   float* ks = qs + RT_C * TC_AP;       // [s][TC_AP]
   float* vs = ks + RT_C * TC_AP;       // [s][TC_BP]
   float* ps = vs + RT_C * TC_BP;       // [d][TC_BP]
   float* ss = ps + TC_D * TC_BP;       // [t][TC_SP]
-  float* sums = ss + RT_C * TC_SP;     // [half][t]
+  float* sums = ss + RT_C * TC_SP;     // [column quarter][t]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
   const int D = a.dim, E = a.vdim, h = blockIdx.y;
   const int64_t c = blockIdx.x, t0 = c * RT_C;
   const int n = (int)min((int64_t)RT_C, rows - t0);
-  const int mt = warp & 3, nh = warp >> 2;
+  const int mt = warp & 3, nq = warp >> 2;
   const bool past = c > 0 || base > 0;
-  stage_rows(qs, TC_AP, a.q.ptr + t0 * a.q.ld + (int64_t)h * D, a.q.ld, n, D, RT_C, tid, 256);
-  stage_rows(ks, TC_AP, a.k.ptr + t0 * a.k.ld + (int64_t)h * D, a.k.ld, n, D, RT_C, tid, 256);
+  stage_rows(qs, TC_AP, a.q.ptr + t0 * a.q.ld + (int64_t)h * D, a.q.ld, n, D, RT_C, tid, TC_THREADS);
+  stage_rows(ks, TC_AP, a.k.ptr + t0 * a.k.ld + (int64_t)h * D, a.k.ld, n, D, RT_C, tid, TC_THREADS);
   asm volatile("cp.async.commit_group;" ::: "memory");
-  if (past) stage_rows(ps, TC_BP, a.scratch + ((c * a.heads + h) * D) * (int64_t)E, E, D, E, (D + 7) / 8 * 8, tid, 256);
-  stage_rows(vs, TC_BP, a.v.ptr + t0 * a.v.ld + (int64_t)h * E, a.v.ld, n, E, RT_C, tid, 256);
+  if (past) stage_rows(ps, TC_BP, a.scratch + ((c * a.heads + h) * D) * (int64_t)E, E, D, E, (D + 7) / 8 * 8, tid, TC_THREADS);
+  stage_rows(vs, TC_BP, a.v.ptr + t0 * a.v.ld + (int64_t)h * E, a.v.ld, n, E, RT_C, tid, TC_THREADS);
   asm volatile("cp.async.commit_group;" ::: "memory");
   const float decay = a.decay[h];
   asm volatile("cp.async.wait_group 1;" ::: "memory");
   __syncthreads();
   // ---- decayed causal scores
   {
-    float s[4][4] = {};
-    for (int d = 0; d < D; d += 8) {
-      AFrag f;
-      const float* q = qs + (16 * mt + g) * TC_AP + d + t4;
-      split_into(f, 0, q[0]), split_into(f, 1, q[8 * TC_AP]), split_into(f, 2, q[4]), split_into(f, 3, q[8 * TC_AP + 4]);
-#pragma unroll
-      for (int nt = 0; nt < 4; nt++) {
-        const float* k = ks + (nh * 32 + 8 * nt + g) * TC_AP + d + t4;
-        mma3(s[nt], f, k[0], k[4]);
+    float s[2][4] = {};
+    if (nq <= mt) {  // keys 16 nq .. are not all later than the tokens
+#pragma unroll 4
+      for (int d = 0; d < D; d += 8) {
+        AFrag f;
+        const float* q = qs + (16 * mt + g) * TC_AP + d + t4;
+        split_into(f, 0, q[0]), split_into(f, 1, q[8 * TC_AP]), split_into(f, 2, q[4]), split_into(f, 3, q[8 * TC_AP + 4]);
+        mma3<2>(s, f, [&](int nt, int half) { return ks[(nq * 16 + 8 * nt + g) * TC_AP + d + t4 + 4 * half]; });
       }
     }
 #pragma unroll
-    for (int nt = 0; nt < 4; nt++)
+    for (int nt = 0; nt < 2; nt++)
 #pragma unroll
       for (int e = 0; e < 4; e++) {
-        const int t = 16 * mt + g + 8 * (e >> 1), u = nh * 32 + 8 * nt + 2 * t4 + (e & 1);
+        const int t = 16 * mt + g + 8 * (e >> 1), u = nq * 16 + 8 * nt + 2 * t4 + (e & 1);
         ss[t * TC_SP + u] = u <= t ? s[nt][e] * powf(decay, (float)(t - u)) : 0.f;
       }
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
-  float o[8][4] = {};
+  float o[4][4] = {};
   auto accumulate = [&](const float* A, int pitch, int depth, const float* B) {
+#pragma unroll 2
     for (int k = 0; k < depth; k += 8) {
       AFrag f;
       const float* p = A + (16 * mt + g) * pitch + k + t4;
       split_into(f, 0, p[0]), split_into(f, 1, p[8 * pitch]), split_into(f, 2, p[4]), split_into(f, 3, p[8 * pitch + 4]);
-#pragma unroll
-      for (int nt = 0; nt < 8; nt++) {
-        const float* b = B + (k + t4) * TC_BP + nh * 64 + 8 * nt + g;
-        if (nh * 64 + 8 * nt < E) mma3(o[nt], f, b[0], b[4 * TC_BP]);
-      }
+      mma3<4>(o, f, [&](int nt, int half) { return B[(k + t4 + 4 * half) * TC_BP + nq * 32 + 8 * nt + g]; });
     }
   };
   if (past) {  // the state before the chunk, decayed to each token
     accumulate(qs, TC_AP, D, ps);
     const float w0 = powf(decay, (float)(16 * mt + g + 1)), w1 = powf(decay, (float)(16 * mt + g + 9));
 #pragma unroll
-    for (int nt = 0; nt < 8; nt++) o[nt][0] *= w0, o[nt][1] *= w0, o[nt][2] *= w1, o[nt][3] *= w1;
+    for (int nt = 0; nt < 4; nt++) o[nt][0] *= w0, o[nt][1] *= w0, o[nt][2] *= w1, o[nt][3] *= w1;
   }
   accumulate(ss, TC_SP, 16 * (mt + 1), vs);  // later keys score zero
   // ---- norm over the head's value dims (columns past E hold zeros), gate
   float q0 = 0.f, q1 = 0.f;
 #pragma unroll
-  for (int nt = 0; nt < 8; nt++) {
+  for (int nt = 0; nt < 4; nt++) {
     q0 = fmaf(o[nt][0], o[nt][0], q0), q0 = fmaf(o[nt][1], o[nt][1], q0);
     q1 = fmaf(o[nt][2], o[nt][2], q1), q1 = fmaf(o[nt][3], o[nt][3], q1);
   }
   q0 += __shfl_xor_sync(0xffffffffu, q0, 1), q0 += __shfl_xor_sync(0xffffffffu, q0, 2);
   q1 += __shfl_xor_sync(0xffffffffu, q1, 1), q1 += __shfl_xor_sync(0xffffffffu, q1, 2);
-  if (t4 == 0) sums[nh * RT_C + 16 * mt + g] = q0, sums[nh * RT_C + 16 * mt + g + 8] = q1;
+  if (t4 == 0) sums[nq * RT_C + 16 * mt + g] = q0, sums[nq * RT_C + 16 * mt + g + 8] = q1;
   __syncthreads();
 #pragma unroll
   for (int i = 0; i < 2; i++) {
     const int t = 16 * mt + g + 8 * i;
     if (t >= n) continue;
-    const float inv = 1.0f / sqrtf((sums[t] + sums[RT_C + t]) / (float)E + a.eps);
+    const float inv = 1.0f / sqrtf(((sums[t] + sums[RT_C + t]) + (sums[2 * RT_C + t] + sums[3 * RT_C + t])) / (float)E + a.eps);
     const float* gate = a.g.ptr + (t0 + t) * a.g.ld + (int64_t)h * E;
     float* out = a.out + (t0 + t) * (int64_t)a.heads * E + (int64_t)h * E;
 #pragma unroll
-    for (int nt = 0; nt < 8; nt++) {
-      const int e = nh * 64 + 8 * nt + 2 * t4;
+    for (int nt = 0; nt < 4; nt++) {
+      const int e = nq * 32 + 8 * nt + 2 * t4;
       if (e >= E) continue;
       const float2 z = *reinterpret_cast<const float2*>(gate + e);
       *reinterpret_cast<float2*>(out + e) = make_float2(o[nt][2 * i] * inv * silu_of(z.x), o[nt][2 * i + 1] * inv * silu_of(z.y));
@@ -608,7 +609,7 @@ int launch_retention(const RetentionArgs& a, const StepRows& r, cudaStream_t st)
     const unsigned dt = (unsigned)((a.dim + 63) / 64), et = (unsigned)((a.vdim + 63) / 64);
     if (tensor_core_shape(a)) {
       if (ensure_dynamic_smem(reinterpret_cast<const void*>(retention_chunk_state_tc_kernel), TCS_SMEM)) return 1;
-      retention_chunk_state_tc_kernel<<<dim3(nc, (unsigned)a.heads, dt), 256, TCS_SMEM, st>>>(a, r.rows);
+      retention_chunk_state_tc_kernel<<<dim3(nc, (unsigned)a.heads, dt), TC_THREADS, TCS_SMEM, st>>>(a, r.rows);
     } else {
       retention_chunk_state_kernel<<<dim3(nc, (unsigned)a.heads, dt * et), 64, 0, st>>>(a, r.rows);
     }
@@ -618,7 +619,7 @@ int launch_retention(const RetentionArgs& a, const StepRows& r, cudaStream_t st)
   }
   if (tensor_core_shape(a)) {
     if (ensure_dynamic_smem(reinterpret_cast<const void*>(retention_chunk_out_tc_kernel), TCO_SMEM)) return 1;
-    retention_chunk_out_tc_kernel<<<dim3(nc, (unsigned)a.heads), 256, TCO_SMEM, st>>>(a, r.rows, r.base);
+    retention_chunk_out_tc_kernel<<<dim3(nc, (unsigned)a.heads), TC_THREADS, TCO_SMEM, st>>>(a, r.rows, r.base);
     count_launch();
     DYN_CUDA(cudaGetLastError());
     return 0;

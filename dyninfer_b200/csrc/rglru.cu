@@ -193,29 +193,50 @@ rglru_gates_tc_kernel(RglruArgs a, int64_t rows, const float* __restrict__ u, fl
   const int64_t t0 = (int64_t)blockIdx.y * GT_T;
   const int mt = warp & 3, mat = warp >> 2;
   float acc[8][4] = {};
+  constexpr int UQ = GT_T * GT_K / 4 / 256, WQ = 2 * GT_T * GT_K / 8 / 256;
+  float4 uq[UQ];
+  uint4 wq[WQ];
+  auto fetch = [&](int k0) {  // the next slice is under way while the current one is used
+#pragma unroll
+    for (int j = 0; j < UQ; j++) {
+      const int i = tid + 256 * j, tok = i / (GT_K / 4), k = (i % (GT_K / 4)) * 4;  // n is a multiple of 8: whole quads
+      uq[j] = t0 + tok < rows && k0 + k < n ? *reinterpret_cast<const float4*>(u + (t0 + tok) * a.width + blk * n + k0 + k)
+                                            : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int j = 0; j < WQ; j++) {
+      const int i = tid + 256 * j, m = i / (GT_T * GT_K / 8), o = (i / (GT_K / 8)) % GT_T, k = (i % (GT_K / 8)) * 8;
+      wq[j] = o0 + o < n && k0 + k < n
+                  ? *reinterpret_cast<const uint4*>((m ? a.ri.ptr : a.ra.ptr) + (((int64_t)blk * n + o0 + o) * n + k0 + k) * 2)
+                  : make_uint4(0, 0, 0, 0);
+    }
+  };
+  fetch(0);
   for (int k0 = 0; k0 < n; k0 += GT_K) {
 #pragma unroll
-    for (int j = 0; j < GT_T * GT_K / 4 / 256; j++) {
+    for (int j = 0; j < UQ; j++) {
       const int i = tid + 256 * j, tok = i / (GT_K / 4), k = (i % (GT_K / 4)) * 4;
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);  // n is a multiple of 8: whole quads
-      if (t0 + tok < rows && k0 + k < n) v = *reinterpret_cast<const float4*>(u + (t0 + tok) * a.width + blk * n + k0 + k);
-      const float x[4] = {v.x, v.y, v.z, v.w};
+      const float x[4] = {uq[j].x, uq[j].y, uq[j].z, uq[j].w};
+      uint32_t t3[3][2];
 #pragma unroll
       for (int e = 0; e < 4; e++) {
         const __nv_bfloat16 h = __float2bfloat16_rn(x[e]);
         const float r1 = x[e] - __bfloat162float(h);
         const __nv_bfloat16 m = __float2bfloat16_rn(r1);
-        us[0][tok][k + e] = h, us[1][tok][k + e] = m, us[2][tok][k + e] = __float2bfloat16_rn(r1 - __bfloat162float(m));
+        const uint32_t b[3] = {__bfloat16_as_ushort(h), __bfloat16_as_ushort(m),
+                               __bfloat16_as_ushort(__float2bfloat16_rn(r1 - __bfloat162float(m)))};
+#pragma unroll
+        for (int s = 0; s < 3; s++) t3[s][e / 2] = e % 2 ? t3[s][e / 2] | (b[s] << 16) : b[s];
       }
+#pragma unroll
+      for (int s = 0; s < 3; s++) *reinterpret_cast<uint2*>(&us[s][tok][k]) = make_uint2(t3[s][0], t3[s][1]);
     }
 #pragma unroll
-    for (int j = 0; j < 2 * GT_T * GT_K / 8 / 256; j++) {
+    for (int j = 0; j < WQ; j++) {
       const int i = tid + 256 * j, m = i / (GT_T * GT_K / 8), o = (i / (GT_K / 8)) % GT_T, k = (i % (GT_K / 8)) * 8;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (o0 + o < n && k0 + k < n)
-        v = *reinterpret_cast<const uint4*>((m ? a.ri.ptr : a.ra.ptr) + (((int64_t)blk * n + o0 + o) * n + k0 + k) * 2);
-      *reinterpret_cast<uint4*>(&ws[m][o][k]) = v;
+      *reinterpret_cast<uint4*>(&ws[m][o][k]) = wq[j];
     }
+    if (k0 + GT_K < n) fetch(k0 + GT_K);
     __syncthreads();
 #pragma unroll
     for (int kk = 0; kk < GT_K / 16; kk++) {

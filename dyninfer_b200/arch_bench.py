@@ -109,9 +109,10 @@ def run(sizes, prompt_len: int, steps: int, warmup: int, clocks) -> None:
         line = {"metric": "arch_tokens_per_s", "arch": "zupudra", "size": size, "prompt": prompt_len, "steps": steps,
                 "warmup": warmup, "dtype": "bf16 weights and cache", "data": "synthetic", "n_gpus": 1,
                 "l2": "each decode step streams more weight bytes than L2 holds"}
+        paths = {kind: checkpoint(kind, size) for kind in ("zupudra", "qwen3")}
         with clocks() as c:
-            for kind in ("zupudra", "qwen3"):
-                line[kind] = measure(checkpoint(kind, size), prompt_len, steps, warmup)
+            for kind, path in paths.items():
+                line[kind] = measure(path, prompt_len, steps, warmup)
         line["clocks"] = c.summary()
         print(json.dumps(line), flush=True)
 

@@ -31,7 +31,7 @@ def gelu_tanh(z):
 
 
 def rotate_half(v, position, dims, base):
-    """The first `dims` entries of one head's vector, entry i paired with entry i + dims/2."""
+    """Rotates (v[i], v[i + dims/2]) by position * base^(-2i/dims) for i < dims/2; v[dims:] stays."""
     out = v.copy()
     half = dims // 2
     for i in range(half):

@@ -25,7 +25,7 @@ import os
 import struct
 from dataclasses import dataclass, field
 
-from . import zupudra
+from . import rufusun, zupudra
 
 # ggml type code -> (encoding id, elements per block, bytes per block)
 GGML_TYPES = {
@@ -448,7 +448,7 @@ def catalog_from_listed_layers(path: str, reader) -> Catalog:
 
 
 # config.json "architecture" -> reader; directories without the key follow the HF / MLX convention
-ARCHITECTURES = {zupudra.ARCHITECTURE: zupudra}
+ARCHITECTURES = {reader.ARCHITECTURE: reader for reader in (rufusun, zupudra)}
 
 
 def _architecture_reader(path: str):

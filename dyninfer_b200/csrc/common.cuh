@@ -255,6 +255,16 @@ struct TgIo {
 };
 int launch_dqgemm_tc(const WRef& w, const void* x, int x_type, int64_t M, float* y, const float* residual,
                      cudaStream_t s, bool* handled, TgIo* io = nullptr);
+// f32 rows -> the GEMM's activation operand.
+int launch_activation_prepare(const float* x, int64_t rows, int64_t K, __half* xh, float* inv_s, cudaStream_t s);
+// Grouped form for plain 16-bit weights: rows sorted by matrix; tile t multiplies rows [y, y + z) (z <= bn, 0: none)
+// of the operand by matrix bases[x] of the shape of w. The operand's buffer holds at least bn rows.
+struct TgGroups {
+  const int4* tiles = nullptr;             // device, [max_tiles]
+  const uint8_t* const* bases = nullptr;   // device
+  int max_tiles = 0, bn = 0;               // bn: a multiple of 16, at most 256
+};
+int launch_dqgemm_tc_grouped(const WRef& w, const TgGroups& g, const __half* xh, const float* inv_s, int64_t M, float* y, cudaStream_t s);
 // Whether launch_dqgemm_tc takes the product, and the activation rows its tiling pads M to.
 bool dqgemm_tc_takes(const WRef& w, int64_t M);
 int64_t dqgemm_tc_padded_rows(const WRef& w, int64_t M);
@@ -270,12 +280,14 @@ size_t gemv_cs_workspace_bytes(const WRef& w, int M);
 int launch_gemv_cs(const WRef& w, const void* x, int x_type, int M, float* y, const float* residual,
                    uint8_t* ws, cudaStream_t s, bool* handled);
 // What the streaming GEMV of plain weights does besides the product: RMSNorm of its f32 activation rows
-// (norm_w given), and silu(gate) * up of a matrix [gate; up] (pairs: half as many outputs).
+// (norm_w given), a bias per output, and silu(gate) * up of a matrix [gate; up] (pairs: half as many outputs).
 struct GemvForm {
   const void* norm_w = nullptr;
   int norm_type = E_F32;
   float eps = 0.f;
   int pairs = 0;
+  const void* bias = nullptr;
+  int bias_type = E_F32;
 };
 bool gemv_plain_takes(const WRef& w, int64_t M);
 int launch_gemv_plain(const WRef& w, const void* x, int x_type, int M, float* y, const float* residual,
@@ -298,10 +310,14 @@ int launch_norm_prepare(const float* x, const float* partial, int splits, const 
                         cudaStream_t s);
 // The same for the SwiGLU: rows of [gate | up] -> silu(gate) * up as the GEMM's activation operand.
 int launch_silu_prepare(const float* gate_up, int64_t rows, int64_t inter, __half* xh, float* inv_s, cudaStream_t s);
+// and for min(gate, limit) * sigmoid(1.702 min(gate, limit)) * (clamp(up, +-limit) + 1)
+int launch_clamped_glu_prepare(const float* gate_up, int64_t rows, int64_t inter, float limit, __half* xh, float* inv_s, cudaStream_t s);
 // One row of [gate | up] (2 * inter values, deferred or in `gate_up`): y = silu(gate) * up
 int launch_silu_mul_deferred(const Deferred& d, const float* gate_up, int64_t inter, float* y, cudaStream_t s);
 int launch_rope(float* x, int64_t s_rows, int64_t heads, int64_t d, int64_t start_pos,
                 const FreqTable& ft, cudaStream_t s);
+// y[row][:] += bias
+int launch_add_bias(float* y, const void* bias, int bias_type, int64_t rows, int64_t width, cudaStream_t s);
 int launch_silu_mul(const float* gate, const float* up, int64_t n, float* y, cudaStream_t s);
 int launch_silu_mul_rows(const float* gate_up, int64_t rows, int64_t inter, float* y, cudaStream_t s);
 
@@ -343,11 +359,17 @@ struct AttnArgs {
   // row_pos / row_seq are given (prefill chunks); lets the tensor-core prefill kernel take them
   int64_t uniform_base = -1, uniform_seq = 0;
   int64_t ldq = 0;  // floats between consecutive rows of q (0: dense, nh*d)
-  float scale = 0.f;  // score factor of the tensor-core prefill kernel (0: 1/sqrt(d))
+  // tensor-core prefill kernel only: score factor (0: 1/sqrt(d)), values of another width than keys (0: d; ctx rows
+  // are then nh * dv wide), scores capped to softcap * tanh(score / softcap) (0: as they are)
+  float scale = 0.f;
+  int64_t dv = 0;
+  float softcap = 0.f;
 };
 int launch_attention(const AttnArgs& a, cudaStream_t s);
 size_t attention_split_scratch_bytes(int64_t rows, int64_t nh, int64_t d, int nsplit);
 int launch_attention_split(const AttnArgs& a, float* part, int nsplit, cudaStream_t s, bool* handled);
+// Slices [row][head][nsplit][d + 2] (unnormalised output, maximum, sum) -> ctx [rows, nh * d].
+int launch_attention_merge(const float* part, int nsplit, float* ctx, int64_t rows, int64_t nh, int64_t d, cudaStream_t s);
 int launch_attention_prefill(const AttnArgs& a, int64_t base_pos, int64_t seq, cudaStream_t s, bool* handled);
 
 size_t argmax_scratch_bytes(int64_t n);

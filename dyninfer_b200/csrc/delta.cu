@@ -1,0 +1,763 @@
+// Gated delta rule: linear attention whose state is corrected towards each value,
+//   S <- g_t S;  u_t = beta_t (v_t - S^T k_t);  S <- S + k_t u_t^T;  o_t = S^T q_t,
+// behind short causal convolutions of q, k and v, with a norm per head and an output gate.
+//
+// The convolutions' inputs live in a ring of `taps` rows per slot, position p in row p mod taps, so a decode
+// step writes its own row while other CTAs still read the rows before it.
+//
+// Decode rows: one cluster per (head, row), a CTA per slice of the value columns. The state arrives in shared
+// memory while the step's products are still under way; convolution, unit norms, decay and step size are formed
+// by every CTA for itself; one pass over the state gives S^T k and S^T q, because o = g S^T q + (k . q) u; the squared
+// sums of the slices meet through distributed shared memory.
+//
+// Portions: convolution, gates and unit norms of all rows at once; then
+//   * a few rows, f32 sessions and unusual heads: one CTA per (head, value slice) walks the tokens, state in
+//     shared memory (delta_tokens_kernel);
+//   * otherwise chunks of 64 tokens. With b_t the decay from the chunk's start through t, the corrections of a chunk
+//     solve (I + A) u = beta v - beta b (K S_0), A_ts = beta_t b_t / b_s (k_t . k_s) for s < t. delta_chunk_kernel forms
+//     T = (I + A)^-1 by 16 x 16 blocks, U = T (beta v), W = T (beta b k) and P_ts = b_t / b_s (q_t . k_s) for every chunk at
+//     once; delta_scan_kernel walks the chunks: V = U - W S, o = b (Q S) + P V, S <- b_C S + (K b_C / b)^T V, a
+//     CTA per (head, 32 value columns), state in registers. All products with pairs of tf32 terms.
+// delta_finish_kernel applies norm and gate to a portion's rows.
+#include <cooperative_groups.h>
+
+#include <algorithm>
+
+#include "mixers.cuh"
+#include "tf32x3.cuh"
+
+namespace cg = cooperative_groups;
+
+namespace dyn {
+namespace {
+
+constexpr int DL_C = 64;        // tokens per chunk
+constexpr int DL_THREADS = 256;
+constexpr int DL_FEW = 16;      // portions up to this long walk their tokens
+
+__host__ __device__ inline int64_t channels_of(const DeltaArgs& a) {
+  return 2ll * a.kv_heads * a.dim + (int64_t)a.heads * a.vdim;
+}
+__device__ __forceinline__ float decay_log(const DeltaArgs& a, int h, float z) {
+  return -expf(vec_at(a.a_log, h)) * softplus_of(z + vec_at(a.dt, h));
+}
+__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async16(float* dst, const float* src, bool live) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src),
+               "r"(live ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// One head of q, k or v: where its inputs, weights and ring channels are. Slots 0 .. 2 kv_heads + heads - 1.
+struct HeadIn {
+  const float* x;   // row 0
+  int64_t ld, ch;   // floats between rows; first ring channel
+  Vec w;
+  int64_t w0;       // first channel of its weights
+  int n;
+};
+__device__ __forceinline__ HeadIn head_in(const DeltaArgs& a, int slot) {
+  HeadIn s;
+  const int G = a.kv_heads, part = slot < G ? 0 : slot < 2 * G ? 1 : 2, h = slot - part * G;
+  const Rows& r = part == 0 ? a.q : part == 1 ? a.k : a.v;
+  s.n = part < 2 ? a.dim : a.vdim;
+  s.w0 = (int64_t)h * s.n;
+  s.x = r.ptr + s.w0, s.ld = r.ld;
+  s.ch = (int64_t)min(part, 2) * G * a.dim + s.w0;
+  s.w = part == 0 ? a.conv_q : part == 1 ? a.conv_k : a.conv_v;
+  return s;
+}
+
+// silu(conv) of channel c of a head at position pos; x is the current input, earlier ones come from the slot's ring.
+__device__ __forceinline__ float conv_at(const DeltaArgs& a, const HeadIn& s, int c, float x, int64_t pos, const float* ring,
+                                         int64_t C) {
+  const int64_t w = (s.w0 + c) * a.taps;
+  float u = vec_at(s.w, w + a.taps - 1) * x;
+#pragma unroll 4
+  for (int j = 1; j < a.taps; j++)
+    if (pos >= j) u = fmaf(vec_at(s.w, w + a.taps - 1 - j), ring[((pos - j) % a.taps) * C + s.ch + c], u);
+  return silu_of(u);
+}
+
+__device__ __forceinline__ float block_total(float v, float* red) {  // red: 8 floats; all 256 threads
+  v = warp_sum(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; w++) t += red[w];
+  return t;
+}
+
+// One token of one (head, slice): S [D][per] in shared memory is updated, os[c] = o.
+// red: [2][8][per]; us: [per]. q and k final, kq = k . q.
+__device__ __forceinline__ void delta_token(float* S, int D, int per, int ne, const float* ks, const float* qs, const float* vs,
+                                            float g, float beta, float kq, float* red, float* us, float* os) {
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  for (int c = lane; c < ne; c += 32) {
+    float rk = 0.f, rq = 0.f;
+    for (int d = warp; d < D; d += 8) {
+      const float s = S[d * per + c];
+      rk = fmaf(s, ks[d], rk), rq = fmaf(s, qs[d], rq);
+    }
+    red[warp * per + c] = rk, red[(8 + warp) * per + c] = rq;
+  }
+  __syncthreads();
+  for (int c = tid; c < ne; c += DL_THREADS) {
+    float rk = 0.f, rq = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; w++) rk += red[w * per + c], rq += red[(8 + w) * per + c];
+    const float u = beta * (vs[c] - g * rk);
+    us[c] = u;
+    os[c] = fmaf(kq, u, g * rq);
+  }
+  __syncthreads();
+  for (int c = lane; c < ne; c += 32) {
+    const float u = us[c];
+    for (int d = warp; d < D; d += 8) S[d * per + c] = fmaf(g, S[d * per + c], ks[d] * u);
+  }
+}
+
+// ---- decode: independent rows ----------------------------------------------------------------
+__global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(DeltaArgs a, const int64_t* row_pos, const int64_t* row_seq,
+                                                                int64_t pos0, int64_t seq0, int64_t row0) {
+  extern __shared__ __align__(16) float dl_smem[];
+  __shared__ float part_ss, red8[8];
+  const cg::cluster_group cl = cg::this_cluster();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int D = a.dim, E = a.vdim, nsplit = gridDim.x, h = blockIdx.y;
+  const int64_t r = row0 + blockIdx.z, C = channels_of(a);
+  const int per = (E + nsplit - 1) / nsplit, e0 = min((int)blockIdx.x * per, E), ne = min(per, E - e0);
+  float* S = dl_smem;             // [D][per]
+  float* qs = S + D * per;        // [D]
+  float* ks = qs + D;             // [D]
+  float* vs = ks + D;             // [per]
+  float* us = vs + per;           // [per]
+  float* os = us + per;           // [per]
+  float* red = os + per;          // [2][8][per]
+  pdl_trigger();
+  const int64_t pos = row_pos ? row_pos[r] : pos0, seq = row_seq ? row_seq[r] : seq0;
+  // the state was written one token ago, with ordinary launches in between: it is fetched before the kernel waits
+  // for this token's products
+  float* Sg = a.state + ((seq * a.heads + h) * D) * (int64_t)E + e0;
+  for (int d = warp; d < D; d += 8)
+    for (int c = lane; c < ne; c += 32) {
+      if (pos > 0) cp_async4(S + d * per + c, Sg + (int64_t)d * E + c);
+      else S[d * per + c] = 0.f;
+    }
+  cp_commit();
+  pdl_wait();
+  const int j = h / (a.heads / a.kv_heads);
+  const HeadIn hq = head_in(a, j), hk = head_in(a, a.kv_heads + j), hv = head_in(a, 2 * a.kv_heads + h);
+  float* ring = a.ring + seq * (int64_t)a.taps * C;
+  const int64_t now = (pos % a.taps) * C;
+  const bool keeps = blockIdx.x == 0 && h % (a.heads / a.kv_heads) == 0;  // this CTA writes the head's ring rows
+  float sq = 0.f, sk = 0.f;
+  for (int c = tid; c < D; c += DL_THREADS) {
+    const float xq = hq.x[r * hq.ld + c], xk = hk.x[r * hk.ld + c];
+    const float q = conv_at(a, hq, c, xq, pos, ring, C), k = conv_at(a, hk, c, xk, pos, ring, C);
+    if (keeps) ring[now + hq.ch + c] = xq, ring[now + hk.ch + c] = xk;
+    qs[c] = q, ks[c] = k;
+    sq = fmaf(q, q, sq), sk = fmaf(k, k, sk);
+  }
+  for (int c = tid; c < ne; c += DL_THREADS) {
+    const float x = hv.x[r * hv.ld + e0 + c];
+    vs[c] = conv_at(a, hv, e0 + c, x, pos, ring, C);
+    ring[now + hv.ch + e0 + c] = x;
+  }
+  sq = block_total(sq, red8), sk = block_total(sk, red8);
+  const float iq = 1.0f / sqrtf(sq + a.unit_eps) * (1.0f / sqrtf((float)D)), ik = 1.0f / sqrtf(sk + a.unit_eps);
+  float kq = 0.f;
+  for (int c = tid; c < D; c += DL_THREADS) {
+    const float q = qs[c] * iq, k = ks[c] * ik;
+    qs[c] = q, ks[c] = k;
+    kq = fmaf(k, q, kq);
+  }
+  const float beta = sigmoid_of(a.b.ptr[r * a.b.ld + h]), g = expf(decay_log(a, h, a.a.ptr[r * a.a.ld + h]));
+  cp_wait<0>();
+  kq = block_total(kq, red8);  // also publishes q, k, v and the state
+  delta_token(S, D, per, ne, ks, qs, vs, g, beta, kq, red, us, os);
+  for (int c = lane; c < ne; c += 32)  // a thread's own elements
+    for (int d = warp; d < D; d += 8) Sg[(int64_t)d * E + c] = S[d * per + c];
+  float ss = 0.f;
+  for (int c = tid; c < ne; c += DL_THREADS) ss = fmaf(os[c], os[c], ss);
+  ss = block_total(ss, red8);
+  if (tid == 0) part_ss = ss;
+  cl.sync();
+  float total = 0.f;
+  for (int i = 0; i < nsplit; i++) total += *cl.map_shared_rank(&part_ss, i);
+  cl.sync();  // nobody leaves while another CTA still reads its sum
+  const float inv = 1.0f / sqrtf(total / (float)E + a.eps);
+  const float* gate = a.g.ptr + r * a.g.ld + (int64_t)h * E + e0;
+  float* out = a.out + r * (int64_t)a.heads * E + (int64_t)h * E + e0;
+  for (int c = tid; c < ne; c += DL_THREADS) out[c] = os[c] * inv * vec_at(a.norm, e0 + c) * silu_of(gate[c]);
+}
+
+constexpr int DL_MAX_SMEM = 200 * 1024;
+
+int step_rows(const DeltaArgs& a, const int64_t* pos, const int64_t* seq, int64_t pos0, int64_t seq0, int64_t rows,
+              cudaStream_t st) {
+  int nsplit = 1;
+  while (nsplit < 8 && (a.vdim + nsplit - 1) / nsplit > 32) nsplit *= 2;
+  const int per = (a.vdim + nsplit - 1) / nsplit;
+  const size_t smem = ((size_t)a.dim * per + 2 * a.dim + 19 * per) * 4;
+  DYN_CHECK(smem <= DL_MAX_SMEM, "delta rule: head of %d x %d is too large", a.dim, a.vdim);
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(delta_step_kernel), DL_MAX_SMEM)) return 1;
+  for (int64_t r0 = 0; r0 < rows; r0 += 65535) {
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = dim3((unsigned)nsplit, (unsigned)a.heads, (unsigned)std::min<int64_t>(65535, rows - r0));
+    cfg.blockDim = dim3(DL_THREADS);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[2] = {};
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = (unsigned)nsplit, attr[0].val.clusterDim.y = 1, attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr, cfg.numAttrs = pos && pdl_enabled() ? 2 : 1;
+    DYN_CUDA(cudaLaunchKernelEx(&cfg, delta_step_kernel, a, pos, seq, pos0, seq0, r0));
+    count_launch();
+  }
+  return 0;
+}
+
+// ---- portions ---------------------------------------------------------------------------------
+// Scratch of a portion: convolved rows [rows][q | k | v], gates [rows][beta | log g], then the chunks' W, U, P.
+struct DeltaScratch {
+  float *cv, *gates, *w, *u, *p;
+};
+__host__ __device__ inline DeltaScratch carve(const DeltaArgs& a, int64_t rows) {
+  const int64_t nc = (rows + DL_C - 1) / DL_C, ch = nc * a.heads;
+  DeltaScratch s;
+  s.cv = a.scratch;
+  s.gates = s.cv + (rows * channels_of(a) + 3) / 4 * 4;
+  s.w = s.gates + (rows * 2 * a.heads + 3) / 4 * 4;
+  s.u = s.w + ch * DL_C * ((a.dim + 3) / 4 * 4);
+  s.p = s.u + ch * DL_C * ((a.vdim + 3) / 4 * 4);
+  return s;
+}
+
+constexpr int DV_ROWS = 8;  // consecutive rows a warp convolves
+// Warp = (eight rows, one head of q, k or v). TAPS: compile-time window (taps <= TAPS), 0: any.
+template <int TAPS>
+__global__ void __launch_bounds__(DL_THREADS) delta_conv_kernel(DeltaArgs a, int64_t rows, int64_t base, int64_t slot) {
+  const DeltaScratch sc = carve(a, rows);
+  const int lane = threadIdx.x & 31;
+  const int slots = 2 * a.kv_heads + a.heads;
+  const int64_t item = blockIdx.x * 8ll + (threadIdx.x >> 5), groups = (rows + DV_ROWS - 1) / DV_ROWS;
+  if (item >= groups * slots) return;
+  const int s = (int)(item % slots);
+  const int64_t r0 = item / slots * DV_ROWS, C = channels_of(a);
+  const HeadIn in = head_in(a, s);
+  const float* ring = a.ring + slot * (int64_t)a.taps * C;
+  const int live = (int)min((int64_t)DV_ROWS, rows - r0);
+  const bool unit = s < 2 * a.kv_heads;
+  float ss[DV_ROWS] = {};
+  for (int c = lane; c < in.n; c += 32) {
+    auto input = [&](int64_t row) -> float {  // row < 0: before the portion
+      if (row >= 0) return in.x[row * in.ld + c];
+      const int64_t p = base + row;
+      return p >= 0 ? ring[(p % a.taps) * C + in.ch + c] : 0.f;
+    };
+    float* out = sc.cv + r0 * C + in.ch + c;
+    if constexpr (TAPS > 0) {
+      float w[TAPS], x[TAPS + DV_ROWS - 1];
+#pragma unroll
+      for (int t = 0; t < TAPS; t++) w[t] = t >= TAPS - a.taps ? vec_at(in.w, (in.w0 + c) * a.taps + t - (TAPS - a.taps)) : 0.f;
+#pragma unroll
+      for (int t = 0; t < TAPS + DV_ROWS - 1; t++) {
+        const int64_t row = r0 + t - (TAPS - 1);
+        x[t] = t >= TAPS - a.taps && row < rows ? input(row) : 0.f;
+      }
+#pragma unroll
+      for (int i = 0; i < DV_ROWS; i++) {
+        if (i < live) {
+          float u = w[TAPS - 1] * x[i + TAPS - 1];
+#pragma unroll
+          for (int j = 1; j < TAPS; j++) u = fmaf(w[TAPS - 1 - j], x[i + TAPS - 1 - j], u);
+          u = silu_of(u);
+          out[i * C] = u;
+          ss[i] = fmaf(u, u, ss[i]);
+        }
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < DV_ROWS; i++) {
+        if (i < live) {
+          float u = 0.f;
+          for (int j = 0; j < a.taps; j++) u = fmaf(vec_at(in.w, (in.w0 + c) * a.taps + a.taps - 1 - j), input(r0 + i - j), u);
+          u = silu_of(u);
+          out[i * C] = u;
+          ss[i] = fmaf(u, u, ss[i]);
+        }
+      }
+    }
+  }
+  if (unit) {
+    const float extra = s < a.kv_heads ? 1.0f / sqrtf((float)a.dim) : 1.0f;
+#pragma unroll
+    for (int i = 0; i < DV_ROWS; i++) ss[i] = 1.0f / sqrtf(warp_sum(ss[i]) + a.unit_eps) * extra;
+    for (int c = lane; c < in.n; c += 32) {  // the lane's own elements
+      float* out = sc.cv + r0 * C + in.ch + c;
+#pragma unroll
+      for (int i = 0; i < DV_ROWS; i++)
+        if (i < live) out[i * C] *= ss[i];
+    }
+  } else if (lane < live) {
+    const int h = s - 2 * a.kv_heads;
+    const int64_t r = r0 + lane;
+    sc.gates[r * 2 * a.heads + h] = sigmoid_of(a.b.ptr[r * a.b.ld + h]);
+    sc.gates[r * 2 * a.heads + a.heads + h] = decay_log(a, h, a.a.ptr[r * a.a.ld + h]);
+  }
+}
+
+// The ring after the portion; a launch after the convolutions' (they read the rows before it).
+__device__ __forceinline__ void keep_inputs(const DeltaArgs& a, int64_t rows, int64_t base, int64_t slot, int block, int blocks) {
+  const int64_t C = channels_of(a), qk = (int64_t)a.kv_heads * a.dim, from = max((int64_t)0, rows - a.taps);
+  float* ring = a.ring + slot * (int64_t)a.taps * C;
+  const int64_t total = (rows - from) * C;
+  for (int64_t i = block * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)blocks * blockDim.x) {
+    const int64_t row = from + i / C, c = i % C;
+    const float x = c < qk ? a.q.ptr[row * a.q.ld + c] : c < 2 * qk ? a.k.ptr[row * a.k.ld + c - qk] : a.v.ptr[row * a.v.ld + c - 2 * qk];
+    ring[((base + row) % a.taps) * C + c] = x;
+  }
+}
+
+// Token by token: CTA = (value slice, head). Leaves o without norm and gate in a.out.
+__global__ void __launch_bounds__(DL_THREADS) delta_tokens_kernel(DeltaArgs a, int64_t rows, int64_t base, int64_t slot) {
+  extern __shared__ __align__(16) float dt_smem[];
+  const DeltaScratch sc = carve(a, rows);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int D = a.dim, E = a.vdim, h = blockIdx.y, j = h / (a.heads / a.kv_heads);
+  const int per = (E + gridDim.x - 1) / gridDim.x, e0 = min((int)blockIdx.x * per, E), ne = min(per, E - e0);
+  const int64_t C = channels_of(a), qk = (int64_t)a.kv_heads * D;
+  float* S = dt_smem;              // [D][per]
+  float* qs = S + D * per;         // [D]
+  float* ks = qs + D;              // [D]
+  float* vs = ks + D;              // [per]
+  float* us = vs + per;            // [per]
+  float* os = us + per;            // [per]
+  float* red = os + per;           // [2][8][per]
+  __shared__ float red8[8];
+  keep_inputs(a, rows, base, slot, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
+  float* Sg = a.state + ((slot * a.heads + h) * D) * (int64_t)E + e0;
+  for (int d = warp; d < D; d += 8)
+    for (int c = lane; c < ne; c += 32) S[d * per + c] = base > 0 ? Sg[(int64_t)d * E + c] : 0.f;
+  for (int64_t t = 0; t < rows; t++) {
+    const float* cv = sc.cv + t * C;
+    float kq = 0.f;
+    for (int d = tid; d < D; d += DL_THREADS) {
+      const float q = cv[(int64_t)j * D + d], k = cv[qk + (int64_t)j * D + d];
+      qs[d] = q, ks[d] = k;
+      kq = fmaf(k, q, kq);
+    }
+    for (int c = tid; c < ne; c += DL_THREADS) vs[c] = cv[2 * qk + (int64_t)h * E + e0 + c];
+    const float beta = sc.gates[t * 2 * a.heads + h], g = expf(sc.gates[t * 2 * a.heads + a.heads + h]);
+    kq = block_total(kq, red8);
+    delta_token(S, D, per, ne, ks, qs, vs, g, beta, kq, red, us, os);
+    for (int c = tid; c < ne; c += DL_THREADS) a.out[t * (int64_t)a.heads * E + (int64_t)h * E + e0 + c] = os[c];
+    __syncthreads();  // the token's vectors are read
+  }
+  for (int d = warp; d < D; d += 8)
+    for (int c = lane; c < ne; c += 32) Sg[(int64_t)d * E + c] = S[d * per + c];
+}
+
+// rows x cols floats (16-byte aligned, cols % 4 == 0) into shared memory, zeros up to fill_rows x fill_cols
+__device__ __forceinline__ void stage(float* dst, int pitch, const float* src, int64_t ld, int rows, int cols, int fill_rows,
+                                      int fill_cols) {
+  const int q = fill_cols / 4;
+  for (int i = threadIdx.x; i < fill_rows * q; i += DL_THREADS) {
+    const int r = i / q, c = (i - r * q) * 4;
+    const bool live = r < rows && c < cols;
+    cp_async16(dst + r * pitch + c, live ? src + r * ld + c : src, live);
+  }
+}
+__device__ __forceinline__ void load_a(AFrag& f, const float* p, int pitch) {  // rows g, g + 8; columns t4, t4 + 4
+  split_into(f, 0, p[0]), split_into(f, 1, p[8 * pitch]), split_into(f, 2, p[4]), split_into(f, 3, p[8 * pitch + 4]);
+}
+
+// Decays of a chunk: lane 0 .. 31 of one warp, two tokens each. Gd[t] = sum of log g through t.
+__device__ __forceinline__ void chunk_decay(const DeltaArgs& a, const float* gates, int64_t t0, int n, int h, double* Gd, float* beta) {
+  const int lane = threadIdx.x & 31;
+  double v[2];
+#pragma unroll
+  for (int i = 0; i < 2; i++) {
+    const int t = 2 * lane + i;
+    v[i] = t < n ? (double)gates[(t0 + t) * 2 * a.heads + a.heads + h] : 0.0;
+    if (beta) beta[t] = t < n ? gates[(t0 + t) * 2 * a.heads + h] : 0.f;
+  }
+  double s = v[0] + v[1];
+#pragma unroll
+  for (int o = 1; o < 32; o *= 2) {
+    const double other = __shfl_up_sync(0xffffffffu, s, o);
+    if (lane >= o) s += other;
+  }
+  Gd[2 * lane] = s - v[1], Gd[2 * lane + 1] = s;
+}
+
+constexpr int DC_D = 128;                   // widest q/k head of the chunk kernels
+constexpr int DC_P = DC_D + 4, DC_S = DL_C + 4;
+constexpr int DC_SMEM = (2 * DL_C * DC_P + 2 * DL_C * DC_S) * 4 + DL_C * 8 + DL_C * 4;
+
+// W, U and P of one (chunk, head).
+__global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(DeltaArgs a, int64_t rows) {
+  extern __shared__ __align__(16) float dc_smem[];
+  const DeltaScratch sc = carve(a, rows);
+  float* ks = dc_smem;                 // [t][DC_P]
+  float* qs = ks + DL_C * DC_P;        // [t][DC_P]; then blocks of v
+  float* A = qs + DL_C * DC_P;         // [t][DC_S]
+  float* T = A + DL_C * DC_S;          // [t][DC_S]
+  double* Gd = reinterpret_cast<double*>(T + DL_C * DC_S);
+  float* beta = reinterpret_cast<float*>(Gd + DL_C);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
+  const int D = a.dim, E = a.vdim, h = blockIdx.y, j = h / (a.heads / a.kv_heads);
+  const int64_t c = blockIdx.x, t0 = c * DL_C, C = channels_of(a), qk = (int64_t)a.kv_heads * D;
+  const int n = (int)min((int64_t)DL_C, rows - t0);
+  const float* cv = sc.cv + t0 * C;
+  stage(ks, DC_P, cv + qk + (int64_t)j * D, C, n, D, DL_C, D);
+  stage(qs, DC_P, cv + (int64_t)j * D, C, n, D, DL_C, D);
+  cp_commit();
+  if (warp == 0) chunk_decay(a, sc.gates, t0, n, h, Gd, beta);
+  cp_wait<0>();
+  __syncthreads();
+  const int mt = warp & 3, nh = warp >> 2;   // 16 tokens x half of the keys (or of the columns)
+  {
+    float s[4][4] = {}, p[4][4] = {};
+#pragma unroll 2
+    for (int d = 0; d < D; d += 8) {
+      AFrag fk, fq;
+      load_a(fk, ks + (16 * mt + g) * DC_P + d + t4, DC_P);
+      load_a(fq, qs + (16 * mt + g) * DC_P + d + t4, DC_P);
+      Tf32Pair b0[4], b1[4];
+#pragma unroll
+      for (int nt = 0; nt < 4; nt++) {
+        const float* b = ks + (nh * 32 + 8 * nt + g) * DC_P + d + t4;
+        b0[nt] = tf32_split(b[0]), b1[nt] = tf32_split(b[4]);
+      }
+      mma3_split<4>(s, fk, b0, b1);
+      mma3_split<4>(p, fq, b0, b1);
+    }
+    float* P = sc.p + (c * a.heads + h) * DL_C * DL_C;
+#pragma unroll
+    for (int nt = 0; nt < 4; nt++)
+#pragma unroll
+      for (int i = 0; i < 2; i++) {
+        const int t = 16 * mt + g + 8 * i, u = nh * 32 + 8 * nt + 2 * t4;
+        float2 pv;
+        float av[2];
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+          const float w = u + e <= t ? expf((float)(Gd[t] - Gd[u + e])) : 0.f;
+          (e ? pv.y : pv.x) = p[nt][2 * i + e] * w;
+          av[e] = u + e < t ? beta[t] * w * s[nt][2 * i + e] : 0.f;
+        }
+        A[t * DC_S + u] = av[0], A[t * DC_S + u + 1] = av[1];
+        *reinterpret_cast<float2*>(P + t * DL_C + u) = pv;
+      }
+  }
+  __syncthreads();
+  // ---- T = (I + A)^-1. Diagonal blocks by forward substitution, thread = (block, column); qs is free
+  for (int i = tid; i < DL_C * DC_S; i += DL_THREADS) T[i] = 0.f;
+  __syncthreads();
+  if (tid < DL_C) {
+    const int b = tid & ~15, col = tid & 15;
+    float x[16];
+#pragma unroll
+    for (int i = 0; i < 16; i++) {
+      float v = i == col ? 1.f : 0.f;
+#pragma unroll
+      for (int k = 0; k < 16; k++)
+        if (k < i) v = fmaf(-A[(b + i) * DC_S + b + k], x[k], v);
+      x[i] = i >= col ? v : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < 16; i++) T[(b + i) * DC_S + b + col] = x[i];
+  }
+  __syncthreads();
+  // blocks below: T_ij = -T_ii sum_{k = j .. i-1} A_ik T_kj, one block diagonal after the other
+  {
+    float* M = qs;  // [block][16][17]
+    const int rr = (tid >> 4) & 15, cc = tid & 15;
+    for (int dist = 1; dist < 4; dist++) {
+      for (int jb = 0; jb + dist < 4; jb++) {
+        const int ib = jb + dist;
+        float v = 0.f;
+        for (int k = jb * 16; k < ib * 16; k++) v = fmaf(A[(ib * 16 + rr) * DC_S + k], T[k * DC_S + jb * 16 + cc], v);
+        M[jb * 272 + rr * 17 + cc] = v;
+      }
+      __syncthreads();
+      for (int jb = 0; jb + dist < 4; jb++) {
+        const int ib = jb + dist;
+        float v = 0.f;
+#pragma unroll
+        for (int k = 0; k < 16; k++) v = fmaf(-T[(ib * 16 + rr) * DC_S + ib * 16 + k], M[jb * 272 + k * 17 + cc], v);
+        T[(ib * 16 + rr) * DC_S + jb * 16 + cc] = v;
+      }
+      __syncthreads();
+    }
+  }
+  // ---- U = T (beta v), W = T (beta b k): 64 rows x up to 128 columns at a time, a warp 16 rows x half of them
+  auto product = [&](const float* B, int cols, bool decay, float* out, int64_t ld) {
+    float acc[8][4] = {};
+    for (int k = 0; k < 16 * (mt + 1); k += 8) {  // T is lower triangular
+      AFrag f;
+      load_a(f, T + (16 * mt + g) * DC_S + k + t4, DC_S);
+      const int ka = k + t4, kb = ka + 4;
+      const float wa = decay ? beta[ka] * expf((float)Gd[ka]) : beta[ka], wb = decay ? beta[kb] * expf((float)Gd[kb]) : beta[kb];
+      mma3<8>(acc, f, [&](int nt, int half) {
+        const int col = nh * 64 + 8 * nt + g;
+        return col < cols ? (half ? wb * B[kb * DC_P + col] : wa * B[ka * DC_P + col]) : 0.f;
+      });
+    }
+#pragma unroll
+    for (int nt = 0; nt < 8; nt++) {
+      const int col = nh * 64 + 8 * nt + 2 * t4;
+      if (col >= cols) continue;
+#pragma unroll
+      for (int i = 0; i < 2; i++)
+        *reinterpret_cast<float2*>(out + (16 * mt + g + 8 * i) * ld + col) = make_float2(acc[nt][2 * i], acc[nt][2 * i + 1]);
+    }
+  };
+  for (int e0 = 0; e0 < E; e0 += DC_D) {
+    const int cols = min(DC_D, E - e0);
+    if (e0) __syncthreads();
+    stage(qs, DC_P, cv + 2 * qk + (int64_t)h * E + e0, C, n, cols, DL_C, cols);
+    cp_commit();
+    if (e0 == 0) product(ks, D, true, sc.w + (c * a.heads + h) * DL_C * (int64_t)D, D);
+    cp_wait<0>();
+    __syncthreads();
+    product(qs, cols, false, sc.u + (c * a.heads + h) * DL_C * (int64_t)E + e0, E);
+  }
+}
+
+constexpr int DS_N = 32;                       // value columns per CTA
+constexpr int DS_B = DS_N + 8;                 // pitch of the split operands: conflict-free B fragments
+constexpr int DS_KP = DC_D + 8;
+constexpr int DS_SMEM = (2 * DL_C * DC_P + DL_C * DS_KP + DL_C * DC_S + 2 * DC_D * DS_B + 2 * DL_C * DS_B) * 4 + DL_C * 8;
+
+// The walk over the chunks for one (value slice, head).
+__global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs a, int64_t rows, int64_t base, int64_t slot) {
+  extern __shared__ __align__(16) float ds_smem[];
+  const DeltaScratch sc = carve(a, rows);
+  float* Ws = ds_smem;                    // [t][DC_P]
+  float* Qs = Ws + DL_C * DC_P;           // [t][DC_P]
+  float* Ks = Qs + DL_C * DC_P;           // [t][DS_KP]
+  float* Ps = Ks + DL_C * DS_KP;          // [t][DC_S]
+  float* Sh = Ps + DL_C * DC_S;           // [d][DS_B] tf32 terms of the state
+  float* Sl = Sh + DC_D * DS_B;
+  float* Vh = Sl + DC_D * DS_B;           // [t][DS_B] of the corrections
+  float* Vl = Vh + DL_C * DS_B;
+  double* Gd = reinterpret_cast<double*>(Vl + DL_C * DS_B);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
+  const int D = a.dim, E = a.vdim, h = blockIdx.y, j = h / (a.heads / a.kv_heads), e0 = blockIdx.x * DS_N;
+  const int64_t C = channels_of(a), qk = (int64_t)a.kv_heads * D, nc = (rows + DL_C - 1) / DL_C;
+  keep_inputs(a, rows, base, slot, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
+  float* Sg = a.state + ((slot * a.heads + h) * D) * (int64_t)E + e0;
+  auto stage_wq = [&](int64_t c) {
+    const int n = (int)min((int64_t)DL_C, rows - c * DL_C);
+    stage(Ws, DC_P, sc.w + (c * a.heads + h) * DL_C * (int64_t)D, D, DL_C, D, DL_C, D);
+    stage(Qs, DC_P, sc.cv + c * DL_C * C + (int64_t)j * D, C, n, D, DL_C, D);
+    cp_commit();
+  };
+  auto stage_kp = [&](int64_t c) {
+    const int n = (int)min((int64_t)DL_C, rows - c * DL_C);
+    stage(Ks, DS_KP, sc.cv + c * DL_C * C + qk + (int64_t)j * D, C, n, D, DL_C, D);
+    stage(Ps, DC_S, sc.p + (c * a.heads + h) * DL_C * DL_C, DL_C, DL_C, DL_C, DL_C, DL_C);
+    cp_commit();
+  };
+  stage_wq(0);
+  stage_kp(0);
+  // the warp's 16 rows of the state, as accumulators
+  const int d0 = 16 * warp;
+  float S[4][4];
+#pragma unroll
+  for (int nt = 0; nt < 4; nt++)
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      const int d = d0 + g + 8 * (i >> 1), e = 8 * nt + 2 * t4 + (i & 1);
+      S[nt][i] = base > 0 && d < D && e0 + e < E ? Sg[(int64_t)d * E + e] : 0.f;
+    }
+  const int mt = warp & 3, nh = warp >> 2;  // 16 tokens x 16 value columns
+  for (int64_t c = 0; c < nc; c++) {
+    const int64_t t0 = c * DL_C;
+    const int n = (int)min((int64_t)DL_C, rows - t0);
+    if (d0 < D) {
+#pragma unroll
+      for (int nt = 0; nt < 4; nt++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+          const int d = d0 + g + 8 * (i >> 1), e = 8 * nt + 2 * t4 + (i & 1);
+          const Tf32Pair p = tf32_split(S[nt][i]);
+          Sh[d * DS_B + e] = __uint_as_float(p.hi), Sl[d * DS_B + e] = __uint_as_float(p.lo);
+        }
+    }
+    if (warp == 0) chunk_decay(a, sc.gates, t0, n, h, Gd, nullptr);
+    // U of the warp's tile, on its way while W and Q arrive
+    float uv[2][4];
+    const float* U = sc.u + (c * a.heads + h) * DL_C * (int64_t)E + e0;
+#pragma unroll
+    for (int nt = 0; nt < 2; nt++)
+#pragma unroll
+      for (int i = 0; i < 2; i++) {
+        const int t = 16 * mt + g + 8 * i, e = nh * 16 + 8 * nt + 2 * t4;
+        const float2 v = e0 + e < E ? *reinterpret_cast<const float2*>(U + t * (int64_t)E + e) : make_float2(0.f, 0.f);
+        uv[nt][2 * i] = v.x, uv[nt][2 * i + 1] = v.y;
+      }
+    cp_wait<1>();
+    __syncthreads();
+    // ---- W S and Q S
+    float ws[2][4] = {}, o[2][4] = {};
+#pragma unroll 2
+    for (int d = 0; d < D; d += 8) {
+      AFrag fw, fq;
+      load_a(fw, Ws + (16 * mt + g) * DC_P + d + t4, DC_P);
+      load_a(fq, Qs + (16 * mt + g) * DC_P + d + t4, DC_P);
+      Tf32Pair b0[2], b1[2];
+#pragma unroll
+      for (int nt = 0; nt < 2; nt++) {
+        const int at = (d + t4) * DS_B + nh * 16 + 8 * nt + g;
+        b0[nt].hi = __float_as_uint(Sh[at]), b0[nt].lo = __float_as_uint(Sl[at]);
+        b1[nt].hi = __float_as_uint(Sh[at + 4 * DS_B]), b1[nt].lo = __float_as_uint(Sl[at + 4 * DS_B]);
+      }
+      mma3_split<2>(ws, fw, b0, b1);
+      mma3_split<2>(o, fq, b0, b1);
+    }
+    const float w0 = expf((float)Gd[16 * mt + g]), w1 = expf((float)Gd[16 * mt + g + 8]);
+#pragma unroll
+    for (int nt = 0; nt < 2; nt++)
+#pragma unroll
+      for (int i = 0; i < 4; i++) {
+        const int t = 16 * mt + g + 8 * (i >> 1), e = nh * 16 + 8 * nt + 2 * t4 + (i & 1);
+        const Tf32Pair p = tf32_split(uv[nt][i] - ws[nt][i]);
+        Vh[t * DS_B + e] = __uint_as_float(p.hi), Vl[t * DS_B + e] = __uint_as_float(p.lo);
+        o[nt][i] *= i < 2 ? w0 : w1;
+      }
+    cp_wait<0>();
+    __syncthreads();  // V, K and P are there; W and Q are read
+    if (c + 1 < nc) stage_wq(c + 1);
+    auto v_pair = [&](Tf32Pair& b0, Tf32Pair& b1, int k, int col) {
+      const int at = (k + t4) * DS_B + col;
+      b0.hi = __float_as_uint(Vh[at]), b0.lo = __float_as_uint(Vl[at]);
+      b1.hi = __float_as_uint(Vh[at + 4 * DS_B]), b1.lo = __float_as_uint(Vl[at + 4 * DS_B]);
+    };
+    // ---- o += P V (P is lower triangular)
+    for (int k = 0; k < 16 * (mt + 1); k += 8) {
+      AFrag f;
+      load_a(f, Ps + (16 * mt + g) * DC_S + k + t4, DC_S);
+      Tf32Pair b0[2], b1[2];
+#pragma unroll
+      for (int nt = 0; nt < 2; nt++) v_pair(b0[nt], b1[nt], k, nh * 16 + 8 * nt + g);
+      mma3_split<2>(o, f, b0, b1);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+      const int t = 16 * mt + g + 8 * i;
+      if (t >= n) continue;
+      float* out = a.out + (t0 + t) * (int64_t)a.heads * E + (int64_t)h * E + e0;
+#pragma unroll
+      for (int nt = 0; nt < 2; nt++) {
+        const int e = nh * 16 + 8 * nt + 2 * t4;
+        if (e0 + e < E) *reinterpret_cast<float2*>(out + e) = make_float2(o[nt][2 * i], o[nt][2 * i + 1]);
+      }
+    }
+    // ---- S <- b_C S + (K b_C / b)^T V
+    if (d0 < D) {
+      const double last = Gd[DL_C - 1];
+      const float full = expf((float)last);
+#pragma unroll
+      for (int nt = 0; nt < 4; nt++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) S[nt][i] *= full;
+#pragma unroll 2
+      for (int k = 0; k < DL_C; k += 8) {
+        const float wa = expf((float)(last - Gd[k + t4])), wb = expf((float)(last - Gd[k + t4 + 4]));
+        const float *ka = Ks + (k + t4) * DS_KP + d0 + g, *kb = ka + 4 * DS_KP;
+        const bool second = d0 + 8 < D;
+        AFrag f;
+        split_into(f, 0, ka[0] * wa), split_into(f, 1, second ? ka[8] * wa : 0.f);
+        split_into(f, 2, kb[0] * wb), split_into(f, 3, second ? kb[8] * wb : 0.f);
+        Tf32Pair b0[4], b1[4];
+#pragma unroll
+        for (int nt = 0; nt < 4; nt++) v_pair(b0[nt], b1[nt], k, 8 * nt + g);
+        mma3_split<4>(S, f, b0, b1);
+      }
+    }
+    __syncthreads();  // K, P, V and the decays are read
+    if (c + 1 < nc) stage_kp(c + 1);
+  }
+#pragma unroll
+  for (int nt = 0; nt < 4; nt++)
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      const int d = d0 + g + 8 * (i >> 1), e = 8 * nt + 2 * t4 + (i & 1);
+      if (d < D && e0 + e < E) Sg[(int64_t)d * E + e] = S[nt][i];
+    }
+}
+
+// Norm and gate of a portion's rows, in place: warp = (row, head).
+__global__ void __launch_bounds__(DL_THREADS) delta_finish_kernel(DeltaArgs a, int64_t rows) {
+  const int lane = threadIdx.x & 31, E = a.vdim;
+  const int64_t item = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  if (item >= rows * a.heads) return;
+  const int64_t r = item / a.heads, h = item % a.heads;
+  float* out = a.out + item * E;
+  const float* gate = a.g.ptr + r * a.g.ld + h * E;
+  float ss = 0.f;
+  for (int e = lane; e < E; e += 32) ss = fmaf(out[e], out[e], ss);
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)E + a.eps);
+  for (int e = lane; e < E; e += 32) out[e] = out[e] * inv * vec_at(a.norm, e) * silu_of(gate[e]);
+}
+
+bool chunk_shape(const DeltaArgs& a, int64_t rows) {
+  return !a.exact && rows > DL_FEW && a.dim <= DC_D && a.dim % 8 == 0 && a.vdim % 8 == 0;
+}
+
+}  // namespace
+
+size_t delta_scratch_floats(const DeltaArgs& a, int64_t rows) {
+  DeltaArgs z = a;
+  z.scratch = nullptr;
+  const int64_t nc = (rows + DL_C - 1) / DL_C;
+  const size_t small = carve(z, rows).w - z.scratch;
+  return chunk_shape(a, rows) ? (size_t)(carve(z, rows).p - z.scratch) + (size_t)nc * a.heads * DL_C * DL_C : small;
+}
+
+int launch_delta(const DeltaArgs& a, const StepRows& r, cudaStream_t st) {
+  if (r.rows == 0) return 0;
+  DYN_CHECK(a.kv_heads > 0 && a.heads % a.kv_heads == 0, "delta rule: %d heads over %d q/k heads", a.heads, a.kv_heads);
+  if (r.base < 0) return step_rows(a, r.pos, r.seq, 0, 0, r.rows, st);
+  if (r.rows == 1) return step_rows(a, nullptr, nullptr, r.base, r.slot, 1, st);
+  const int64_t items = (r.rows + DV_ROWS - 1) / DV_ROWS * (2 * a.kv_heads + a.heads);
+  const unsigned grid = (unsigned)((items + 7) / 8);
+  if (a.taps <= 4) delta_conv_kernel<4><<<grid, DL_THREADS, 0, st>>>(a, r.rows, r.base, r.slot);
+  else delta_conv_kernel<0><<<grid, DL_THREADS, 0, st>>>(a, r.rows, r.base, r.slot);
+  if (chunk_shape(a, r.rows)) {
+    const unsigned nc = (unsigned)((r.rows + DL_C - 1) / DL_C);
+    if (ensure_dynamic_smem(reinterpret_cast<const void*>(delta_chunk_kernel), DC_SMEM) ||
+        ensure_dynamic_smem(reinterpret_cast<const void*>(delta_scan_kernel), DS_SMEM))
+      return 1;
+    delta_chunk_kernel<<<dim3(nc, (unsigned)a.heads), DL_THREADS, DC_SMEM, st>>>(a, r.rows);
+    delta_scan_kernel<<<dim3((unsigned)((a.vdim + DS_N - 1) / DS_N), (unsigned)a.heads), DL_THREADS, DS_SMEM, st>>>(
+        a, r.rows, r.base, r.slot);
+    count_launch(2);
+  } else {
+    int nsplit = std::max(1, (a.vdim + 31) / 32);
+    const int per = (a.vdim + nsplit - 1) / nsplit;
+    const size_t smem = ((size_t)a.dim * per + 2 * a.dim + 19 * per) * 4;
+    DYN_CHECK(smem <= DL_MAX_SMEM, "delta rule: head of %d x %d is too large", a.dim, a.vdim);
+    if (ensure_dynamic_smem(reinterpret_cast<const void*>(delta_tokens_kernel), DL_MAX_SMEM)) return 1;
+    delta_tokens_kernel<<<dim3((unsigned)nsplit, (unsigned)a.heads), DL_THREADS, smem, st>>>(a, r.rows, r.base, r.slot);
+    count_launch();
+  }
+  delta_finish_kernel<<<(unsigned)((r.rows * a.heads + 7) / 8), DL_THREADS, 0, st>>>(a, r.rows);
+  count_launch(2);
+  DYN_CUDA(cudaGetLastError());
+  return 0;
+}
+
+}  // namespace dyn

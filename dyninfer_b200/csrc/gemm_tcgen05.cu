@@ -158,6 +158,9 @@ struct TgArgs {
   // chunks [z * nk_split, ...) and writes its scaled sums to partial[z][M][N]; a second pass adds them
   int nk_split;      // chunks per split (all of them when gridDim.z == 1)
   float* partial;
+  // grouped form (plain 16-bit weights): blockIdx.y names a tile (matrix, first row, rows); 0 rows: nothing to do
+  const int4* tiles;
+  const uint8_t* const* bases;
 };
 
 // Items of one row in a K chunk: every item is one decoder part; its groups that fall inside the
@@ -238,7 +241,16 @@ dqgemm_tc_kernel(const TgArgs a, const __grid_constant__ CUtensorMap xmap) {
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int bn = a.bn;
   const int64_t N = a.w.rows, K = a.w.cols;
-  const int64_t n0 = (int64_t)blockIdx.x * TG_BM, m0 = (int64_t)blockIdx.y * bn;
+  const int64_t n0 = (int64_t)blockIdx.x * TG_BM;
+  int64_t m0 = (int64_t)blockIdx.y * bn, mend = a.M;  // activation rows [m0, mend) at most
+  const uint8_t* wdata = a.w.data;
+  if constexpr (tg_plain16(ENC)) {
+    if (a.tiles) {
+      const int4 t = a.tiles[blockIdx.y];
+      if (t.z == 0) return;
+      m0 = t.y, mend = m0 + t.z, wdata = a.bases[t.x];
+    }
+  }
   const int kbase = (int)blockIdx.z * a.nk_split;  // first chunk of this CTA's share of K
   const int nk = min(a.nk_split, (int)(K / TG_BK) - kbase);
   constexpr bool AT = tg_a_in_tmem(ENC);
@@ -377,7 +389,7 @@ dqgemm_tc_kernel(const TgArgs a, const __grid_constant__ CUtensorMap xmap) {
       const int64_t last = N - 1 - (n0 + quarter * 32);  // rows past the matrix repeat its last row (never stored)
       const int rsub = lane >> 2, piece = lane & 3;
       auto fetch = [&](int kc, int sub, uint32_t (&q)[16]) {
-        const uint8_t* cb = a.w.data + ((int64_t)(kbase + kc) * TG_BK + sub * 32) * 2 + piece * 16;
+        const uint8_t* cb = wdata + ((int64_t)(kbase + kc) * TG_BK + sub * 32) * 2 + piece * 16;
 #pragma unroll
         for (int it = 0; it < 4; it++) {
           const int r = it * 8 + rsub;
@@ -710,7 +722,7 @@ dqgemm_tc_kernel(const TgArgs a, const __grid_constant__ CUtensorMap xmap) {
   // before its first store (y may be the residual's own buffer).
   {
     __syncwarp();  // the issuing lanes of the MMA and copy warps rejoin here
-    for (int j = tid; j < bn; j += TG_THREADS) s_inv[j] = m0 + j < a.M ? __ldg(a.inv_s + m0 + j) : 0.f;
+    for (int j = tid; j < bn; j += TG_THREADS) s_inv[j] = m0 + j < mend ? __ldg(a.inv_s + m0 + j) : 0.f;
     __syncthreads();
     const bool ok = mbar_wait_bounded(&accum_bar, 0, TG_SPINS, &s_abort);
     if (!ok && !s_abort) s_abort = 3;
@@ -722,7 +734,7 @@ dqgemm_tc_kernel(const TgArgs a, const __grid_constant__ CUtensorMap xmap) {
       const bool split = gridDim.z > 1;
       float* const out = (split ? a.partial + (int64_t)blockIdx.z * a.M * N : a.y) + m0 * N + n;
       const float* const res = split || !a.residual ? nullptr : a.residual + m0 * N + n;
-      const int mleft = (int)min((int64_t)bn, a.M - m0);  // live activation rows of this tile
+      const int mleft = (int)min((int64_t)bn, mend - m0);  // live activation rows of this tile
       const int quarter_warps = (TG_WARPS - quarter + 3) / 4;
       for (int j0 = (warp >> 2) * 16; j0 < mleft; j0 += quarter_warps * 16) {
         uint32_t v[16];
@@ -935,7 +947,7 @@ int launch_dqgemm_tc(const WRef& w, const void* x, int x_type, int64_t M, float*
   a.w = w, a.xh = xh, a.inv_s = inv_s, a.M = M, a.bn = bn, a.tmem_cols = cols, a.y = y, a.residual = residual, a.error = err;
   CUtensorMap xmap;
   if (tg_make_xmap(const_cast<__half*>(xh), Mpad, K, bn, &xmap)) return 1;
-  a.nk_split = nk_split, a.partial = partial;
+  a.nk_split = nk_split, a.partial = partial, a.tiles = nullptr, a.bases = nullptr;
   const dim3 grid((unsigned)((w.rows + TG_BM - 1) / TG_BM), (unsigned)mtiles, (unsigned)splits);
   const bool a_tmem = tg_a_in_tmem(w.enc);
   const size_t stage_b = (a_tmem ? 0 : TG_A_BYTES) + (size_t)bn * 128;
@@ -970,6 +982,37 @@ int launch_dqgemm_tc(const WRef& w, const void* x, int x_type, int64_t M, float*
   }
   DYN_CUDA(cudaGetLastError());
   *handled = true;
+  return 0;
+}
+
+int launch_activation_prepare(const float* x, int64_t rows, int64_t K, __half* xh, float* inv_s, cudaStream_t s) {
+  DYN_CHECK(K % 2 == 0, "activation operand: odd width %lld", (long long)K);
+  tg_prepare_x_kernel<<<(unsigned)rows, 256, 0, s>>>(x, 0, rows, K, xh, inv_s);
+  count_launch();
+  DYN_CUDA(cudaGetLastError());
+  return 0;
+}
+
+int launch_dqgemm_tc_grouped(const WRef& w, const TgGroups& g, const __half* xh, const float* inv_s, int64_t M, float* y, cudaStream_t s) {
+  DYN_CHECK(tg_plain16(w.enc) && w.cols % TG_BK == 0 && w.cols >= TG_BK && w.rows >= 1 && M >= 1, "grouped GEMM: shape %lld x %lld",
+            (long long)w.rows, (long long)w.cols);
+  DYN_CHECK(g.bn >= 16 && g.bn <= 256 && g.bn % 16 == 0 && g.max_tiles >= 1 && g.max_tiles <= 65535, "grouped GEMM: %d tiles of %d rows",
+            g.max_tiles, g.bn);
+  int* err = device_error_word();
+  if (!err) return 1;
+  TgArgs a;
+  a.w = w, a.xh = xh, a.inv_s = inv_s, a.M = M, a.bn = g.bn, a.y = y, a.residual = nullptr, a.error = err;
+  a.tiles = g.tiles, a.bases = g.bases, a.partial = nullptr, a.nk_split = (int)(w.cols / TG_BK);
+  CUtensorMap xmap;
+  if (tg_make_xmap(const_cast<__half*>(xh), std::max<int64_t>(M, g.bn), w.cols, g.bn, &xmap)) return 1;
+  const size_t stage_b = (size_t)g.bn * 128, raw_b = (size_t)TG_A_WARPS * TG_RAW_WORDS * 4;
+  a.nslot = 2 * TG_GROUPS * stage_b + raw_b + 1024 <= 200 * 1024 ? 2 * TG_GROUPS : TG_GROUPS;
+  a.tmem_cols = 512;
+  const size_t smem = (size_t)a.nslot * stage_b + raw_b + 1024;
+  const dim3 grid((unsigned)((w.rows + TG_BM - 1) / TG_BM), (unsigned)g.max_tiles);
+  if (w.enc == E_BF16 ? tg_launch<E_BF16>(a, xmap, grid, smem, s) : tg_launch<E_F16>(a, xmap, grid, smem, s)) return 1;
+  count_launch();
+  DYN_CUDA(cudaGetLastError());
   return 0;
 }
 

@@ -148,8 +148,10 @@ __global__ void __launch_bounds__(gp_warps(M) * 32, 1) gemv_plain_kernel(const u
     const float v = row_sum(o);
     if (PAIRS)
       y[at] = (v / (1.0f + expf(-v))) * row_sum(own + o);
-    else
-      y[at] = residual ? v + residual[at] : v;
+    else {
+      const float b = form.bias ? v + aux_load(reinterpret_cast<const uint8_t*>(form.bias), form.bias_type, out0 + o) : v;
+      y[at] = residual ? b + residual[at] : b;
+    }
   }
 }
 
@@ -202,6 +204,7 @@ int launch_gemv_plain(const WRef& w, const void* x, int x_type, int M, float* y,
   *handled = false;
   if (!gemv_plain_takes(w, M)) return 0;
   DYN_CHECK(!form.norm_w || x_type == E_F32, "gemv: normalised input must be f32");
+  DYN_CHECK(!form.pairs || !form.bias, "gemv: pairs have no bias");
   DYN_CHECK(!form.pairs || (w.rows % 2 == 0 && !residual), "gemv: pairs need an even row count and no residual");
   int rc;
   const bool bf = w.enc == E_BF16;

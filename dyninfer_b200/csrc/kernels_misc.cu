@@ -227,16 +227,21 @@ int launch_norm_prepare(const float* x, const float* partial, int splits, const 
 }
 
 // PER > 0: the row fits PER elements per thread, computed once and kept in registers.
-template <int PER>
+// CLAMPED: min(g, limit) * sigmoid(1.702 min(g, limit)) * (clamp(u, +-limit) + 1) instead of silu(g) * u.
+template <int PER, bool CLAMPED>
 __global__ void __launch_bounds__(512)
-silu_prepare_kernel(const float* __restrict__ gu, int64_t I, __half* __restrict__ xh, float* __restrict__ inv_s) {
+silu_prepare_kernel(const float* __restrict__ gu, int64_t I, float limit, __half* __restrict__ xh, float* __restrict__ inv_s) {
   __shared__ float red[32];
   const int64_t row = blockIdx.x;
   const float* g = gu + row * 2 * I;
-  auto val = [&](int64_t i) {
-    const float gv = g[i];
-    return (gv / (1.0f + expf(-gv))) * g[I + i];
+  auto gated = [&](float gv, float uv) {
+    if (CLAMPED) {
+      gv = fminf(gv, limit), uv = fminf(fmaxf(uv, -limit), limit) + 1.0f;
+      return gv * (1.0f / (1.0f + expf(-1.702f * gv))) * uv;
+    }
+    return (gv / (1.0f + expf(-gv))) * uv;
   };
+  auto val = [&](int64_t i) { return gated(g[i], g[I + i]); };
   float mx = 0.f, sc, is;
   if constexpr (PER > 0) {
     float v[PER], up[PER];
@@ -247,7 +252,7 @@ silu_prepare_kernel(const float* __restrict__ gu, int64_t I, __half* __restrict_
     }
 #pragma unroll
     for (int k = 0; k < PER; k++) {
-      v[k] = (v[k] / (1.0f + expf(-v[k]))) * up[k];
+      v[k] = gated(v[k], up[k]);  // absent elements: 0
       mx = fmaxf(mx, fabsf(v[k]));
     }
     f16_row_scale(mx, red, &sc, &is);
@@ -264,16 +269,38 @@ silu_prepare_kernel(const float* __restrict__ gu, int64_t I, __half* __restrict_
   if (threadIdx.x == 0) inv_s[row] = is;
 }
 
-int launch_silu_prepare(const float* gate_up, int64_t rows, int64_t inter, __half* xh, float* inv_s, cudaStream_t s) {
+template <bool CLAMPED>
+static int run_glu_prepare(const float* gate_up, int64_t rows, int64_t inter, float limit, __half* xh, float* inv_s, cudaStream_t s) {
   if (rows == 0 || inter == 0) return 0;
-  if (inter <= 8 * 512)
-    silu_prepare_kernel<8><<<(unsigned)rows, 512, 0, s>>>(gate_up, inter, xh, inv_s);
-  else if (inter <= 16 * 512)
-    silu_prepare_kernel<16><<<(unsigned)rows, 512, 0, s>>>(gate_up, inter, xh, inv_s);
-  else if (inter <= 24 * 512)
-    silu_prepare_kernel<24><<<(unsigned)rows, 512, 0, s>>>(gate_up, inter, xh, inv_s);
-  else
-    silu_prepare_kernel<0><<<(unsigned)rows, 512, 0, s>>>(gate_up, inter, xh, inv_s);
+  const auto kernel = inter <= 8 * 512    ? silu_prepare_kernel<8, CLAMPED>
+                      : inter <= 16 * 512 ? silu_prepare_kernel<16, CLAMPED>
+                      : inter <= 24 * 512 ? silu_prepare_kernel<24, CLAMPED>
+                                          : silu_prepare_kernel<0, CLAMPED>;
+  kernel<<<(unsigned)rows, 512, 0, s>>>(gate_up, inter, limit, xh, inv_s);
+  count_launch();
+  DYN_CUDA(cudaGetLastError());
+  return 0;
+}
+
+int launch_silu_prepare(const float* gate_up, int64_t rows, int64_t inter, __half* xh, float* inv_s, cudaStream_t s) {
+  return run_glu_prepare<false>(gate_up, rows, inter, 0.f, xh, inv_s, s);
+}
+
+int launch_clamped_glu_prepare(const float* gate_up, int64_t rows, int64_t inter, float limit, __half* xh, float* inv_s, cudaStream_t s) {
+  return run_glu_prepare<true>(gate_up, rows, inter, limit, xh, inv_s, s);
+}
+
+__global__ void __launch_bounds__(256)
+add_bias_kernel(float* y, const uint8_t* __restrict__ bias, int bias_type, int64_t rows, int64_t width) {
+  for (int64_t i = blockIdx.x * 256ll + threadIdx.x; i < rows * width; i += (int64_t)gridDim.x * 256)
+    y[i] += aux_load(bias, bias_type, i % width);
+}
+
+int launch_add_bias(float* y, const void* bias, int bias_type, int64_t rows, int64_t width, cudaStream_t s) {
+  const int64_t n = rows * width;
+  if (n == 0) return 0;
+  add_bias_kernel<<<(unsigned)((n + 255) / 256 < 2368 ? (n + 255) / 256 : 2368), 256, 0, s>>>(
+      y, reinterpret_cast<const uint8_t*>(bias), bias_type, rows, width);
   count_launch();
   DYN_CUDA(cudaGetLastError());
   return 0;
@@ -685,6 +712,13 @@ attention_merge_kernel(const float* __restrict__ part, int nsplit, float* ctx, i
   }
 }
 
+int launch_attention_merge(const float* part, int nsplit, float* ctx, int64_t rows, int64_t nh, int64_t d, cudaStream_t s) {
+  attention_merge_kernel<<<dim3((unsigned)nh, (unsigned)rows), 256, 0, s>>>(part, nsplit, ctx, nh, d);
+  count_launch();
+  DYN_CUDA(cudaGetLastError());
+  return 0;
+}
+
 template <int KV>
 static int run_attention_split(const AttnArgs& a, float* part, int nsplit, cudaStream_t s) {
   const dim3 grid((unsigned)a.nh, (unsigned)a.rows, (unsigned)nsplit);
@@ -695,10 +729,8 @@ static int run_attention_split(const AttnArgs& a, float* part, int nsplit, cudaS
   } else {
     attention_split_kernel<KV, 8><<<grid, ATT_WARPS * 32, 0, s>>>(a, part, nsplit);
   }
-  attention_merge_kernel<<<dim3((unsigned)a.nh, (unsigned)a.rows), 256, 0, s>>>(part, nsplit, a.ctx, a.nh, a.d);
-  count_launch(2);
-  DYN_CUDA(cudaGetLastError());
-  return 0;
+  count_launch();
+  return launch_attention_merge(part, nsplit, a.ctx, a.rows, a.nh, a.d, s);
 }
 
 size_t attention_split_scratch_bytes(int64_t rows, int64_t nh, int64_t d, int nsplit) {

@@ -16,7 +16,6 @@
 namespace dyn {
 namespace {
 
-__device__ __forceinline__ float sigmoid_of(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 template <int KV>
 struct Lat;

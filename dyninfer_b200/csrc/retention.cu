@@ -19,6 +19,7 @@
 #include <algorithm>
 
 #include "mixers.cuh"
+#include "tf32x3.cuh"
 
 namespace cg = cooperative_groups;
 
@@ -30,19 +31,10 @@ constexpr int RT_PITCH = RT_C + 4;
 constexpr int RT_SLICE = 32;  // reduction elements staged at a time
 constexpr int RT_PRE = 16;    // state rows a decode thread fetches ahead
 
-// The angle of a position, reduced in double precision: p * f is far from 0 for long contexts.
-__device__ __forceinline__ void sincos_position(int64_t pos, double freq, float* sv, float* cv) {
-  const double turns = (double)pos * freq * 0.15915494309189535;  // 1 / 2 pi
-  const double frac = turns - rint(turns);
-  sincospif((float)(2.0 * frac), sv, cv);
-}
-
 __device__ __forceinline__ void load4(float* dst, const float* src) {  // src 16-byte aligned
   const float4 v = *reinterpret_cast<const float4*>(src);
   dst[0] = v.x, dst[1] = v.y, dst[2] = v.z, dst[3] = v.w;
 }
-
-__device__ __forceinline__ float silu_of(float z) { return z / (1.0f + expf(-z)); }
 
 // ---- decode: independent rows ----------------------------------------------------------------
 __global__ void __launch_bounds__(256) retention_step_kernel(RetentionArgs a, const int64_t* row_pos,
@@ -392,41 +384,6 @@ int chunk_out(const RetentionArgs& a, int64_t rows, int64_t base, cudaStream_t s
 // ---- the same two products on the tensor cores -----------------------------------------------------------
 constexpr int TC_D = 128;  // widest head (dim and vdim)
 constexpr int TC_AP = TC_D + 4, TC_BP = TC_D + 8, TC_SP = RT_C + 4;  // pitches: A-side and B-side fragment reads conflict-free
-
-struct Tf32Pair {
-  uint32_t hi, lo;
-};
-__device__ __forceinline__ Tf32Pair tf32_split(float x) {
-  Tf32Pair p;
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(p.hi) : "f"(x));
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(p.lo) : "f"(x - __uint_as_float(p.hi)));
-  return p;
-}
-__device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-struct AFrag {
-  uint32_t hi[4], lo[4];
-};
-__device__ __forceinline__ void split_into(AFrag& f, int i, float x) {
-  const Tf32Pair p = tf32_split(x);
-  f.hi[i] = p.hi, f.lo[i] = p.lo;
-}
-// c[nt] += a b[nt] for NT column tiles of one k-step; b(nt, 0 / 1) are the tile's two operand values. Term by term,
-// so that the products of consecutive instructions are independent.
-template <int NT, class B>
-__device__ __forceinline__ void mma3(float (&c)[NT][4], const AFrag& a, B b) {
-  Tf32Pair p[NT], q[NT];
-#pragma unroll
-  for (int nt = 0; nt < NT; nt++) p[nt] = tf32_split(b(nt, 0)), q[nt] = tf32_split(b(nt, 1));
-#pragma unroll
-  for (int nt = 0; nt < NT; nt++) mma_tf32(c[nt], a.lo, p[nt].hi, q[nt].hi);
-#pragma unroll
-  for (int nt = 0; nt < NT; nt++) mma_tf32(c[nt], a.hi, p[nt].lo, q[nt].lo);
-#pragma unroll
-  for (int nt = 0; nt < NT; nt++) mma_tf32(c[nt], a.hi, p[nt].hi, q[nt].hi);
-}
 
 // rows x cols floats (cols <= 128, both 16-byte aligned) into shared memory, zeros to `fill_rows` x 128
 __device__ __forceinline__ void stage_rows(float* dst, int pitch, const float* src, int64_t ld, int rows, int cols, int fill_rows,

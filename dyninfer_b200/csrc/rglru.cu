@@ -19,9 +19,6 @@
 namespace dyn {
 namespace {
 
-__device__ __forceinline__ float vec_at(const Vec& v, int64_t i) { return aux_load(v.ptr, v.type, i); }
-__device__ __forceinline__ float sigmoid_of(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ __forceinline__ float softplus_of(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float gelu_tanh_of(float z) {
   return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }

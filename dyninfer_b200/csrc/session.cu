@@ -34,6 +34,19 @@ bool follows_in_arena(const WRef& a, const WRef& b) {
          reinterpret_cast<const uint8_t*>(b.data) == reinterpret_cast<const uint8_t*>(a.data) + a.total_bytes();
 }
 
+__global__ void derive_norm_kernel(const uint8_t* w, int type, int64_t n, float offset, float scale, float* y) {
+  const int64_t i = blockIdx.x * 256ll + threadIdx.x;
+  if (i < n) y[i] = (offset + aux_load(w, type, i)) * scale;
+}
+
+int derive_norm(Session* s, NormW* w, int64_t n, float offset, float scale, float* dst) {
+  derive_norm_kernel<<<(unsigned)((n + 255) / 256), 256, 0, s->stream>>>(reinterpret_cast<const uint8_t*>(w->ptr), w->type, n, offset, scale, dst);
+  DYN_CUDA(cudaGetLastError());
+  DYN_CUDA(cudaStreamSynchronize(s->stream));
+  w->ptr = dst, w->type = E_F32, w->bytes = (uint64_t)n * 4;
+  return 0;
+}
+
 // A product in the session's arithmetic: the framework's choice of kernel, or f32 throughout.
 int session_linear(Session* s, const WRef& w, const void* x, int x_type, int64_t m, float* y, const float* residual) {
   return s->cfg.exact ? launch_linear_exact(w, x, x_type, m, y, residual, s->stream)
@@ -775,6 +788,8 @@ int dyninfer_cuda_session_create_with_file_params(
   cfg.vocab = (int)desc.number("vocab", 0);
   cfg.eps = (float)desc.number("eps", 1e-6);
   cfg.theta = (float)desc.number("theta", 10000.0);
+  cfg.norm_offset = (float)desc.number("norm_offset", 0);
+  cfg.logit_scale = (float)desc.number("logit_scale", 1);
   cfg.qk_norm = desc.number("qk_norm", 1) != 0;
   cfg.rope = desc.number("rope", 1) != 0;
   cfg.batch = (int)desc.number("batch", 1);
@@ -803,6 +818,8 @@ int dyninfer_cuda_session_create_with_file_params(
   if (cfg.tp_world > 1) cfg.persistent = false;  // the single-GPU persistent kernel has no exchange step
   const bool mixers = !cfg.mixers.empty();
   DYN_CHECK(!mixers || cfg.tp_world == 1, "a decoder with mixers has no tensor-parallel form");
+  DYN_CHECK(mixers || (cfg.norm_offset == 0.f && cfg.logit_scale == 1.f),
+            "norm weights around an offset and scaled logits need a decoder with listed mixers");
   DYN_CHECK(cfg.layers > 0 && cfg.hidden > 0 && cfg.vocab > 0 && cfg.batch > 0 &&
                 (mixers || (cfg.inter > 0 && cfg.heads > 0 && cfg.kv_heads > 0 && cfg.head_dim > 0)),
             "model descriptor lacks geometry (layers/hidden/intermediate/heads/kv_heads/head_dim/vocab)");
@@ -1100,7 +1117,7 @@ int dyninfer_cuda_session_create_with_file_params(
     grow(s->lm_head);
     for (const MixerLayer& L : s->mix) {
       for (const WRef& w : L.in) grow(w);
-      for (const WRef* w : {&L.o, &L.gate, &L.up, &L.gate_up, &L.down})
+      for (const WRef* w : {&L.o, &L.gate, &L.up, &L.gate_up, &L.down, &L.router})
         if (w->data) grow(*w);
     }
     for (const LayerW& L : s->layers) {
@@ -1189,7 +1206,7 @@ void dyninfer_cuda_session_destroy(dyninfer_cuda_session_t* s) {
                  s->hist_dev, s->hist_count_dev, s->argmax_scratch, s->mega_layers, s->io_dev,
                  s->prof_dev, s->trace_dev, s->prog_dev, s->ll_dev, s->batch_logits, s->batch_tokens_dev, s->tp_part, s->tp_logits,
                  s->tp_gather, s->scratch, s->qkv1, s->gu1, s->xh, s->xinv, s->gpart,
-                 s->lcache, s->state, s->mix_scratch, s->tables, s->want_logits, s->want_index_dev};
+                 s->lcache, s->state, s->mix_scratch, s->tables, s->expert_tables, s->want_logits, s->want_index_dev};
   for (void* p : dev)
     if (p) cudaFree(p);
   if (s->logits_host) cudaFreeHost(s->logits_host);

@@ -29,28 +29,48 @@ struct LayerW {
 };
 
 // One layer of a decoder whose layers are listed one by one: which mixer, its sizes, its feed-forward.
-enum MixerKind { MIX_RETENTION = 0, MIX_RGLRU = 1, MIX_LATENT = 2 };
+enum MixerKind { MIX_RETENTION = 0, MIX_RGLRU = 1, MIX_LATENT = 2, MIX_SOFTMAX = 3, MIX_DELTA = 4 };
 struct MixerCfg {
   MixerKind kind = MIX_RETENTION;
   int tensors = 0;  // the layer whose parameters this one runs with (itself, or one it shares them with)
+  bool parallel = false;  // mixer and feed-forward read the same residual row; otherwise one after the other
   int ff = 0;       // width of the gated feed-forward, 0: none
-  int heads = 0, dim = 0, vdim = 0, rot_dims = 0;
+  int heads = 0, kv_heads = 0, dim = 0, vdim = 0, rot_dims = 0;
   double rot_base = 0;
   std::vector<double> decay;
   int width = 0, blocks = 0, taps = 0;
   int rank = 0;
-  float scale = 0.f;
+  float scale = 0.f, softcap = 0.f;
+  bool bias = false;  // products of the mixer have biases
+  // a mixture of experts instead of the feed-forward (experts > 0), with a shared one (shared_ff > 0)
+  int experts = 0, top = 0, expert_ff = 0, shared_ff = 0;
+  float expert_limit = 0.f, shared_limit = 0.f;
+  bool feeds_forward() const { return ff > 0 || experts > 0; }
+  int gated_width() const { return experts ? shared_ff : ff; }  // width of the matrices gate, up and down
+  // cached elements per token and slot
+  size_t cached() const {
+    return kind == MIX_LATENT ? (size_t)rank : kind == MIX_SOFTMAX ? (size_t)kv_heads * (dim + vdim) : 0;
+  }
+  bool same_sizes(const MixerCfg& o) const {
+    return heads == o.heads && kv_heads == o.kv_heads && dim == o.dim && vdim == o.vdim && rot_dims == o.rot_dims && width == o.width &&
+           blocks == o.blocks && taps == o.taps && rank == o.rank && bias == o.bias && ff == o.ff && experts == o.experts &&
+           expert_ff == o.expert_ff && shared_ff == o.shared_ff;
+  }
 };
 
 struct MixerLayer {
   MixerCfg c;
   NormW norm1, norm2;
   std::vector<WRef> in;       // input products; matrices laid back to back are one
-  int part_in[4] = {}, parts = 0;
-  int64_t part_col[4] = {};   // part p = columns from part_col[p] of product part_in[p]
+  int part_in[6] = {}, parts = 0;
+  int64_t part_col[6] = {};   // part p = columns from part_col[p] of product part_in[p]
   WRef o, gate, up, gate_up, down;
   NormW by, bx, conv, bc, ra, bra, ri, bri, lam, lat_norm;
   WRef uk, uv, ukv;
+  NormW qb, kb, vb, ob;       // softmax attention
+  NormW conv_q, conv_k, conv_v, a_log, dt, head_norm;  // delta rule
+  WRef router;
+  MoeArgs moe;                // experts' tables and shapes; scratch is the session's
   double* freq = nullptr;     // device tables of the owning layer
   float* decay = nullptr;
   size_t state_off = 0, state_floats = 0;  // per slot: floats in the state pool (regions [slot][...])
@@ -62,6 +82,8 @@ struct ModelCfg {
   std::vector<MixerCfg> mixers;  // non-empty: one entry per layer
   int layers = 0, hidden = 0, inter = 0, heads = 0, kv_heads = 0, head_dim = 0, vocab = 0;
   float eps = 1e-6f, theta = 10000.f;
+  // what the stored norm weights count from (0: plain weights), and the factor of the logits
+  float norm_offset = 0.f, logit_scale = 1.f;
   bool qk_norm = true, rope = true;
   int batch = 1;
   int kv2_type = E_BF16;  // element type used when the KV cache is configured with 2 bytes
@@ -106,7 +128,8 @@ struct dyninfer_cuda_session_t {
   size_t state_floats = 0;
   float* mix_scratch = nullptr;
   size_t mix_scratch_floats = 0;
-  float* tables = nullptr;       // decays and angles per position of all layers
+  float* tables = nullptr;       // decays, angles per position, norm weights counted from an offset
+  const uint8_t** expert_tables = nullptr;  // addresses of the experts' matrices
   std::vector<int64_t> slot_pos;
   // logits of several rows of a portion
   float* want_logits = nullptr;  // [want_cap, vocab]
@@ -214,6 +237,8 @@ struct ParamTable {
   virtual int plain(const std::string& name, const std::vector<int64_t>& shape, NormW* out) const = 0;
   virtual ~ParamTable() = default;
 };
+// The derived weights scale * (offset + w) of a norm, in f32 at `dst` (device); *w then refers to them.
+int derive_norm(Session* s, NormW* w, int64_t n, float offset, float scale, float* dst);
 bool follows_in_arena(const WRef& a, const WRef& b);
 int session_linear(Session* s, const WRef& w, const void* x, int x_type, int64_t m, float* y, const float* residual);
 

@@ -17,7 +17,8 @@ OPERATIONS = ("Input", "Embedding", "Linear", "RmsNorm", "PerHeadRmsNorm", "Rope
               "KvCacheRead", "Attention", "ShortConv", "Silu", "Multiply", "Residual",
               "OutputProjection",
               # mixers beyond the reference's GQA attention
-              "Retention", "GatedRecurrence", "LatentAttention", "OutputGate")
+              "Retention", "GatedRecurrence", "LatentAttention", "GatedDelta", "OutputGate", "Bias",
+              "ExpertChoice", "ExpertSum")
 MODES = ("prefill", "decode")
 
 
@@ -168,6 +169,8 @@ def register_cuda_candidates(reg: KernelRegistry) -> KernelRegistry:
                     ("ShortConv", "short_conv.cuda_sm100.f32"), ("Retention", "retention.cuda_sm100.f32"),
                     ("GatedRecurrence", "rglru.cuda_sm100.f32"),
                     ("LatentAttention", "attention.latent.cuda_sm100"),
+                    ("GatedDelta", "gated_delta.cuda_sm100.f32"), ("Bias", "bias.cuda_sm100.f32"),
+                    ("ExpertChoice", "moe.choice.cuda_sm100.f32"), ("ExpertSum", "moe.sum.cuda_sm100.f32"),
                     ("OutputGate", "output_gate.cuda_sm100.f32")):
         reg.register(KernelCandidate(id=kid, operation=op, encoding=None, target=CUDA_SM100,
                                      deterministic_score=200, lowering=kid))
@@ -213,6 +216,22 @@ def _mixer_operations(config: dict, par):
             ops += [*linear("rec_y", "rec_x"), (p + "rec_conv", "ShortConv", None, None),
                     (p + "recurrence", "GatedRecurrence", None, None),
                     (p + "output_gate", "OutputGate", None, None), *linear("rec_output")]
+        elif m["type"] == "softmax_attention":
+            ops += linear("attn_q", "attn_k", "attn_v")
+            if m["bias"]:
+                ops.append((p + "qkv_bias", "Bias", None, None))
+            if m["rot_dims"]:
+                ops += [(p + "rope_q", "Rope", None, None), (p + "rope_k", "Rope", None, None)]
+            ops += [(p + "kv_write_k", "KvCacheWrite", None, None), (p + "kv_write_v", "KvCacheWrite", None, None),
+                    (p + "kv_read_k", "KvCacheRead", None, None), (p + "kv_read_v", "KvCacheRead", None, None),
+                    (p + "attention", "Attention", None, None), *linear("attn_output")]
+            if m["bias"]:
+                ops.append((p + "output_bias", "Bias", None, None))
+        elif m["type"] == "gated_delta":
+            ops += [*linear("attn_q", "attn_k", "attn_v", "attn_gate", "delta_beta", "delta_decay"),
+                    *((p + f"conv_{x}", "ShortConv", None, None) for x in "qkv"), (p + "delta", "GatedDelta", None, None),
+                    (p + "head_norm", "PerHeadRmsNorm", None, None), (p + "output_gate", "OutputGate", None, None),
+                    *linear("attn_output")]
         else:
             ops += [*linear("attn_q", "attn_kv_down", "attn_gate"), (p + "attn_kv_norm", "RmsNorm", None, None),
                     (p + "kv_write_latent", "KvCacheWrite", None, None), *linear("attn_k_up", "attn_v_up"),
@@ -220,7 +239,13 @@ def _mixer_operations(config: dict, par):
                     (p + "attention", "LatentAttention", None, None),
                     (p + "output_gate", "OutputGate", None, None), *linear("attn_output")]
         ops.append((p + "mixer_residual", "Residual", None, None))
-        if m["ff"]:
+        if m.get("experts"):
+            ops += [(p + "ffn_norm", "RmsNorm", None, None), *linear("ffn_router"), (p + "expert_choice", "ExpertChoice", None, None)]
+            for x in [f"expert_{e}" for e in range(m["experts"])] + (["ffn"] if m["shared_ff"] else []):
+                ops += [*linear(x + "_gate", x + "_up"), (p + x + "_silu", "Silu", None, None),
+                        (p + x + "_mul", "Multiply", None, None), *linear(x + "_down")]
+            ops += [(p + "expert_sum", "ExpertSum", None, None), (p + "ffn_residual", "Residual", None, None)]
+        elif m["ff"]:
             ops += [(p + "ffn_norm", "RmsNorm", None, None), *linear("ffn_gate", "ffn_up"),
                     (p + "ffn_silu", "Silu", None, None), (p + "ffn_mul", "Multiply", None, None),
                     *linear("ffn_down"), (p + "ffn_residual", "Residual", None, None)]

@@ -340,12 +340,81 @@ def zupudra_tensors(doc: dict, seed: int = 0, dtype=np.float32) -> dict:
     return out
 
 
-def write_zupudra(dirpath: str, doc: dict, seed: int = 0, tensors: dict | None = None) -> str:
-    """Seeded Zupudra directory (config.json + bf16 model.safetensors). `tensors` replaces the random weights."""
+def _write_listed(dirpath: str, doc: dict, architecture: str, t: dict) -> str:
     os.makedirs(dirpath, exist_ok=True)
-    t = zupudra_tensors(doc, seed) if tensors is None else tensors
     ck.write_safetensors(os.path.join(dirpath, "model.safetensors"),
                          {k: ("BF16", v.shape, f32_to_bf16_bits(np.ascontiguousarray(v, np.float32))) for k, v in t.items()})
     with open(os.path.join(dirpath, "config.json"), "w") as f:
-        json.dump(dict(doc, architecture="Zupudra"), f)
+        json.dump(dict(doc, architecture=architecture), f)
     return dirpath
+
+
+def write_zupudra(dirpath: str, doc: dict, seed: int = 0, tensors: dict | None = None) -> str:
+    """Seeded Zupudra directory (config.json + bf16 model.safetensors). `tensors` replaces the random weights."""
+    return _write_listed(dirpath, doc, "Zupudra", zupudra_tensors(doc, seed) if tensors is None else tensors)
+
+
+def rufusun_shapes(doc: dict) -> dict:
+    """Tensor name -> shape of a Rufusun configuration."""
+    W = doc["width"]
+    out = {"embed": (doc["vocab"], W), "final.norm": (W,), "head": (doc["vocab"], W)}
+
+    def gated(prefix, ff):
+        out.update({prefix + "gate": (ff, W), prefix + "up": (ff, W), prefix + "down": (W, ff)})
+
+    for i, layer in enumerate(doc["layers"]):
+        m, p, mx, mlp = layer["mixer"], f"l{i}.", f"l{i}.mix.", layer.get("mlp")
+        out[p + "norm1"] = (W,)
+        H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        if layer["type"] == "attention":
+            for n, rows in (("q", H * D), ("k", G * D), ("v", G * E)):
+                out.update({mx + n: (rows, W), mx + n + ".b": (rows,)})
+            out.update({mx + "o": (W, H * E), mx + "o.b": (W,)})
+        else:
+            for n, rows in (("q", G * D), ("k", G * D), ("v", H * E)):
+                out.update({mx + n: (rows, W), mx + n + ".conv": (rows, m["conv"])})
+            out.update({mx + "g": (H * E, W), mx + "b": (H, W), mx + "a": (H, W), mx + "A_log": (H,), mx + "dt_bias": (H,),
+                        mx + "norm": (E,), mx + "o": (W, H * E)})
+        if not mlp:
+            continue
+        out[p + "norm2"] = (W,)
+        if mlp["kind"] == "dense":
+            gated(p + "mlp.", mlp["ff"])
+            continue
+        out[p + "mlp.router"] = (mlp["router"]["experts"], W)
+        for e in range(mlp["router"]["experts"]):
+            gated(p + f"mlp.e{e}.", mlp["expert"]["ff"])
+        if mlp.get("shared"):
+            gated(p + "mlp.shared.", mlp["shared"]["ff"])
+    return out
+
+
+def rufusun_tensors(doc: dict, seed: int = 0, dtype=np.float32) -> dict:
+    """Seeded random weights: matrices of unit gain (routers spread further), norms of the residual around 0 and of
+    the heads around 1, decays that forget over a few to a few hundred tokens."""
+    out = {}
+    for name, shape in rufusun_shapes(doc).items():
+        rng = np.random.default_rng(tensor_seed(seed, name))
+        if name.endswith(".mix.norm"):
+            w = rng.uniform(0.7, 1.3, size=shape)
+        elif name.endswith(("norm", "norm1", "norm2")):
+            w = rng.uniform(-0.3, 0.3, size=shape)
+        elif name.endswith(".A_log"):
+            w = rng.uniform(-3.0, 0.5, size=shape)
+        elif name.endswith(".dt_bias"):
+            w = rng.uniform(-4.0, 0.0, size=shape)
+        elif name.endswith(".b") and len(shape) == 1:
+            w = rng.normal(0.0, 0.3, size=shape)
+        elif name.endswith(".router"):
+            w = rng.normal(0.0, 3.0 * shape[-1] ** -0.5, size=shape)
+        elif name == "embed":
+            w = rng.normal(0.0, 1.0, size=shape)
+        else:
+            w = rng.normal(0.0, shape[-1] ** -0.5, size=shape)
+        out[name] = w.astype(dtype)
+    return out
+
+
+def write_rufusun(dirpath: str, doc: dict, seed: int = 0, tensors: dict | None = None) -> str:
+    """Seeded Rufusun directory (config.json + bf16 model.safetensors). `tensors` replaces the random weights."""
+    return _write_listed(dirpath, doc, "Rufusun", rufusun_tensors(doc, seed) if tensors is None else tensors)

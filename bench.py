@@ -372,11 +372,11 @@ def main():
     ap.add_argument("--no-tp", action="store_true", help="skip the tensor-parallel section (32B shape)")
     ap.add_argument("--decode-only", action="store_true",
                     help="prompt + W + K device-loop decode steps and nothing else (small case for profiler captures)")
-    ap.add_argument("--arch", choices=["zupudra"], help="throughput of this design beside a Qwen3-shaped model of equal size "
+    ap.add_argument("--arch", choices=["zupudra", "rufusun"], help="throughput of this design beside a Qwen3-shaped model of equal size "
                                                         "instead of the headline workload (one GPU)")
     ap.add_argument("--arch-size", default="0.4b,1b,7b-layers")
     ap.add_argument("--arch-prompt", type=int, default=2048)
-    ap.add_argument("--arch-profile", choices=["zupudra", "qwen3"], help="one prompt and four decode steps of one model, nothing "
+    ap.add_argument("--arch-profile", choices=["zupudra", "rufusun", "qwen3"], help="one prompt and four decode steps of one model, nothing "
                                                                          "else (small case for a launch list)")
     args = ap.parse_args()
     args.warmup = max(3, args.warmup)
@@ -397,7 +397,7 @@ def main():
         if args.arch_profile:
             arch_bench.profile_case(args.arch_profile, args.arch_size.split(",")[0], args.arch_prompt, 4)
         else:
-            arch_bench.run(args.arch_size.split(","), args.arch_prompt, args.steps, args.warmup,
+            arch_bench.run(args.arch, args.arch_size.split(","), args.arch_prompt, args.steps, args.warmup,
                            lambda: ClockSampler(local_rank))
         return
 

@@ -1,9 +1,11 @@
-"""Throughput of the Zupudra design beside a Qwen3-shaped model of equal size (random bf16 weights).
+"""Throughput of a design with listed mixers beside a Qwen3-shaped model of equal size (random bf16 weights).
 
-    python bench.py --arch zupudra [--arch-size 0.4b,1b,7b-layers] [--steps K] [--warmup W]
+    python bench.py --arch zupudra|rufusun [--arch-size 0.4b,1b,7b-layers] [--steps K] [--warmup W]
 
 Both models of a size have the same width, layer count, feed-forward width, heads of 128, vocabulary and 16-bit
-plain weights; Zupudra's layers alternate retention, gated recurrence and latent attention. Measured
+plain weights. Zupudra's layers alternate retention, gated recurrence and latent attention. Rufusun's alternate gated
+delta rule and softmax attention, two layers with a dense feed-forward, then two with 16 experts of which a token uses
+four beside a shared one: as many feed-forward weights per token as the dense one. Measured
 through the session: prefill of a random prompt (host clock around `prefill_argmax`), single-sequence greedy
 decode after it (`decode_loop`, CUDA events on the session stream) and batched decode (`step`, host clock,
 tokens in and out through host memory). Prints one JSON line per size.
@@ -41,6 +43,24 @@ def zupudra_doc(size: str) -> dict:
     return {"layers": [kinds[i % 3] for i in range(layers)], "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6}}
 
 
+def rufusun_doc(size: str) -> dict:
+    width, layers, heads, _, _, ff, kv = SIZES[size]
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 6, "limit": 7.0}, "router": {"experts": 16, "top": 4},
+           "shared": {"ff": ff // 3, "limit": 7.0}}
+    delta = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}
+    attention = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+                 "rot": {"dims": 128, "base": 5e5}}
+    kinds = [{"type": t, "mixer": m, "mlp": f} for f in (dense, moe) for t, m in (("delta", delta), ("attention", attention))]
+    return {"layers": [kinds[i % 4] for i in range(layers)], "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6},
+            "logit_scale": 1.0}
+
+
+# architecture -> configuration, shapes, weights, writer, kinds of layers in turn
+DESIGNS = {"zupudra": (zupudra_doc, synth.zupudra_shapes, synth.zupudra_tensors, synth.write_zupudra, 3),
+           "rufusun": (rufusun_doc, synth.rufusun_shapes, synth.rufusun_tensors, synth.write_rufusun, 4)}
+
+
 def qwen_config(size: str) -> dict:
     width, layers, heads, _, _, ff, kv = SIZES[size]
     return dict(layers=layers, hidden=width, heads=heads, kv_heads=kv, head_dim=128, intermediate=ff, vocab=VOCAB, eps=1e-6,
@@ -58,14 +78,15 @@ def checkpoint(kind: str, size: str) -> str:
     if kind == "qwen3":
         synth.write_qwen3_gguf(tmp, qwen_config(size), seed=SEED, default="plain.bf16", embd="plain.bf16", repeat_layers=True)
     else:
-        doc = zupudra_doc(size)
-        first = synth.zupudra_tensors(dict(doc, layers=doc["layers"][:3]), SEED)
+        doc_of, shapes, random_tensors, write, kinds = DESIGNS[kind]
+        doc = doc_of(size)
+        first = random_tensors(dict(doc, layers=doc["layers"][:kinds]), SEED)
         tensors = {}
-        for name in synth.zupudra_shapes(doc):
+        for name in shapes(doc):
             p, _, rest = name.partition(".")
-            src = f"l{int(p[1:]) % 3}.{rest}" if p[0] == "l" and p[1:].isdigit() else name
+            src = f"l{int(p[1:]) % kinds}.{rest}" if p[0] == "l" and p[1:].isdigit() else name
             tensors[name] = first[src]
-        synth.write_zupudra(tmp, doc, tensors=tensors)
+        write(tmp, doc, tensors=tensors)
     os.replace(tmp, path)
     return path
 
@@ -104,12 +125,12 @@ def measure(path: str, prompt_len: int, steps: int, warmup: int, batches=(8, 32)
     return out
 
 
-def run(sizes, prompt_len: int, steps: int, warmup: int, clocks) -> None:
+def run(arch: str, sizes, prompt_len: int, steps: int, warmup: int, clocks) -> None:
     for size in sizes:
-        line = {"metric": "arch_tokens_per_s", "arch": "zupudra", "size": size, "prompt": prompt_len, "steps": steps,
+        line = {"metric": "arch_tokens_per_s", "arch": arch, "size": size, "prompt": prompt_len, "steps": steps,
                 "warmup": warmup, "dtype": "bf16 weights and cache", "data": "synthetic", "n_gpus": 1,
                 "l2": "each decode step streams more weight bytes than L2 holds"}
-        paths = {kind: checkpoint(kind, size) for kind in ("zupudra", "qwen3")}
+        paths = {kind: checkpoint(kind, size) for kind in (arch, "qwen3")}
         with clocks() as c:
             for kind, path in paths.items():
                 line[kind] = measure(path, prompt_len, steps, warmup)

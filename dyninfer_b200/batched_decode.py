@@ -1,12 +1,12 @@
 """Batched prefill + greedy decode benchmark on seeded synthetic checkpoints, bf16 KV cache.
 
-    python -m dyninfer_b200.batched_decode [--model 0.6b-mlx|8b-mixed|0.6b-q4_0|zupudra-0.4b|zupudra-1b] [--batch 1,8,32,64]
+    python -m dyninfer_b200.batched_decode [--model 0.6b-mlx|8b-mixed|0.6b-q4_0|zupudra-0.4b|zupudra-1b|rufusun-0.4b|rufusun-1b] [--batch 1,8,32,64]
                                            [--prompt 512] [--steps 256] [--chunk 512]
 
 Models: `0.6b-mlx` = Qwen3-0.6B shape, MLX affine-U4 linears (group 64, bf16 scales and biases), tied
 bf16 embeddings, SafeTensors; `8b-mixed` = Qwen3-8B shape GGUF with q/k/o/gate/up Q4_0, attn_v Q4_1,
-ffn_down Q8_0, token_embd and output Q6_K (untied); `0.6b-q4_0` = the headline decode model; `zupudra-*` = the
-Zupudra models of `arch_bench` (bf16).
+ffn_down Q8_0, token_embd and output Q6_K (untied); `0.6b-q4_0` = the headline decode model; `zupudra-*`, `rufusun-*` = the
+models of that name of `arch_bench` (bf16).
 
 For every batch size B: B sequences are prefilled with `--prompt` random token ids each (timed, one
 sequence after the other, in chunks of `--chunk` rows),
@@ -59,15 +59,16 @@ def checkpoint(model: str):
             synth.write_qwen3_gguf(tmp, synth.QWEN3_0_6B, seed=SEED)
             os.replace(tmp, path)
         return path, synth.QWEN3_0_6B
-    if model.startswith("zupudra-"):
+    if model.startswith(("zupudra-", "rufusun-")):
         from . import arch_bench
-        return arch_bench.checkpoint("zupudra", model[len("zupudra-"):]), {"vocab": arch_bench.VOCAB}
+        return arch_bench.checkpoint(*model.split("-", 1)), {"vocab": arch_bench.VOCAB}
     raise SystemExit(f"unknown model {model!r}")
 
 
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", default="0.6b-mlx", choices=["0.6b-mlx", "8b-mixed", "0.6b-q4_0", "zupudra-0.4b", "zupudra-1b"])
+    ap.add_argument("--model", default="0.6b-mlx", choices=["0.6b-mlx", "8b-mixed", "0.6b-q4_0", "zupudra-0.4b", "zupudra-1b",
+                                                             "rufusun-0.4b", "rufusun-1b"])
     ap.add_argument("--chunk", type=int, default=512, help="prefill chunk size (rows per forward call)")
     ap.add_argument("--batch", default="1,8,32,64")
     ap.add_argument("--prompt", type=int, default=512)

@@ -265,6 +265,28 @@ struct TgGroups {
   int max_tiles = 0, bn = 0;               // bn: a multiple of 16, at most 256
 };
 int launch_dqgemm_tc_grouped(const WRef& w, const TgGroups& g, const __half* xh, const float* inv_s, int64_t M, float* y, cudaStream_t s);
+// Grouped GEMM of f16 matrices by tile copies (gemm_grouped.cu): as above, weights as tensor maps [matrices][gate, up, down]. y:
+// rows times `down`, scaled per row; yh: gate and up of the rows, gated with `limit`, times out_scale as f16 [M, N].
+struct GroupedGemm {
+  const void* maps = nullptr;  // device, of 128 bytes each (make_grouped_weight_map)
+  const int4* tiles = nullptr;
+  int max_tiles = 0, bn = 0;
+  const __half* xh = nullptr;  // [M, K], at least bn rows allocated
+  const float* inv_s = nullptr;  // nullptr: in_scale for every row
+  float in_scale = 1.f;
+  int64_t M = 0, N = 0, K = 0;
+  float* y = nullptr;
+  __half* yh = nullptr;
+  float limit = 0.f, out_scale = 1.f;
+};
+constexpr int GROUPED_MAP_BYTES = 128;
+bool grouped_gemm_takes(int64_t rows, int64_t K);
+int make_grouped_weight_map(const uint8_t* w, int64_t rows, int64_t K, void* map);
+int launch_grouped_gemm(const GroupedGemm& g, cudaStream_t s);
+// The largest magnitude of `count` bf16 values of every matrix of a device table (as float bits, kept in *largest_dev), and
+// their conversion to f16 in place.
+int bf16_table_range(const uint8_t* const* table, int matrices, int64_t count, int* largest_dev, cudaStream_t s);
+int bf16_table_to_f16(const uint8_t* const* table, int matrices, int64_t count, cudaStream_t s);
 // Whether launch_dqgemm_tc takes the product, and the activation rows its tiling pads M to.
 bool dqgemm_tc_takes(const WRef& w, int64_t M);
 int64_t dqgemm_tc_padded_rows(const WRef& w, int64_t M);
@@ -305,9 +327,19 @@ int launch_rms_norm(const float* x, const void* w, int w_type, int64_t rows, int
 //   v = (splits ? sum over the K-split sums partial[z][row][:] : x[row][:]) + residual[row][:]  -> hidden (if given)
 //   y = RMSNorm(v) * w, written as the GEMM's activation operand: xh[row][:] = f16(y * 2^k), inv_s[row] = 2^-k.
 // Bit for bit what tg_split_reduce_kernel, rms_norm_kernel and the GEMM's activation pass produce in turn.
+// A second norm of the same v as a second operand, and a bias added to v where it is left in `hidden` (not where it is
+// normalised): layers whose two branches read one residual row.
+struct NormPair {
+  const void* w = nullptr;
+  int type = E_F32;
+  __half* xh = nullptr;
+  float* inv_s = nullptr;
+  const void* bias = nullptr;
+  int bias_type = E_F32;
+};
 int launch_norm_prepare(const float* x, const float* partial, int splits, const float* residual, float* hidden,
                         const void* w, int w_type, int64_t rows, int64_t width, float eps, __half* xh, float* inv_s,
-                        cudaStream_t s);
+                        cudaStream_t s, const NormPair& pair = NormPair());
 // The same for the SwiGLU: rows of [gate | up] -> silu(gate) * up as the GEMM's activation operand.
 int launch_silu_prepare(const float* gate_up, int64_t rows, int64_t inter, __half* xh, float* inv_s, cudaStream_t s);
 // and for min(gate, limit) * sigmoid(1.702 min(gate, limit)) * (clamp(up, +-limit) + 1)

@@ -17,8 +17,10 @@
 //     solve (I + A) u = beta v - beta b (K S_0), A_ts = beta_t b_t / b_s (k_t . k_s) for s < t. delta_chunk_kernel forms
 //     T = (I + A)^-1 by 16 x 16 blocks, U = T (beta v), W = T (beta b k) and P_ts = b_t / b_s (q_t . k_s) for every chunk at
 //     once; delta_scan_kernel walks the chunks: V = U - W S, o = b (Q S) + P V, S <- b_C S + (K b_C / b)^T V, a
-//     CTA per (head, 32 value columns), state in registers. All products with pairs of tf32 terms.
-// delta_finish_kernel applies norm and gate to a portion's rows.
+//     CTA per (head, 32 value columns): half of its warps hold the state in registers and form corrections and updates,
+//     the other half the outputs. All products with pairs of tf32 terms.
+// delta_finish_kernel applies norm and gate to a portion's rows; delta_finish_operand_kernel leaves them as the dequant
+// GEMM's activation operand.
 #include <cooperative_groups.h>
 
 #include <algorithm>
@@ -72,17 +74,6 @@ __device__ __forceinline__ HeadIn head_in(const DeltaArgs& a, int slot) {
   return s;
 }
 
-// silu(conv) of channel c of a head at position pos; x is the current input, earlier ones come from the slot's ring.
-__device__ __forceinline__ float conv_at(const DeltaArgs& a, const HeadIn& s, int c, float x, int64_t pos, const float* ring,
-                                         int64_t C) {
-  const int64_t w = (s.w0 + c) * a.taps;
-  float u = vec_at(s.w, w + a.taps - 1) * x;
-#pragma unroll 4
-  for (int j = 1; j < a.taps; j++)
-    if (pos >= j) u = fmaf(vec_at(s.w, w + a.taps - 1 - j), ring[((pos - j) % a.taps) * C + s.ch + c], u);
-  return silu_of(u);
-}
-
 __device__ __forceinline__ float block_total(float v, float* red) {  // red: 8 floats; all 256 threads
   v = warp_sum(v);
   __syncthreads();
@@ -124,78 +115,134 @@ __device__ __forceinline__ void delta_token(float* S, int D, int per, int ne, co
 }
 
 // ---- decode: independent rows ----------------------------------------------------------------
+// Everything that earlier tokens left (state, convolution history) is gathered before the wait for this token's
+// products. Sums over the state run on the convolved q and k as they are; their lengths enter afterwards, as factors.
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire;" ::: "memory"); }
+
 __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(DeltaArgs a, const int64_t* row_pos, const int64_t* row_seq,
-                                                                int64_t pos0, int64_t seq0, int64_t row0) {
+                                                                int64_t pos0, int64_t seq0, int64_t row0, int wide) {
   extern __shared__ __align__(16) float dl_smem[];
-  __shared__ float part_ss, red8[8];
+  __shared__ float part_ss, red[3];
   const cg::cluster_group cl = cg::this_cluster();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int D = a.dim, E = a.vdim, nsplit = gridDim.x, h = blockIdx.y;
   const int64_t r = row0 + blockIdx.z, C = channels_of(a);
   const int per = (E + nsplit - 1) / nsplit, e0 = min((int)blockIdx.x * per, E), ne = min(per, E - e0);
   float* S = dl_smem;             // [D][per]
-  float* qs = S + D * per;        // [D]
+  float* us = S + D * per;        // [per]
+  float* os = us + per;           // [per]
+  float* sums = os + per;         // [2][8][per]
+  float* qs = sums + 16 * per;    // [D]
   float* ks = qs + D;             // [D]
   float* vs = ks + D;             // [per]
-  float* us = vs + per;           // [per]
-  float* os = us + per;           // [per]
-  float* red = os + per;          // [2][8][per]
+  float* w0s = vs + per;          // [2 D + per] weights of the current input
   pdl_trigger();
   const int64_t pos = row_pos ? row_pos[r] : pos0, seq = row_seq ? row_seq[r] : seq0;
-  // the state was written one token ago, with ordinary launches in between: it is fetched before the kernel waits
-  // for this token's products
+  // the state was written one token ago, with ordinary launches in between
   float* Sg = a.state + ((seq * a.heads + h) * D) * (int64_t)E + e0;
-  for (int d = warp; d < D; d += 8)
-    for (int c = lane; c < ne; c += 32) {
-      if (pos > 0) cp_async4(S + d * per + c, Sg + (int64_t)d * E + c);
-      else S[d * per + c] = 0.f;
+  if (pos > 0 && wide) {  // whole pieces of four columns
+    const int q4 = per / 4;
+    for (int i = tid; i < D * q4; i += DL_THREADS) {
+      const int d = i / q4, c = (i - d * q4) * 4;
+      if (c < ne) cp_async16(S + d * per + c, Sg + (int64_t)d * E + c, true);
     }
+  } else {
+    for (int d = warp; d < D; d += 8)
+      for (int c = lane; c < ne; c += 32) {
+        if (pos > 0) cp_async4(S + d * per + c, Sg + (int64_t)d * E + c);
+        else S[d * per + c] = 0.f;
+      }
+  }
   cp_commit();
-  pdl_wait();
-  const int j = h / (a.heads / a.kv_heads);
+  const int group = a.heads / a.kv_heads, j = h / group;
   const HeadIn hq = head_in(a, j), hk = head_in(a, a.kv_heads + j), hv = head_in(a, 2 * a.kv_heads + h);
   float* ring = a.ring + seq * (int64_t)a.taps * C;
-  const int64_t now = (pos % a.taps) * C;
-  const bool keeps = blockIdx.x == 0 && h % (a.heads / a.kv_heads) == 0;  // this CTA writes the head's ring rows
-  float sq = 0.f, sk = 0.f;
-  for (int c = tid; c < D; c += DL_THREADS) {
-    const float xq = hq.x[r * hq.ld + c], xk = hk.x[r * hk.ld + c];
-    const float q = conv_at(a, hq, c, xq, pos, ring, C), k = conv_at(a, hk, c, xk, pos, ring, C);
-    if (keeps) ring[now + hq.ch + c] = xq, ring[now + hk.ch + c] = xk;
-    qs[c] = q, ks[c] = k;
-    sq = fmaf(q, q, sq), sk = fmaf(k, k, sk);
+  const int now = (int)(pos % a.taps), back = (int)min(pos, (int64_t)(a.taps - 1)), channels = 2 * D + ne;
+  // channel i of this CTA: q, k, its columns of v. First what the earlier inputs add to its convolution.
+  auto locate = [&](int i, int* c) -> const HeadIn& {
+    *c = i < D ? i : i < 2 * D ? i - D : e0 + i - 2 * D;
+    return i < D ? hq : i < 2 * D ? hk : hv;
+  };
+  for (int i = tid; i < channels; i += DL_THREADS) {
+    int c;
+    const HeadIn& s = locate(i, &c);
+    const int64_t w = (s.w0 + c) * a.taps + a.taps - 1, ch = s.ch + c;
+    float wt[3], x[3], u = 0.f;
+#pragma unroll
+    for (int t = 1; t <= 3; t++) {  // in flight together
+      wt[t - 1] = t <= back ? vec_at(s.w, w - t) : 0.f;
+      x[t - 1] = t <= back ? ring[(now >= t ? now - t : now - t + a.taps) * C + ch] : 0.f;
+    }
+#pragma unroll
+    for (int t = 0; t < 3; t++) u = fmaf(wt[t], x[t], u);
+    for (int t = 4; t <= back; t++) u = fmaf(vec_at(s.w, w - t), ring[(now >= t ? now - t : now - t + a.taps) * C + ch], u);
+    qs[i] = u;  // a thread's own channels until the block meets
+    w0s[i] = vec_at(s.w, w);
   }
-  for (int c = tid; c < ne; c += DL_THREADS) {
-    const float x = hv.x[r * hv.ld + e0 + c];
-    vs[c] = conv_at(a, hv, e0 + c, x, pos, ring, C);
-    ring[now + hv.ch + e0 + c] = x;
+  const float A = expf(vec_at(a.a_log, h)), dt = vec_at(a.dt, h);
+  pdl_wait();
+  const bool keeps = blockIdx.x == 0 && h % group == 0;  // this CTA writes the head's ring rows of q and k
+  float* row = ring + now * C;
+  const float zb = a.b.ptr[r * a.b.ld + h], za = a.a.ptr[r * a.a.ld + h];
+  const float* gate = a.g.ptr + r * a.g.ld + (int64_t)h * E + e0;
+  const float gate0 = tid < ne ? gate[tid] : 0.f;
+  for (int i = tid; i < channels; i += DL_THREADS) {
+    int c;
+    const HeadIn& s = locate(i, &c);
+    const float x = s.x[r * s.ld + c];
+    qs[i] = silu_of(fmaf(w0s[i], x, qs[i]));
+    if (keeps || i >= 2 * D) row[s.ch + c] = x;
   }
-  sq = block_total(sq, red8), sk = block_total(sk, red8);
-  const float iq = 1.0f / sqrtf(sq + a.unit_eps) * (1.0f / sqrtf((float)D)), ik = 1.0f / sqrtf(sk + a.unit_eps);
-  float kq = 0.f;
-  for (int c = tid; c < D; c += DL_THREADS) {
-    const float q = qs[c] * iq, k = ks[c] * ik;
-    qs[c] = q, ks[c] = k;
-    kq = fmaf(k, q, kq);
-  }
-  const float beta = sigmoid_of(a.b.ptr[r * a.b.ld + h]), g = expf(decay_log(a, h, a.a.ptr[r * a.a.ld + h]));
   cp_wait<0>();
-  kq = block_total(kq, red8);  // also publishes q, k, v and the state
-  delta_token(S, D, per, ne, ks, qs, vs, g, beta, kq, red, us, os);
-  for (int c = lane; c < ne; c += 32)  // a thread's own elements
-    for (int d = warp; d < D; d += 8) Sg[(int64_t)d * E + c] = S[d * per + c];
-  float ss = 0.f;
-  for (int c = tid; c < ne; c += DL_THREADS) ss = fmaf(os[c], os[c], ss);
-  ss = block_total(ss, red8);
-  if (tid == 0) part_ss = ss;
-  cl.sync();
+  __syncthreads();
+  if (warp < 3) {  // squared lengths and the product of q and k
+    const float *x = warp == 1 ? ks : qs, *y = warp == 0 ? qs : ks;
+    float t = 0.f;
+    for (int d = lane; d < D; d += 32) t = fmaf(x[d], y[d], t);
+    t = warp_sum(t);
+    if (lane == 0) red[warp] = t;
+  }
+  for (int c = lane; c < ne; c += 32) {
+    float rk = 0.f, rq = 0.f;
+#pragma unroll 8
+    for (int d = warp; d < D; d += 8) {
+      const float s = S[d * per + c];
+      rk = fmaf(s, ks[d], rk), rq = fmaf(s, qs[d], rq);
+    }
+    sums[warp * per + c] = rk, sums[(8 + warp) * per + c] = rq;
+  }
+  const float beta = sigmoid_of(zb), g = expf(-A * softplus_of(za + dt));
+  __syncthreads();
+  if (warp == 0) {
+    const float iq = 1.0f / sqrtf(red[0] + a.unit_eps) * (1.0f / sqrtf((float)D)), ik = 1.0f / sqrtf(red[1] + a.unit_eps);
+    float ss = 0.f;
+    for (int c = lane; c < ne; c += 32) {
+      float rk = 0.f, rq = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; w++) rk += sums[w * per + c], rq += sums[(8 + w) * per + c];
+      const float u = beta * (vs[c] - g * (rk * ik)), o = fmaf(red[2] * iq * ik, u, g * (rq * iq));
+      us[c] = u * ik, os[c] = o;
+      ss = fmaf(o, o, ss);
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) part_ss = ss;
+  }
+  __syncthreads();
+  cluster_arrive();  // the slices' sums meet while the state is written back
+  for (int c = lane; c < ne; c += 32) {
+    const float u = us[c];
+#pragma unroll 8
+    for (int d = warp; d < D; d += 8) Sg[(int64_t)d * E + c] = fmaf(g, S[d * per + c], ks[d] * u);
+  }
+  cluster_wait();
   float total = 0.f;
   for (int i = 0; i < nsplit; i++) total += *cl.map_shared_rank(&part_ss, i);
-  cl.sync();  // nobody leaves while another CTA still reads its sum
+  cluster_arrive();
   const float inv = 1.0f / sqrtf(total / (float)E + a.eps);
-  const float* gate = a.g.ptr + r * a.g.ld + (int64_t)h * E + e0;
   float* out = a.out + r * (int64_t)a.heads * E + (int64_t)h * E + e0;
-  for (int c = tid; c < ne; c += DL_THREADS) out[c] = os[c] * inv * vec_at(a.norm, e0 + c) * silu_of(gate[c]);
+  for (int c = tid; c < ne; c += DL_THREADS) out[c] = os[c] * inv * vec_at(a.norm, e0 + c) * silu_of(c == tid ? gate0 : gate[c]);
+  cluster_wait();  // nobody leaves while another CTA still reads its sum
 }
 
 constexpr int DL_MAX_SMEM = 200 * 1024;
@@ -205,9 +252,10 @@ int step_rows(const DeltaArgs& a, const int64_t* pos, const int64_t* seq, int64_
   int nsplit = 1;
   while (nsplit < 8 && (a.vdim + nsplit - 1) / nsplit > 32) nsplit *= 2;
   const int per = (a.vdim + nsplit - 1) / nsplit;
-  const size_t smem = ((size_t)a.dim * per + 2 * a.dim + 19 * per) * 4;
+  const size_t smem = ((size_t)a.dim * per + 4 * a.dim + 20 * per) * 4;
   DYN_CHECK(smem <= DL_MAX_SMEM, "delta rule: head of %d x %d is too large", a.dim, a.vdim);
   if (ensure_dynamic_smem(reinterpret_cast<const void*>(delta_step_kernel), DL_MAX_SMEM)) return 1;
+  const int wide = per % 4 == 0 && a.vdim % 4 == 0 && (reinterpret_cast<uintptr_t>(a.state) & 15) == 0;
   for (int64_t r0 = 0; r0 < rows; r0 += 65535) {
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3((unsigned)nsplit, (unsigned)a.heads, (unsigned)std::min<int64_t>(65535, rows - r0));
@@ -220,16 +268,17 @@ int step_rows(const DeltaArgs& a, const int64_t* pos, const int64_t* seq, int64_
     attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr, cfg.numAttrs = pos && pdl_enabled() ? 2 : 1;
-    DYN_CUDA(cudaLaunchKernelEx(&cfg, delta_step_kernel, a, pos, seq, pos0, seq0, r0));
+    DYN_CUDA(cudaLaunchKernelEx(&cfg, delta_step_kernel, a, pos, seq, pos0, seq0, r0, wide));
     count_launch();
   }
   return 0;
 }
 
 // ---- portions ---------------------------------------------------------------------------------
-// Scratch of a portion: convolved rows [rows][q | k | v], gates [rows][beta | log g], then the chunks' W, U, P.
+// Scratch of a portion: convolved rows [rows][q | k | v], gates [rows][beta | log g], then per chunk and head W, U, P and
+// decays [b_t | b_C / b_t].
 struct DeltaScratch {
-  float *cv, *gates, *w, *u, *p;
+  float *cv, *gates, *w, *u, *p, *decay, *end;
 };
 __host__ __device__ inline DeltaScratch carve(const DeltaArgs& a, int64_t rows) {
   const int64_t nc = (rows + DL_C - 1) / DL_C, ch = nc * a.heads;
@@ -239,6 +288,8 @@ __host__ __device__ inline DeltaScratch carve(const DeltaArgs& a, int64_t rows) 
   s.w = s.gates + (rows * 2 * a.heads + 3) / 4 * 4;
   s.u = s.w + ch * DL_C * ((a.dim + 3) / 4 * 4);
   s.p = s.u + ch * DL_C * ((a.vdim + 3) / 4 * 4);
+  s.decay = s.p + ch * DL_C * DL_C;
+  s.end = s.decay + ch * 2 * DL_C;
   return s;
 }
 
@@ -316,6 +367,93 @@ __global__ void __launch_bounds__(DL_THREADS) delta_conv_kernel(DeltaArgs a, int
   }
 }
 
+constexpr int DX_ROWS = 4;  // consecutive rows a warp convolves below
+// The same for windows of up to four taps and heads of whole groups of four channels, NV * 128 at most: a lane holds four
+// neighbouring channels, every input is in flight before the first is used, and rows leave once, in final form.
+template <int NV>
+__global__ void __launch_bounds__(DL_THREADS) delta_conv_wide_kernel(DeltaArgs a, int64_t rows, int64_t base, int64_t slot) {
+  constexpr int T = 4, NX = T + DX_ROWS - 1;
+  const DeltaScratch sc = carve(a, rows);
+  const int lane = threadIdx.x & 31;
+  const int slots = 2 * a.kv_heads + a.heads;
+  const unsigned item = blockIdx.x * 8u + (threadIdx.x >> 5), groups = (unsigned)((rows + DX_ROWS - 1) / DX_ROWS);
+  if (item >= groups * slots) return;
+  const int s = (int)(item % slots);
+  const int64_t r0 = (int64_t)(item / slots) * DX_ROWS, C = channels_of(a);
+  const HeadIn in = head_in(a, s);
+  const float* ring = a.ring + slot * (int64_t)a.taps * C;
+  const int live = (int)min((int64_t)DX_ROWS, rows - r0);
+  float4 x[NV][NX], y[NV][DX_ROWS];
+#pragma unroll
+  for (int v = 0; v < NV; v++) {
+    const int c = 128 * v + 4 * lane;
+#pragma unroll
+    for (int t = 0; t < NX; t++) {
+      const int64_t row = r0 + t - (T - 1), p = base + row;
+      x[v][t] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < in.n && t >= T - a.taps && row < rows) {
+        if (row >= 0) x[v][t] = *reinterpret_cast<const float4*>(in.x + row * in.ld + c);
+        else if (p >= 0) x[v][t] = *reinterpret_cast<const float4*>(ring + (p % a.taps) * C + in.ch + c);
+      }
+    }
+  }
+  float ss[DX_ROWS] = {};
+#pragma unroll
+  for (int v = 0; v < NV; v++) {
+    const int c = 128 * v + 4 * lane;
+    float w[4][T];
+#pragma unroll
+    for (int k = 0; k < 4; k++)
+#pragma unroll
+      for (int t = 0; t < T; t++)
+        w[k][t] = c < in.n && t >= T - a.taps ? vec_at(in.w, (in.w0 + c + k) * a.taps + t - (T - a.taps)) : 0.f;
+#pragma unroll
+    for (int i = 0; i < DX_ROWS; i++) {
+      float u[4];
+#pragma unroll
+      for (int k = 0; k < 4; k++) {
+        u[k] = 0.f;
+#pragma unroll
+        for (int t = T - 1; t >= 0; t--) {
+          const float4& q = x[v][i + t];
+          u[k] = fmaf(w[k][t], k == 0 ? q.x : k == 1 ? q.y : k == 2 ? q.z : q.w, u[k]);
+        }
+        u[k] = silu_of(u[k]);
+        ss[i] = fmaf(u[k], u[k], ss[i]);
+      }
+      y[v][i] = make_float4(u[0], u[1], u[2], u[3]);
+    }
+  }
+  if (s < 2 * a.kv_heads) {
+    const float extra = s < a.kv_heads ? 1.0f / sqrtf((float)a.dim) : 1.0f;
+#pragma unroll
+    for (int i = 0; i < DX_ROWS; i++) {
+      const float f = 1.0f / sqrtf(warp_sum(ss[i]) + a.unit_eps) * extra;
+#pragma unroll
+      for (int v = 0; v < NV; v++) y[v][i].x *= f, y[v][i].y *= f, y[v][i].z *= f, y[v][i].w *= f;
+    }
+  } else if (lane < live) {
+    const int h = s - 2 * a.kv_heads;
+    const int64_t r = r0 + lane;
+    sc.gates[r * 2 * a.heads + h] = sigmoid_of(a.b.ptr[r * a.b.ld + h]);
+    sc.gates[r * 2 * a.heads + a.heads + h] = decay_log(a, h, a.a.ptr[r * a.a.ld + h]);
+  }
+#pragma unroll
+  for (int v = 0; v < NV; v++) {
+    const int c = 128 * v + 4 * lane;
+    if (c >= in.n) continue;
+#pragma unroll
+    for (int i = 0; i < DX_ROWS; i++)
+      if (i < live) *reinterpret_cast<float4*>(sc.cv + (r0 + i) * C + in.ch + c) = y[v][i];
+  }
+}
+
+bool conv_wide(const DeltaArgs& a) {
+  auto ok = [](const Rows& r) { return r.ld % 4 == 0 && (reinterpret_cast<uintptr_t>(r.ptr) & 15) == 0; };
+  return a.taps <= 4 && a.dim % 4 == 0 && a.vdim % 4 == 0 && a.dim <= 256 && a.vdim <= 256 && ok(a.q) && ok(a.k) && ok(a.v) &&
+         (reinterpret_cast<uintptr_t>(a.ring) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.scratch) & 15) == 0;
+}
+
 // The ring after the portion; a launch after the convolutions' (they read the rows before it).
 __device__ __forceinline__ void keep_inputs(const DeltaArgs& a, int64_t rows, int64_t base, int64_t slot, int block, int blocks) {
   const int64_t C = channels_of(a), qk = (int64_t)a.kv_heads * a.dim, from = max((int64_t)0, rows - a.taps);
@@ -368,10 +506,11 @@ __global__ void __launch_bounds__(DL_THREADS) delta_tokens_kernel(DeltaArgs a, i
 }
 
 // rows x cols floats (16-byte aligned, cols % 4 == 0) into shared memory, zeros up to fill_rows x fill_cols
+template <int THREADS = DL_THREADS>
 __device__ __forceinline__ void stage(float* dst, int pitch, const float* src, int64_t ld, int rows, int cols, int fill_rows,
                                       int fill_cols) {
   const int q = fill_cols / 4;
-  for (int i = threadIdx.x; i < fill_rows * q; i += DL_THREADS) {
+  for (int i = threadIdx.x; i < fill_rows * q; i += THREADS) {
     const int r = i / q, c = (i - r * q) * 4;
     const bool live = r < rows && c < cols;
     cp_async16(dst + r * pitch + c, live ? src + r * ld + c : src, live);
@@ -441,6 +580,10 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(DeltaArgs a, in
       }
       mma3_split<4>(s, fk, b0, b1);
       mma3_split<4>(p, fq, b0, b1);
+    }
+    if (tid < DL_C) {
+      float* out = sc.decay + (c * a.heads + h) * 2 * DL_C;
+      out[tid] = expf((float)Gd[tid]), out[DL_C + tid] = expf((float)(Gd[DL_C - 1] - Gd[tid]));
     }
     float* P = sc.p + (c * a.heads + h) * DL_C * DL_C;
 #pragma unroll
@@ -536,12 +679,13 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(DeltaArgs a, in
 }
 
 constexpr int DS_N = 32;                       // value columns per CTA
+constexpr int DS_THREADS = 512;                // warps 0-7: corrections and state; 8-15: outputs
 constexpr int DS_B = DS_N + 8;                 // pitch of the split operands: conflict-free B fragments
 constexpr int DS_KP = DC_D + 8;
-constexpr int DS_SMEM = (2 * DL_C * DC_P + DL_C * DS_KP + DL_C * DC_S + 2 * DC_D * DS_B + 2 * DL_C * DS_B) * 4 + DL_C * 8;
+constexpr int DS_SMEM = (2 * DL_C * DC_P + DL_C * DS_KP + DL_C * DC_S + 2 * DC_D * DS_B + 2 * DL_C * DS_B + 4 * DL_C) * 4;
 
 // The walk over the chunks for one (value slice, head).
-__global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs a, int64_t rows, int64_t base, int64_t slot) {
+__global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a, int64_t rows, int64_t base, int64_t slot) {
   extern __shared__ __align__(16) float ds_smem[];
   const DeltaScratch sc = carve(a, rows);
   float* Ws = ds_smem;                    // [t][DC_P]
@@ -552,54 +696,59 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs a, int
   float* Sl = Sh + DC_D * DS_B;
   float* Vh = Sl + DC_D * DS_B;           // [t][DS_B] of the corrections
   float* Vl = Vh + DL_C * DS_B;
-  double* Gd = reinterpret_cast<double*>(Vl + DL_C * DS_B);
+  float* dec = Vl + DL_C * DS_B;          // [chunk parity][b_t | b_C / b_t]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
   const int D = a.dim, E = a.vdim, h = blockIdx.y, j = h / (a.heads / a.kv_heads), e0 = blockIdx.x * DS_N;
-  const int64_t C = channels_of(a), qk = (int64_t)a.kv_heads * D, nc = (rows + DL_C - 1) / DL_C;
-  keep_inputs(a, rows, base, slot, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
-  float* Sg = a.state + ((slot * a.heads + h) * D) * (int64_t)E + e0;
-  auto stage_wq = [&](int64_t c) {
-    const int n = (int)min((int64_t)DL_C, rows - c * DL_C);
-    stage(Ws, DC_P, sc.w + (c * a.heads + h) * DL_C * (int64_t)D, D, DL_C, D, DL_C, D);
-    stage(Qs, DC_P, sc.cv + c * DL_C * C + (int64_t)j * D, C, n, D, DL_C, D);
+  const int64_t C = channels_of(a), qk = (int64_t)a.kv_heads * D;
+  const int nc = (int)((rows + DL_C - 1) / DL_C);
+  auto stage_wq = [&](int c) {
+    const int n = (int)min((int64_t)DL_C, rows - (int64_t)c * DL_C);
+    const int64_t ch = (int64_t)c * a.heads + h;
+    stage<DS_THREADS>(Ws, DC_P, sc.w + ch * DL_C * D, D, DL_C, D, DL_C, D);
+    stage<DS_THREADS>(Qs, DC_P, sc.cv + (int64_t)c * DL_C * C + (int64_t)j * D, C, n, D, DL_C, D);
+    if (tid < 2 * DL_C / 4) cp_async16(dec + (c & 1) * 2 * DL_C + 4 * tid, sc.decay + ch * 2 * DL_C + 4 * tid, true);
     cp_commit();
   };
-  auto stage_kp = [&](int64_t c) {
-    const int n = (int)min((int64_t)DL_C, rows - c * DL_C);
-    stage(Ks, DS_KP, sc.cv + c * DL_C * C + qk + (int64_t)j * D, C, n, D, DL_C, D);
-    stage(Ps, DC_S, sc.p + (c * a.heads + h) * DL_C * DL_C, DL_C, DL_C, DL_C, DL_C, DL_C);
+  auto stage_kp = [&](int c) {
+    const int n = (int)min((int64_t)DL_C, rows - (int64_t)c * DL_C);
+    stage<DS_THREADS>(Ks, DS_KP, sc.cv + (int64_t)c * DL_C * C + qk + (int64_t)j * D, C, n, D, DL_C, D);
+    stage<DS_THREADS>(Ps, DC_S, sc.p + ((int64_t)c * a.heads + h) * DL_C * DL_C, DL_C, DL_C, DL_C, DL_C, DL_C);
     cp_commit();
   };
   stage_wq(0);
   stage_kp(0);
-  // the warp's 16 rows of the state, as accumulators
-  const int d0 = 16 * warp;
-  float S[4][4];
+  keep_inputs(a, rows, base, slot, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
+  const int mt = warp & 3, nh = (warp >> 2) & 1;  // 16 tokens x 16 value columns
+  const bool states = warp < 8;
+  // warps 0-7: 16 rows of the state as accumulators
+  float* Sg = a.state + ((slot * a.heads + h) * D) * (int64_t)E + e0;
+  const int d0 = 16 * (warp & 7);
+  const bool owns = states && d0 < D;
+  float S[4][4] = {};
+  if (owns && base > 0) {
 #pragma unroll
-  for (int nt = 0; nt < 4; nt++)
+    for (int nt = 0; nt < 4; nt++)
 #pragma unroll
-    for (int i = 0; i < 4; i++) {
-      const int d = d0 + g + 8 * (i >> 1), e = 8 * nt + 2 * t4 + (i & 1);
-      S[nt][i] = base > 0 && d < D && e0 + e < E ? Sg[(int64_t)d * E + e] : 0.f;
-    }
-  const int mt = warp & 3, nh = warp >> 2;  // 16 tokens x 16 value columns
-  for (int64_t c = 0; c < nc; c++) {
-    const int64_t t0 = c * DL_C;
-    const int n = (int)min((int64_t)DL_C, rows - t0);
-    if (d0 < D) {
+      for (int i = 0; i < 4; i++) {
+        const int d = d0 + g + 8 * (i >> 1), e = 8 * nt + 2 * t4 + (i & 1);
+        if (d < D && e0 + e < E) S[nt][i] = Sg[(int64_t)d * E + e];
+      }
+  }
+  auto publish = [&]() {
 #pragma unroll
-      for (int nt = 0; nt < 4; nt++)
+    for (int nt = 0; nt < 4; nt++)
 #pragma unroll
-        for (int i = 0; i < 4; i++) {
-          const int d = d0 + g + 8 * (i >> 1), e = 8 * nt + 2 * t4 + (i & 1);
-          const Tf32Pair p = tf32_split(S[nt][i]);
-          Sh[d * DS_B + e] = __uint_as_float(p.hi), Sl[d * DS_B + e] = __uint_as_float(p.lo);
-        }
-    }
-    if (warp == 0) chunk_decay(a, sc.gates, t0, n, h, Gd, nullptr);
-    // U of the warp's tile, on its way while W and Q arrive
-    float uv[2][4];
-    const float* U = sc.u + (c * a.heads + h) * DL_C * (int64_t)E + e0;
+      for (int i = 0; i < 4; i += 2) {
+        const int d = d0 + g + 4 * i, e = 8 * nt + 2 * t4;
+        const Tf32Pair p = tf32_split(S[nt][i]), q = tf32_split(S[nt][i + 1]);
+        *reinterpret_cast<float2*>(Sh + d * DS_B + e) = make_float2(__uint_as_float(p.hi), __uint_as_float(q.hi));
+        *reinterpret_cast<float2*>(Sl + d * DS_B + e) = make_float2(__uint_as_float(p.lo), __uint_as_float(q.lo));
+      }
+  };
+  if (owns) publish();
+  float uv[2][4] = {};  // U of the warp's tile, fetched a chunk ahead
+  auto fetch_u = [&](int c) {
+    const float* U = sc.u + ((int64_t)c * a.heads + h) * DL_C * E + e0;
 #pragma unroll
     for (int nt = 0; nt < 2; nt++)
 #pragma unroll
@@ -608,88 +757,99 @@ __global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(DeltaArgs a, int
         const float2 v = e0 + e < E ? *reinterpret_cast<const float2*>(U + t * (int64_t)E + e) : make_float2(0.f, 0.f);
         uv[nt][2 * i] = v.x, uv[nt][2 * i + 1] = v.y;
       }
+  };
+  if (states) fetch_u(0);
+  auto split_at = [&](const float* hi, const float* lo, int k, int col, Tf32Pair& b0, Tf32Pair& b1) {
+    const int at = (k + t4) * DS_B + col;
+    b0.hi = __float_as_uint(hi[at]), b0.lo = __float_as_uint(lo[at]);
+    b1.hi = __float_as_uint(hi[at + 4 * DS_B]), b1.lo = __float_as_uint(lo[at + 4 * DS_B]);
+  };
+  for (int c = 0; c < nc; c++) {
+    const int64_t t0 = (int64_t)c * DL_C;
+    const int n = (int)min((int64_t)DL_C, rows - t0);
+    const float* bt = dec + (c & 1) * 2 * DL_C;
     cp_wait<1>();
-    __syncthreads();
-    // ---- W S and Q S
-    float ws[2][4] = {}, o[2][4] = {};
-#pragma unroll 2
-    for (int d = 0; d < D; d += 8) {
-      AFrag fw, fq;
-      load_a(fw, Ws + (16 * mt + g) * DC_P + d + t4, DC_P);
-      load_a(fq, Qs + (16 * mt + g) * DC_P + d + t4, DC_P);
-      Tf32Pair b0[2], b1[2];
+    __syncthreads();  // W, Q, the decays and the state's terms are there
+    // ---- W S, Q S
+    float acc[2][4] = {};
+    {
+      const float* A = (states ? Ws : Qs) + (16 * mt + g) * DC_P + t4;
+#pragma unroll 4
+      for (int d = 0; d < D; d += 8) {
+        AFrag f;
+        load_a(f, A + d, DC_P);
+        Tf32Pair b0[2], b1[2];
 #pragma unroll
-      for (int nt = 0; nt < 2; nt++) {
-        const int at = (d + t4) * DS_B + nh * 16 + 8 * nt + g;
-        b0[nt].hi = __float_as_uint(Sh[at]), b0[nt].lo = __float_as_uint(Sl[at]);
-        b1[nt].hi = __float_as_uint(Sh[at + 4 * DS_B]), b1[nt].lo = __float_as_uint(Sl[at + 4 * DS_B]);
+        for (int nt = 0; nt < 2; nt++) split_at(Sh, Sl, d, nh * 16 + 8 * nt + g, b0[nt], b1[nt]);
+        mma3_split<2>(acc, f, b0, b1);
       }
-      mma3_split<2>(ws, fw, b0, b1);
-      mma3_split<2>(o, fq, b0, b1);
     }
-    const float w0 = expf((float)Gd[16 * mt + g]), w1 = expf((float)Gd[16 * mt + g + 8]);
+    if (states) {
 #pragma unroll
-    for (int nt = 0; nt < 2; nt++)
+      for (int nt = 0; nt < 2; nt++)
 #pragma unroll
-      for (int i = 0; i < 4; i++) {
-        const int t = 16 * mt + g + 8 * (i >> 1), e = nh * 16 + 8 * nt + 2 * t4 + (i & 1);
-        const Tf32Pair p = tf32_split(uv[nt][i] - ws[nt][i]);
-        Vh[t * DS_B + e] = __uint_as_float(p.hi), Vl[t * DS_B + e] = __uint_as_float(p.lo);
-        o[nt][i] *= i < 2 ? w0 : w1;
-      }
+        for (int i = 0; i < 4; i += 2) {
+          const int t = 16 * mt + g + 4 * i, e = nh * 16 + 8 * nt + 2 * t4;
+          const Tf32Pair p = tf32_split(uv[nt][i] - acc[nt][i]), q = tf32_split(uv[nt][i + 1] - acc[nt][i + 1]);
+          *reinterpret_cast<float2*>(Vh + t * DS_B + e) = make_float2(__uint_as_float(p.hi), __uint_as_float(q.hi));
+          *reinterpret_cast<float2*>(Vl + t * DS_B + e) = make_float2(__uint_as_float(p.lo), __uint_as_float(q.lo));
+        }
+      if (c + 1 < nc) fetch_u(c + 1);
+    }
     cp_wait<0>();
-    __syncthreads();  // V, K and P are there; W and Q are read
+    __syncthreads();  // corrections, K and P are there; W, Q and the state's terms are read
     if (c + 1 < nc) stage_wq(c + 1);
-    auto v_pair = [&](Tf32Pair& b0, Tf32Pair& b1, int k, int col) {
-      const int at = (k + t4) * DS_B + col;
-      b0.hi = __float_as_uint(Vh[at]), b0.lo = __float_as_uint(Vl[at]);
-      b1.hi = __float_as_uint(Vh[at + 4 * DS_B]), b1.lo = __float_as_uint(Vl[at + 4 * DS_B]);
-    };
-    // ---- o += P V (P is lower triangular)
-    for (int k = 0; k < 16 * (mt + 1); k += 8) {
-      AFrag f;
-      load_a(f, Ps + (16 * mt + g) * DC_S + k + t4, DC_S);
-      Tf32Pair b0[2], b1[2];
-#pragma unroll
-      for (int nt = 0; nt < 2; nt++) v_pair(b0[nt], b1[nt], k, nh * 16 + 8 * nt + g);
-      mma3_split<2>(o, f, b0, b1);
-    }
-#pragma unroll
-    for (int i = 0; i < 2; i++) {
-      const int t = 16 * mt + g + 8 * i;
-      if (t >= n) continue;
-      float* out = a.out + (t0 + t) * (int64_t)a.heads * E + (int64_t)h * E + e0;
-#pragma unroll
-      for (int nt = 0; nt < 2; nt++) {
-        const int e = nh * 16 + 8 * nt + 2 * t4;
-        if (e0 + e < E) *reinterpret_cast<float2*>(out + e) = make_float2(o[nt][2 * i], o[nt][2 * i + 1]);
-      }
-    }
-    // ---- S <- b_C S + (K b_C / b)^T V
-    if (d0 < D) {
-      const double last = Gd[DL_C - 1];
-      const float full = expf((float)last);
+    if (owns) {
+      // ---- S <- b_C S + (K b_C / b)^T V
+      const float full = bt[DL_C - 1];
+      const bool second = d0 + 8 < D;
 #pragma unroll
       for (int nt = 0; nt < 4; nt++)
 #pragma unroll
         for (int i = 0; i < 4; i++) S[nt][i] *= full;
 #pragma unroll 2
       for (int k = 0; k < DL_C; k += 8) {
-        const float wa = expf((float)(last - Gd[k + t4])), wb = expf((float)(last - Gd[k + t4 + 4]));
+        const float wa = bt[DL_C + k + t4], wb = bt[DL_C + k + t4 + 4];
         const float *ka = Ks + (k + t4) * DS_KP + d0 + g, *kb = ka + 4 * DS_KP;
-        const bool second = d0 + 8 < D;
         AFrag f;
         split_into(f, 0, ka[0] * wa), split_into(f, 1, second ? ka[8] * wa : 0.f);
         split_into(f, 2, kb[0] * wb), split_into(f, 3, second ? kb[8] * wb : 0.f);
         Tf32Pair b0[4], b1[4];
 #pragma unroll
-        for (int nt = 0; nt < 4; nt++) v_pair(b0[nt], b1[nt], k, 8 * nt + g);
+        for (int nt = 0; nt < 4; nt++) split_at(Vh, Vl, k, 8 * nt + g, b0[nt], b1[nt]);
         mma3_split<4>(S, f, b0, b1);
       }
+      publish();
+    } else if (!states) {
+      // ---- o = b Q S + P V (P is lower triangular)
+      const float w0 = bt[16 * mt + g], w1 = bt[16 * mt + g + 8];
+#pragma unroll
+      for (int nt = 0; nt < 2; nt++) acc[nt][0] *= w0, acc[nt][1] *= w0, acc[nt][2] *= w1, acc[nt][3] *= w1;
+#pragma unroll 2
+      for (int k = 0; k < 16 * (mt + 1); k += 8) {
+        AFrag f;
+        load_a(f, Ps + (16 * mt + g) * DC_S + k + t4, DC_S);
+        Tf32Pair b0[2], b1[2];
+#pragma unroll
+        for (int nt = 0; nt < 2; nt++) split_at(Vh, Vl, k, nh * 16 + 8 * nt + g, b0[nt], b1[nt]);
+        mma3_split<2>(acc, f, b0, b1);
+      }
+#pragma unroll
+      for (int i = 0; i < 2; i++) {
+        const int t = 16 * mt + g + 8 * i;
+        if (t >= n) continue;
+        float* out = a.out + (t0 + t) * (int64_t)a.heads * E + (int64_t)h * E + e0;
+#pragma unroll
+        for (int nt = 0; nt < 2; nt++) {
+          const int e = nh * 16 + 8 * nt + 2 * t4;
+          if (e0 + e < E) *reinterpret_cast<float2*>(out + e) = make_float2(acc[nt][2 * i], acc[nt][2 * i + 1]);
+        }
+      }
     }
-    __syncthreads();  // K, P, V and the decays are read
+    __syncthreads();  // K, P and the corrections are read
     if (c + 1 < nc) stage_kp(c + 1);
   }
+  if (!owns) return;
 #pragma unroll
   for (int nt = 0; nt < 4; nt++)
 #pragma unroll
@@ -713,6 +873,49 @@ __global__ void __launch_bounds__(DL_THREADS) delta_finish_kernel(DeltaArgs a, i
   for (int e = lane; e < E; e += 32) out[e] = out[e] * inv * vec_at(a.norm, e) * silu_of(gate[e]);
 }
 
+// CTA = row; a warp takes heads in turn. f16 values scaled by a power of two that puts the row's largest magnitude in
+// [2^12, 2^13), as the GEMM's own activation pass does.
+__global__ void __launch_bounds__(DL_THREADS) delta_finish_operand_kernel(DeltaArgs a) {
+  extern __shared__ __align__(16) float df_row[];  // [heads * vdim]
+  __shared__ float red[8];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, E = a.vdim, total = a.heads * E;
+  const int64_t r = blockIdx.x;
+  const float* o = a.out + r * total;
+  const float* gate = a.g.ptr + r * a.g.ld;
+  float mx = 0.f;
+  for (int h = warp; h < a.heads; h += 8) {
+    float v[8], z[8], ss = 0.f;  // vdim <= 256
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+      const int e = lane + 32 * i;
+      v[i] = e < E ? o[h * E + e] : 0.f, z[i] = e < E ? gate[h * E + e] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < 8; i++) ss = fmaf(v[i], v[i], ss);
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)E + a.eps);
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+      const int e = lane + 32 * i;
+      if (e >= E) continue;
+      const float y = v[i] * inv * vec_at(a.norm, e) * silu_of(z[i]);
+      df_row[h * E + e] = y;
+      mx = fmaxf(mx, fabsf(y));
+    }
+  }
+  mx = warp_max(mx);
+  if (lane == 0) red[warp] = mx;
+  __syncthreads();
+  mx = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; w++) mx = fmaxf(mx, red[w]);
+  int e = 0;
+  if (mx > 0.f && mx < 3.0e38f) frexpf(mx, &e);
+  const float sc = ldexpf(1.0f, 13 - e);
+  if (tid == 0) a.xinv[r] = ldexpf(1.0f, e - 13);
+  for (int i = tid * 2; i < total; i += DL_THREADS * 2)
+    *reinterpret_cast<__half2*>(a.xh + r * total + i) = __floats2half2_rn(df_row[i] * sc, df_row[i + 1] * sc);
+}
+
 bool chunk_shape(const DeltaArgs& a, int64_t rows) {
   return !a.exact && rows > DL_FEW && a.dim <= DC_D && a.dim % 8 == 0 && a.vdim % 8 == 0;
 }
@@ -722,9 +925,12 @@ bool chunk_shape(const DeltaArgs& a, int64_t rows) {
 size_t delta_scratch_floats(const DeltaArgs& a, int64_t rows) {
   DeltaArgs z = a;
   z.scratch = nullptr;
-  const int64_t nc = (rows + DL_C - 1) / DL_C;
-  const size_t small = carve(z, rows).w - z.scratch;
-  return chunk_shape(a, rows) ? (size_t)(carve(z, rows).p - z.scratch) + (size_t)nc * a.heads * DL_C * DL_C : small;
+  const DeltaScratch s = carve(z, rows);
+  return (chunk_shape(a, rows) ? s.end : s.w) - s.cv;
+}
+
+bool delta_writes_operand(const DeltaArgs& a) {
+  return a.vdim <= 256 && a.heads * a.vdim % 2 == 0 && (size_t)a.heads * a.vdim * 4 <= DL_MAX_SMEM;
 }
 
 int launch_delta(const DeltaArgs& a, const StepRows& r, cudaStream_t st) {
@@ -732,17 +938,20 @@ int launch_delta(const DeltaArgs& a, const StepRows& r, cudaStream_t st) {
   DYN_CHECK(a.kv_heads > 0 && a.heads % a.kv_heads == 0, "delta rule: %d heads over %d q/k heads", a.heads, a.kv_heads);
   if (r.base < 0) return step_rows(a, r.pos, r.seq, 0, 0, r.rows, st);
   if (r.rows == 1) return step_rows(a, nullptr, nullptr, r.base, r.slot, 1, st);
-  const int64_t items = (r.rows + DV_ROWS - 1) / DV_ROWS * (2 * a.kv_heads + a.heads);
+  const bool wide = conv_wide(a);
+  const int64_t per = wide ? DX_ROWS : DV_ROWS, items = (r.rows + per - 1) / per * (2 * a.kv_heads + a.heads);
   const unsigned grid = (unsigned)((items + 7) / 8);
-  if (a.taps <= 4) delta_conv_kernel<4><<<grid, DL_THREADS, 0, st>>>(a, r.rows, r.base, r.slot);
-  else delta_conv_kernel<0><<<grid, DL_THREADS, 0, st>>>(a, r.rows, r.base, r.slot);
+  const auto conv = wide          ? (std::max(a.dim, a.vdim) <= 128 ? delta_conv_wide_kernel<1> : delta_conv_wide_kernel<2>)
+                    : a.taps <= 4 ? delta_conv_kernel<4>
+                                  : delta_conv_kernel<0>;
+  conv<<<grid, DL_THREADS, 0, st>>>(a, r.rows, r.base, r.slot);
   if (chunk_shape(a, r.rows)) {
     const unsigned nc = (unsigned)((r.rows + DL_C - 1) / DL_C);
     if (ensure_dynamic_smem(reinterpret_cast<const void*>(delta_chunk_kernel), DC_SMEM) ||
         ensure_dynamic_smem(reinterpret_cast<const void*>(delta_scan_kernel), DS_SMEM))
       return 1;
     delta_chunk_kernel<<<dim3(nc, (unsigned)a.heads), DL_THREADS, DC_SMEM, st>>>(a, r.rows);
-    delta_scan_kernel<<<dim3((unsigned)((a.vdim + DS_N - 1) / DS_N), (unsigned)a.heads), DL_THREADS, DS_SMEM, st>>>(
+    delta_scan_kernel<<<dim3((unsigned)((a.vdim + DS_N - 1) / DS_N), (unsigned)a.heads), DS_THREADS, DS_SMEM, st>>>(
         a, r.rows, r.base, r.slot);
     count_launch(2);
   } else {
@@ -754,7 +963,13 @@ int launch_delta(const DeltaArgs& a, const StepRows& r, cudaStream_t st) {
     delta_tokens_kernel<<<dim3((unsigned)nsplit, (unsigned)a.heads), DL_THREADS, smem, st>>>(a, r.rows, r.base, r.slot);
     count_launch();
   }
-  delta_finish_kernel<<<(unsigned)((r.rows * a.heads + 7) / 8), DL_THREADS, 0, st>>>(a, r.rows);
+  if (a.xh) {
+    DYN_CHECK(delta_writes_operand(a), "delta rule: no operand of %d heads of %d", a.heads, a.vdim);
+    if (ensure_dynamic_smem(reinterpret_cast<const void*>(delta_finish_operand_kernel), DL_MAX_SMEM)) return 1;
+    delta_finish_operand_kernel<<<(unsigned)r.rows, DL_THREADS, (size_t)a.heads * a.vdim * 4, st>>>(a);
+  } else {
+    delta_finish_kernel<<<(unsigned)((r.rows * a.heads + 7) / 8), DL_THREADS, 0, st>>>(a, r.rows);
+  }
   count_launch(2);
   DYN_CUDA(cudaGetLastError());
   return 0;

@@ -149,7 +149,7 @@ template <int PER>
 __global__ void __launch_bounds__(256)
 norm_prepare_kernel(const float* __restrict__ x, const float* __restrict__ partial, int S, int64_t rows,
                     const float* residual, float* hidden, const void* __restrict__ w, int w_type, int64_t width,
-                    float eps, __half* __restrict__ xh, float* __restrict__ inv_s) {
+                    float eps, __half* __restrict__ xh, float* __restrict__ inv_s, NormPair pair) {
   __shared__ float red[32];
   const int64_t row = blockIdx.x;
   float v[PER], wv[PER];
@@ -185,42 +185,51 @@ norm_prepare_kernel(const float* __restrict__ x, const float* __restrict__ parti
   for (int k = 0; k < PER; k++) {
     const int64_t i = threadIdx.x + (int64_t)k * blockDim.x;
     wv[k] = i < width ? aux_load(reinterpret_cast<const uint8_t*>(w), w_type, i) : 0.f;
-    if (hidden && i < width) hidden[row * width + i] = v[k];
+    if (hidden && i < width)
+      hidden[row * width + i] = pair.bias ? v[k] + aux_load(reinterpret_cast<const uint8_t*>(pair.bias), pair.bias_type, i) : v[k];
   }
   float ss = 0.f;
 #pragma unroll
   for (int k = 0; k < PER; k++) ss = fmaf(v[k], v[k], ss);  // absent elements add +0
   ss = block_sum(ss, red);
   const float inv = 1.0f / sqrtf(ss / (float)width + eps);
-  float mx = 0.f;
 #pragma unroll
-  for (int k = 0; k < PER; k++) {
-    v[k] = __fmul_rn(__fmul_rn(v[k], inv), wv[k]);
-    mx = fmaxf(mx, fabsf(v[k]));
-  }
-  float sc, is;
-  f16_row_scale(mx, red, &sc, &is);
-  if (threadIdx.x == 0) inv_s[row] = is;
+  for (int k = 0; k < PER; k++) v[k] = __fmul_rn(v[k], inv);
+  auto leave = [&](__half* out, float* inv_out) {  // v * wv
+    float mx = 0.f, sc, is;
+#pragma unroll
+    for (int k = 0; k < PER; k++) mx = fmaxf(mx, fabsf(__fmul_rn(v[k], wv[k])));
+    f16_row_scale(mx, red, &sc, &is);
+    if (threadIdx.x == 0) inv_out[row] = is;
+#pragma unroll
+    for (int k = 0; k < PER; k++) {
+      const int64_t i = threadIdx.x + (int64_t)k * blockDim.x;
+      if (i < width) out[row * width + i] = __float2half_rn(__fmul_rn(v[k], wv[k]) * sc);
+    }
+  };
+  leave(xh, inv_s);
+  if (!pair.w) return;
 #pragma unroll
   for (int k = 0; k < PER; k++) {
     const int64_t i = threadIdx.x + (int64_t)k * blockDim.x;
-    if (i < width) xh[row * width + i] = __float2half_rn(v[k] * sc);
+    wv[k] = i < width ? aux_load(reinterpret_cast<const uint8_t*>(pair.w), pair.type, i) : 0.f;
   }
+  leave(pair.xh, pair.inv_s);
 }
 
 int launch_norm_prepare(const float* x, const float* partial, int splits, const float* residual, float* hidden,
                         const void* w, int w_type, int64_t rows, int64_t width, float eps, __half* xh, float* inv_s,
-                        cudaStream_t s) {
+                        cudaStream_t s, const NormPair& pair) {
   if (rows == 0) return 0;
   const int threads = width >= 1024 ? 256 : (width >= 256 ? 128 : 32);  // rms_norm_kernel's: same summation order
   DYN_CHECK(width <= 32 * threads, "row of %lld elements is too wide for the fused RMSNorm", (long long)width);
   const int S = splits > 1 ? splits : 0;
   if (width <= 8 * threads)
-    norm_prepare_kernel<8><<<(unsigned)rows, threads, 0, s>>>(x, partial, S, rows, residual, hidden, w, w_type, width, eps, xh, inv_s);
+    norm_prepare_kernel<8><<<(unsigned)rows, threads, 0, s>>>(x, partial, S, rows, residual, hidden, w, w_type, width, eps, xh, inv_s, pair);
   else if (width <= 16 * threads)
-    norm_prepare_kernel<16><<<(unsigned)rows, threads, 0, s>>>(x, partial, S, rows, residual, hidden, w, w_type, width, eps, xh, inv_s);
+    norm_prepare_kernel<16><<<(unsigned)rows, threads, 0, s>>>(x, partial, S, rows, residual, hidden, w, w_type, width, eps, xh, inv_s, pair);
   else
-    norm_prepare_kernel<32><<<(unsigned)rows, threads, 0, s>>>(x, partial, S, rows, residual, hidden, w, w_type, width, eps, xh, inv_s);
+    norm_prepare_kernel<32><<<(unsigned)rows, threads, 0, s>>>(x, partial, S, rows, residual, hidden, w, w_type, width, eps, xh, inv_s, pair);
   count_launch();
   DYN_CUDA(cudaGetLastError());
   return 0;
@@ -693,27 +702,46 @@ attention_split_kernel(AttnArgs a, float* __restrict__ part, int nsplit) {
   if (threadIdx.x == 0) out[d] = gm, out[d + 1] = gl;
 }
 
+constexpr int ATT_MAX_SPLIT = 128;
 __global__ void __launch_bounds__(256)
 attention_merge_kernel(const float* __restrict__ part, int nsplit, float* ctx, int64_t nh, int64_t d) {
+  __shared__ float s_w[ATT_MAX_SPLIT], s_l[ATT_MAX_SPLIT];
   pdl_trigger();  // a product launched next may begin fetching its weights
+  pdl_wait();
   const int64_t h = blockIdx.x, r = blockIdx.y;
   const float* p0 = part + ((r * nh + h) * nsplit) * (d + 2);
-  float gm = -3.40282347e38f;
-  for (int s = 0; s < nsplit; s++) gm = fmaxf(gm, p0[s * (d + 2) + d]);
+  if (threadIdx.x < 32) {
+    float m[ATT_MAX_SPLIT / 32], gm = -3.40282347e38f;
+#pragma unroll
+    for (int j = 0; j < ATT_MAX_SPLIT / 32; j++) {
+      const int s = threadIdx.x + 32 * j;
+      m[j] = s < nsplit ? p0[s * (d + 2) + d] : -3.40282347e38f;
+      if (s < nsplit) s_l[s] = p0[s * (d + 2) + d + 1];
+      gm = fmaxf(gm, m[j]);
+    }
+    gm = warp_max(gm);
+#pragma unroll
+    for (int j = 0; j < ATT_MAX_SPLIT / 32; j++)
+      if (threadIdx.x + 32 * j < nsplit) s_w[threadIdx.x + 32 * j] = expf(m[j] - gm);  // an empty slice has sum 0 and contributes nothing
+  }
+  __syncthreads();
   for (int64_t idx = threadIdx.x; idx < d; idx += blockDim.x) {
     float o = 0.f, gl = 0.f;
-    for (int s = 0; s < nsplit; s++) {
-      const float* ps = p0 + s * (d + 2);
-      const float w = expf(ps[d] - gm);  // an empty slice has sum 0 and contributes nothing
-      o += ps[idx] * w;
-      gl += ps[d + 1] * w;
+    for (int s0 = 0; s0 < nsplit; s0 += 8) {  // eight slices' loads in flight
+      float v[8];
+#pragma unroll
+      for (int j = 0; j < 8; j++) v[j] = s0 + j < nsplit ? p0[(s0 + j) * (d + 2) + idx] : 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; j++)
+        if (s0 + j < nsplit) o += v[j] * s_w[s0 + j], gl += s_l[s0 + j] * s_w[s0 + j];
     }
     ctx[r * nh * d + h * d + idx] = o / gl;
   }
 }
 
 int launch_attention_merge(const float* part, int nsplit, float* ctx, int64_t rows, int64_t nh, int64_t d, cudaStream_t s) {
-  attention_merge_kernel<<<dim3((unsigned)nh, (unsigned)rows), 256, 0, s>>>(part, nsplit, ctx, nh, d);
+  DYN_CHECK(nsplit <= ATT_MAX_SPLIT, "attention: %d slices are too many", nsplit);
+  DYN_CUDA(launch_pdl(attention_merge_kernel, dim3((unsigned)nh, (unsigned)rows), dim3(d <= 128 ? 128 : 256), 0, s, part, nsplit, ctx, nh, d));
   count_launch();
   DYN_CUDA(cudaGetLastError());
   return 0;

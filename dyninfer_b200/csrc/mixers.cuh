@@ -126,9 +126,12 @@ struct DeltaArgs {
   float* ring = nullptr;          // [slot][taps][q | k | v channels]: convolution input of position p in row p mod taps
   float* out = nullptr;           // [rows, heads * vdim]
   float* scratch = nullptr;       // delta_scratch_floats
+  __half* xh = nullptr;           // portions of several rows: the output as the dequant GEMM's operand instead of f32
+  float* xinv = nullptr;
   float eps = 0.f, unit_eps = 1e-6f;
   bool exact = false;             // f32 products only
 };
+bool delta_writes_operand(const DeltaArgs& a);
 size_t delta_scratch_floats(const DeltaArgs& a, int64_t rows);
 int launch_delta(const DeltaArgs& a, const StepRows& r, cudaStream_t st);
 
@@ -144,6 +147,7 @@ struct MoeArgs {
   const uint8_t* const* table = nullptr;    // device, [experts][gate, up, down]
   // device, [experts]: [gate; up] as one matrix each (nullptr: not laid back to back), down
   const uint8_t* const *gate_up_table = nullptr, *const* down_table = nullptr;
+  const void* maps = nullptr;               // device, tensor maps of f16 matrices [experts][gate, up, down] (nullptr: none)
   WRef shared_gate, shared_up, shared_down;
   float* scratch = nullptr;                 // moe_scratch_floats; the router logits [rows, experts] come first
   bool exact = false;

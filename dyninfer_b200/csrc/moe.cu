@@ -5,8 +5,9 @@
 // A few rows: two launches stream the chosen experts' weights (moe_up_kernel, moe_down_kernel); every CTA picks
 // its experts from the logits itself. Scaling the input of gate and up scales their sums, so the score multiplies those.
 // More rows: (row, choice) pairs are sorted by expert (moe_plan_kernel; a fixed order, so results do not depend on
-// timing), then grouped products run on the tensor cores (the grouped form of the dequant GEMM), or in f32 for f32
-// sessions and shapes the GEMM does not take; moe_combine_kernel adds each row's outputs in the order of its choices.
+// timing), then grouped products run on the tensor cores: f16 matrices by tile copies (gemm_grouped.cu; a session turns bf16
+// experts into f16 when their range allows it), others through the grouped form of the dequant GEMM, and in f32 for f32
+// sessions and shapes the GEMMs do not take; moe_combine_kernel adds each row's outputs in the order of its choices.
 #include <algorithm>
 
 #include "mixers.cuh"
@@ -129,15 +130,18 @@ __global__ void __launch_bounds__(MO_THREADS) moe_up_kernel(MoeArgs a, const flo
   }
 }
 
-constexpr int MD_OUT = 2;
-// hidden[row][n] += sum over the slots of down[n] . act
+constexpr int MD_THREADS = 1024, MD_WARPS = MD_THREADS / 32, MD_DEPTH = 8, MD_SPAN = 32 * MD_DEPTH;
+// hidden[row][n] += sum over the slots of down[n] . act. A CTA owns a block of outputs; their rows, all slots one after the
+// other, are cut into spans of MD_SPAN pieces of eight, dealt to the warps.
 template <bool BF16>
-__global__ void __launch_bounds__(MO_THREADS) moe_down_kernel(MoeArgs a, const float* __restrict__ z, const float* __restrict__ act, float* hidden) {
-  extern __shared__ __align__(16) float md_x[];  // planes over all slots' activations, one after the other
+__global__ void __launch_bounds__(MD_THREADS, 1) moe_down_kernel(MoeArgs a, const float* __restrict__ z, const float* __restrict__ act, float* hidden) {
+  extern __shared__ __align__(16) float md_x[];  // planes over all slots' activations, one after the other; then sums
   __shared__ const uint8_t* s_base[64];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int slots = a.top + (a.shared_ff ? 1 : 0), wide = max(a.ff, a.shared_ff), total = a.top * a.ff + a.shared_ff, T8 = total / 8;
   const int64_t r = blockIdx.y, W = a.width;
+  const int64_t out0 = W * blockIdx.x / gridDim.x;
+  const int own = (int)(W * (blockIdx.x + 1) / gridDim.x - out0), parts = (T8 + MD_SPAN - 1) / MD_SPAN;
   pdl_trigger();
   pdl_wait();
   if (warp == 0) {
@@ -146,43 +150,39 @@ __global__ void __launch_bounds__(MO_THREADS) moe_down_kernel(MoeArgs a, const f
     });
     if (lane == 0 && a.shared_ff) s_base[a.top] = a.shared_down.data;
   }
-  for (int i = tid; i < total; i += MO_THREADS) {
+  for (int i = tid; i < total; i += MD_THREADS) {
     const int slot = min(i / a.ff, a.top), f = i - slot * a.ff;
     plane_at(md_x, i, T8) = act[(r * slots + slot) * wide + f];
   }
   __syncthreads();
   const float4* xs = reinterpret_cast<const float4*>(md_x);
-  const int64_t n0 = ((int64_t)blockIdx.x * MO_WARPS + warp) * MD_OUT;
-  if (n0 >= W) return;
-  float sum[MD_OUT] = {};
-  constexpr int U = 4;
-  const int ff8 = a.ff / 8;
-  for (int p0 = lane; p0 < T8; p0 += 32 * U) {
-    uint4 w[MD_OUT][U];
+  float* sums = md_x + total;  // [own][parts]
+  const unsigned ff8 = a.ff / 8;
+  for (int unit = warp; unit < own * parts; unit += MD_WARPS) {
+    const int o = unit / parts, p0 = (unit - o * parts) * MD_SPAN + lane;
+    uint4 w[MD_DEPTH];
 #pragma unroll
-    for (int u = 0; u < U; u++) {
+    for (int u = 0; u < MD_DEPTH; u++) {
       const int p = p0 + 32 * u;
       if (p < T8) {
-        const int slot = min(p / ff8, a.top), k = p - slot * ff8;
-        const int64_t ld = slot < a.top ? a.ff : a.shared_ff;
-#pragma unroll
-        for (int o = 0; o < MD_OUT; o++)
-          w[o][u] = __ldcs(reinterpret_cast<const uint4*>(s_base[slot] + min(n0 + o, W - 1) * ld * 2) + k);
+        const int slot = min((int)((unsigned)p / ff8), a.top), k = p - slot * (int)ff8;
+        w[u] = __ldcs(reinterpret_cast<const uint4*>(s_base[slot] + (out0 + o) * (slot < a.top ? a.ff : a.shared_ff) * 2) + k);
       }
     }
+    float sum = 0.f;
 #pragma unroll
-    for (int u = 0; u < U; u++) {
+    for (int u = 0; u < MD_DEPTH; u++) {
       const int p = p0 + 32 * u;
-      if (p >= T8) break;
-      const float4 xa = xs[p], xb = xs[T8 + p];
-#pragma unroll
-      for (int o = 0; o < MD_OUT; o++) sum[o] += dot8<BF16>(w[o][u], xa, xb);
+      if (p < T8) sum += dot8<BF16>(w[u], xs[p], xs[T8 + p]);
     }
+    sum = warp_sum(sum);
+    if (lane == 0) sums[unit] = sum;
   }
-#pragma unroll
-  for (int o = 0; o < MD_OUT; o++) {
-    const float v = warp_sum(sum[o]);
-    if (lane == 0 && n0 + o < W) hidden[r * W + n0 + o] += v;
+  __syncthreads();
+  for (int o = tid; o < own; o += MD_THREADS) {
+    float v = 0.f;
+    for (int p = 0; p < parts; p++) v += sums[o * parts + p];
+    hidden[r * W + out0 + o] += v;
   }
 }
 
@@ -344,17 +344,15 @@ size_t up256(size_t n) { return (n + 255) / 256 * 256; }
 
 int tile_rows(const MoeArgs& a, int64_t rows, bool tensor) {
   if (!tensor) return MG_T;
-  // one tile per expert for an even spread with some slack
-  const int64_t want = rows * a.top * 5 / (4 * a.experts) + 1;
-  int bn = 16;
-  while (bn < 256 && bn < want) bn *= 2;
-  return bn;
+  // one tile per expert up to twice the even share: the tile-copy GEMM's tiles cost what their rows cost, the other's their full width
+  const int64_t share = rows * a.top / a.experts + 1, want = a.maps ? 2 * share : share + share / 8;
+  return want <= 16 ? 16 : (int)std::min<int64_t>(256, (want + 31) / 32 * 32);
 }
 
 bool few_rows(const MoeArgs& a, int64_t rows) {
   auto ok = [](const WRef& w) { return (reinterpret_cast<uintptr_t>(w.data) & 15) == 0; };
   return rows <= 4 && (a.enc == E_BF16 || a.enc == E_F16) && a.width % 8 == 0 && a.ff % 8 == 0 && a.shared_ff % 8 == 0 && a.aligned &&
-         a.top < 64 && a.width * 4 <= 160 * 1024 && ((int64_t)a.top * a.ff + a.shared_ff) * 4 <= 160 * 1024 &&
+         a.top < 64 && a.width <= 32 * 1024 && (int64_t)a.top * a.ff + a.shared_ff <= 32 * 1024 &&
          (!a.shared_ff || (a.shared_gate.enc == a.enc && a.shared_up.enc == a.enc && a.shared_down.enc == a.enc && ok(a.shared_gate) &&
                            ok(a.shared_up) && ok(a.shared_down)));
 }
@@ -434,10 +432,13 @@ int launch_moe_few(const MoeArgs& a, const float* x, const void* norm_w, int nor
 }
 int launch_moe_few_down(const MoeArgs& a, int64_t rows, const float* z, const float* act, float* hidden, cudaStream_t st) {
   const auto kernel = a.enc == E_BF16 ? moe_down_kernel<true> : moe_down_kernel<false>;
-  const size_t smem = ((size_t)a.top * a.ff + a.shared_ff) * 4;
-  if (ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), 160 * 1024)) return 1;
-  const dim3 grid((unsigned)((a.width + MO_WARPS * MD_OUT - 1) / (MO_WARPS * MD_OUT)), (unsigned)rows);
-  DYN_CUDA(launch_pdl(kernel, grid, dim3(MO_THREADS), smem, st, a, z, act, hidden));
+  const int64_t total = (int64_t)a.top * a.ff + a.shared_ff, parts = (total / 8 + MD_SPAN - 1) / MD_SPAN;
+  const int64_t blocks = std::min<int64_t>(a.width, std::max(1, sm_count()));
+  const size_t smem = (size_t)(total + ((a.width + blocks - 1) / blocks) * parts) * 4;
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), 200 * 1024)) return 1;
+  DYN_CHECK(smem <= 200 * 1024, "mixture of experts: activations of %lld are too wide", (long long)total);
+  const dim3 grid((unsigned)blocks, (unsigned)rows);
+  DYN_CUDA(launch_pdl(kernel, grid, dim3(MD_THREADS), smem, st, a, z, act, hidden));
   count_launch();
   return 0;
 }
@@ -472,6 +473,17 @@ int launch_moe_experts(const MoeArgs& a, const float* xn, const __half* xh, cons
     }
     moe_gather_kernel<<<(unsigned)pairs, 256, 0, st>>>(a, p, xh, xinv, xg, inv_g);
     count_launch();
+    if (a.maps) {
+      // z sigmoid(1.702 z) > -0.17, so gated values are at most max(limit, 0.17) (limit + 1): scaled to at most 2^13
+      int e = 0;
+      frexpf(std::max(a.limit, 0.17f) * (a.limit + 1.0f), &e);
+      GroupedGemm up;
+      up.maps = a.maps, up.tiles = p.tiles, up.max_tiles = p.max_tiles, up.bn = p.bn, up.xh = xg, up.inv_s = inv_g;
+      up.M = pairs, up.N = a.ff, up.K = a.width, up.yh = xa, up.limit = a.limit, up.out_scale = ldexpf(1.0f, 13 - e);
+      GroupedGemm down = up;
+      down.xh = xa, down.N = a.width, down.K = a.ff, down.yh = nullptr, down.y = yo, down.inv_s = nullptr, down.in_scale = ldexpf(1.0f, e - 13);
+      return launch_grouped_gemm(up, st) || launch_grouped_gemm(down, st);
+    }
     TgGroups g;
     g.tiles = p.tiles, g.max_tiles = p.max_tiles, g.bn = p.bn;
     WRef w;

@@ -1206,7 +1206,7 @@ void dyninfer_cuda_session_destroy(dyninfer_cuda_session_t* s) {
                  s->hist_dev, s->hist_count_dev, s->argmax_scratch, s->mega_layers, s->io_dev,
                  s->prof_dev, s->trace_dev, s->prog_dev, s->ll_dev, s->batch_logits, s->batch_tokens_dev, s->tp_part, s->tp_logits,
                  s->tp_gather, s->scratch, s->qkv1, s->gu1, s->xh, s->xinv, s->gpart,
-                 s->lcache, s->state, s->mix_scratch, s->tables, s->expert_tables, s->want_logits, s->want_index_dev};
+                 s->xh2, s->xinv2, s->lcache, s->state, s->mix_scratch, s->tables, s->expert_tables, s->expert_maps, s->want_logits, s->want_index_dev};
   for (void* p : dev)
     if (p) cudaFree(p);
   if (s->logits_host) cudaFreeHost(s->logits_host);

@@ -130,6 +130,7 @@ struct dyninfer_cuda_session_t {
   size_t mix_scratch_floats = 0;
   float* tables = nullptr;       // decays, angles per position, norm weights counted from an offset
   const uint8_t** expert_tables = nullptr;  // addresses of the experts' matrices
+  uint8_t* expert_maps = nullptr;           // their tensor maps
   std::vector<int64_t> slot_pos;
   // logits of several rows of a portion
   float* want_logits = nullptr;  // [want_cap, vocab]
@@ -144,6 +145,8 @@ struct dyninfer_cuda_session_t {
   // K-split sums of o / down waiting for the residual + norm kernel
   __half* xh = nullptr;
   float *xinv = nullptr, *gpart = nullptr;
+  __half* xh2 = nullptr;  // a second operand, for layers whose branches read one residual row
+  float* xinv2 = nullptr;
   int64_t xh_rows = 0, xh_cols = 0;
   size_t gpart_bytes = 0;
   float *qkv1 = nullptr, *gu1 = nullptr;  // rows of [q | k | v] and of [gate | up] for the fused products

@@ -6,6 +6,7 @@
 // A layer may run with another layer's parameters; its cache and state are always its own. The steps,
 // graphs, batching and ABI around the layers are the session's (session.cu).
 #include <math.h>
+#include <string.h>
 
 #include "json_min.h"
 #include "session.cuh"
@@ -138,6 +139,58 @@ static int bind_experts(const ModelCfg& c, int l, const ParamTable& t, MixerLaye
   return 0;
 }
 
+// Experts the tile-copy GEMM takes: bf16 matrices become f16 in place when all of them, and the shared expert's, keep their
+// bits there (largest magnitude between 2^-8 and 2^15: nothing overflows, and what f16 drops below 2^-25 is less than 2^-17 of
+// it), then tensor maps of every matrix. That GEMM's gated values share one scale, set by the limit: wide limits stay out.
+static int prepare_experts(Session* s, MixerLayer* L, const std::vector<const uint8_t*>& host, size_t at, uint8_t* maps) {
+  MoeArgs& a = L->moe;
+  const int64_t count = (int64_t)a.ff * a.width, shared = (int64_t)a.shared_ff * a.width;
+  const int matrices = 3 * a.experts;
+  if (a.limit > 64.f) return 0;
+  if (a.exact || !a.aligned || !grouped_gemm_takes(a.ff, a.width) || !grouped_gemm_takes(a.width, a.ff)) return 0;
+  if (a.enc == E_BF16) {
+    WRef* own[4] = {&L->gate, &L->up, &L->down, &L->gate_up};
+    for (int i = 0; a.shared_ff && i < 3; i++)
+      if (own[i]->enc != E_BF16) return 0;
+    int* largest = nullptr;
+    const uint8_t** extra = nullptr;
+    const uint8_t* shared_host[3] = {L->gate.data, L->up.data, L->down.data};
+    if (dev_alloc(s, (void**)&largest, 256)) return 1;
+    extra = reinterpret_cast<const uint8_t**>(largest + 2);
+    DYN_CUDA(cudaMemset(largest, 0, 8));
+    DYN_CUDA(cudaMemcpy(extra, shared_host, sizeof(shared_host), cudaMemcpyHostToDevice));
+    int bits[2] = {0, 0};
+    if (bf16_table_range(a.table, matrices, count, largest, s->stream) ||
+        (a.shared_ff && bf16_table_range(extra, 3, shared, largest + 1, s->stream)))
+      return 1;
+    DYN_CUDA(cudaStreamSynchronize(s->stream));
+    DYN_CUDA(cudaMemcpy(bits, largest, sizeof(bits), cudaMemcpyDeviceToHost));
+    auto fits = [](int b) {
+      float v;
+      memcpy(&v, &b, 4);
+      return v >= 0x1p-8f && v <= 0x1p15f;
+    };
+    const bool ok = fits(bits[0]) && (!a.shared_ff || fits(bits[1]));
+    if (ok && (bf16_table_to_f16(a.table, matrices, count, s->stream) || (a.shared_ff && bf16_table_to_f16(extra, 3, shared, s->stream)))) return 1;
+    DYN_CUDA(cudaStreamSynchronize(s->stream));
+    dev_free(s, largest, 256);
+    if (!ok) return 0;
+    a.enc = E_F16;
+    for (WRef* w : own)
+      if (w->data) w->enc = E_F16;
+    a.shared_gate = L->gate, a.shared_up = L->up, a.shared_down = L->down;
+  }
+  if (a.enc != E_F16) return 0;
+  std::vector<uint8_t> blob((size_t)matrices * GROUPED_MAP_BYTES + 64);
+  uint8_t* p = blob.data() + (64 - reinterpret_cast<uintptr_t>(blob.data()) % 64) % 64;  // maps are made on 64-byte boundaries
+  for (int i = 0; i < matrices; i++)
+    if (make_grouped_weight_map(host[at + i], i % 3 == 2 ? a.width : a.ff, i % 3 == 2 ? a.ff : a.width, p + (size_t)i * GROUPED_MAP_BYTES))
+      return 1;
+  DYN_CUDA(cudaMemcpy(maps, p, (size_t)matrices * GROUPED_MAP_BYTES, cudaMemcpyHostToDevice));
+  a.maps = maps;
+  return 0;
+}
+
 int bind_mixers(Session* s, const ParamTable& t, uint64_t* decode_bytes) {
   const ModelCfg& c = s->cfg;
   const int64_t H = c.hidden;
@@ -245,8 +298,16 @@ int bind_mixers(Session* s, const ParamTable& t, uint64_t* decode_bytes) {
       if (L.norm2.ptr && derive_norm(s, &L.norm2, H, c.norm_offset, 1.f, s->tables + norm_at[l] + H)) return 1;
     }
   }
-  if (!addresses.empty())
+  if (!addresses.empty()) {
     DYN_CUDA(cudaMemcpy(s->expert_tables, addresses.data(), addresses.size() * sizeof(void*), cudaMemcpyHostToDevice));
+    if (dev_alloc(s, (void**)&s->expert_maps, addresses.size() * GROUPED_MAP_BYTES)) return 1;
+    for (int l = 0; l < c.layers; l++) {
+      MixerLayer& L = s->mix[l];
+      if (c.mixers[l].tensors != l || !L.moe.experts) continue;
+      const size_t at = L.moe.table - s->expert_tables;
+      if (prepare_experts(s, &L, addresses, at, s->expert_maps + at * GROUPED_MAP_BYTES)) return 1;
+    }
+  }
   // layers that run with another layer's parameters; state regions
   size_t off = 0;
   for (int l = 0; l < c.layers; l++) {
@@ -402,10 +463,12 @@ static int grow_mix_scratch(Session* s, int64_t rows, int64_t cap) {
 int configure_mixers(Session* s, int64_t rows) {
   const ModelCfg& c = s->cfg;
   int64_t proj = 0, ctx = 0, ff = 0;
+  bool beside = false;
   for (const MixerLayer& L : s->mix) {
     proj = std::max(proj, input_width(L));
     ctx = std::max(ctx, L.o.cols);
     ff = std::max<int64_t>(ff, L.c.gated_width());
+    beside = beside || (L.c.parallel && L.c.feeds_forward());
   }
   const int64_t wide = std::max({(int64_t)c.hidden, ctx, ff}), alloc = rows + rows / 2 + 64;
   if (dev_alloc(s, (void**)&s->hidden, (size_t)rows * c.hidden * 4) ||
@@ -415,6 +478,8 @@ int configure_mixers(Session* s, int64_t rows) {
       (!c.exact && rows >= 64 &&
        (dev_alloc(s, (void**)&s->xh, (size_t)alloc * wide * 2) || dev_alloc(s, (void**)&s->xinv, (size_t)alloc * 4) ||
         dev_alloc(s, (void**)&s->gpart, (size_t)8 * rows * c.hidden * 4))) ||
+      (!c.exact && rows >= 64 && beside &&
+       (dev_alloc(s, (void**)&s->xh2, (size_t)alloc * c.hidden * 2) || dev_alloc(s, (void**)&s->xinv2, (size_t)alloc * 4))) ||
       dev_alloc(s, (void**)&s->qkv1, (size_t)rows * proj * 4) ||
       dev_alloc(s, (void**)&s->gu1, (size_t)rows * 2 * std::max<int64_t>(1, ff) * 4) ||
       dev_alloc(s, (void**)&s->tokens_dev, (size_t)rows * 8) || dev_alloc(s, (void**)&s->row_pos_dev, (size_t)rows * 8) ||
@@ -508,7 +573,10 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
     return 0;
   };
   int pending = 0;  // K-split sums in gpart that `hidden` still lacks
-  auto norm = [&](const NormW& w) -> int {
+  const __half* operand = nullptr;  // what from_norm multiplies in the fused form, and its scales
+  const float* operand_inv = nullptr;
+  auto norm = [&](const NormW& w, const NormPair& pair = NormPair()) -> int {
+    operand = s->xh, operand_inv = s->xinv;
     if (stream) {
       form.norm_w = w.ptr, form.norm_type = w.type, form.eps = c.eps;
       return 0;
@@ -517,13 +585,14 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
     const int splits = pending;
     pending = 0;
     return splits > 1 ? launch_norm_prepare(nullptr, s->gpart, splits, s->hidden, s->hidden, w.ptr, w.type, rows, H, c.eps,
-                                            s->xh, s->xinv, st)
-                      : launch_norm_prepare(s->hidden, nullptr, 0, nullptr, nullptr, w.ptr, w.type, rows, H, c.eps, s->xh,
-                                            s->xinv, st);
+                                            s->xh, s->xinv, st, pair)
+                      : launch_norm_prepare(s->hidden, nullptr, 0, nullptr, pair.bias ? s->hidden : nullptr, w.ptr, w.type, rows, H,
+                                            c.eps, s->xh, s->xinv, st, pair);
   };
-  auto gemm = [&](const WRef& w, const float* x, float* y, const float* residual, bool defer) -> int {
+  // x == nullptr: the prepared operand
+  auto gemm = [&](const WRef& w, const float* x, const __half* xh, const float* xinv, float* y, const float* residual, bool defer) -> int {
     TgIo io;
-    if (!x) io.xh = s->xh, io.inv_s = s->xinv, io.rows_alloc = s->xh_rows;  // the prepared operand
+    if (!x) io.xh = xh, io.inv_s = xinv, io.rows_alloc = s->xh_rows;
     if (defer) io.partial = s->gpart, io.partial_bytes = s->gpart_bytes;
     bool handled = false;
     if (launch_dqgemm_tc(w, x, E_F32, rows, y, residual, st, &handled, &io)) return 1;
@@ -534,35 +603,47 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
   // a product of the normalised rows
   auto from_norm = [&](const WRef& w, float* y) -> int {
     if (stream) return streamed(w, s->hidden, y);
-    return fuse ? gemm(w, nullptr, y, nullptr, false) : session_linear(s, w, s->xn, E_F32, rows, y, nullptr);
+    return fuse ? gemm(w, nullptr, operand, operand_inv, y, nullptr, false) : session_linear(s, w, s->xn, E_F32, rows, y, nullptr);
   };
   // hidden += W x; `last`: no norm of this function follows to add deferred sums
   auto to_hidden = [&](const WRef& w, const float* x, bool prepared, bool last) -> int {
-    return fuse ? gemm(w, prepared ? nullptr : x, s->hidden, s->hidden, !last)
+    return fuse ? gemm(w, prepared ? nullptr : x, s->xh, s->xinv, s->hidden, s->hidden, !last)
                 : session_linear(s, w, x, E_F32, rows, s->hidden, s->hidden);
   };
   for (int l = 0; l < c.layers; l++) {
     const MixerLayer& L = s->mix[l];
     const bool final_layer = l + 1 == c.layers;
-    if (norm(L.norm1)) return 1;
+    const bool forward = L.c.feeds_forward();
+    const bool beside = L.c.parallel && forward;  // the feed-forward reads the residual as the mixer does
+    // many rows: both norms, and the output bias into the residual, in one launch; the mixer's output may then follow at once
+    const bool paired = beside && fuse && s->xh2;
+    NormPair pair;
+    if (paired) pair.w = L.norm2.ptr, pair.type = L.norm2.type, pair.xh = s->xh2, pair.inv_s = s->xinv2, pair.bias = L.ob.ptr, pair.bias_type = L.ob.type;
+    if (norm(L.norm1, pair)) return 1;
     float* y = s->qkv1;
     for (const WRef& w : L.in) {
       if (from_norm(w, y)) return 1;
       y += rows * w.rows;
     }
+    bool mixed_operand = false;  // the mixer's output is the operand in xh (the input products are done with it)
     int rc;
     switch (L.c.kind) {
       case MIX_RETENTION: rc = launch_retention(retention_args(s, L, rows), step, st); break;
       case MIX_RGLRU: rc = launch_rglru(rglru_args(s, L, rows), step, st); break;
       case MIX_SOFTMAX: rc = launch_softmax_attention(softmax_args(s, L, l, rows, cap), step, st); break;
-      case MIX_DELTA: rc = launch_delta(delta_args(s, L, rows), step, st); break;
+      case MIX_DELTA: {
+        DeltaArgs a = delta_args(s, L, rows);
+        mixed_operand = fuse && step.base >= 0 && delta_writes_operand(a) && (!beside || paired);
+        if (mixed_operand) a.xh = s->xh, a.xinv = s->xinv;
+        rc = launch_delta(a, step, st);
+        break;
+      }
       default: rc = launch_latent_attention(latent_args(s, L, l, rows, cap), step, st);
     }
     if (rc) return 1;
-    const bool forward = L.c.feeds_forward();
     // the mixer's output into the residual
     auto add_mixer = [&](bool last) -> int {
-      if (!L.ob.ptr) return to_hidden(L.o, s->ctx, false, last);
+      if (!L.ob.ptr || paired) return to_hidden(L.o, s->ctx, mixed_operand, last);
       if (stream && gemv_plain_takes(L.o, rows)) {
         GemvForm f;
         f.bias = L.ob.ptr, f.bias_type = L.ob.type;
@@ -571,10 +652,10 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
       }
       return to_hidden(L.o, s->ctx, false, last) || launch_add_bias(s->hidden, L.ob.ptr, L.ob.type, rows, H, st);
     };
-    const bool beside = L.c.parallel && forward;  // the feed-forward reads the residual as the mixer did
-    if (!beside && add_mixer(final_layer && !forward)) return 1;
+    if ((!beside || paired) && add_mixer(paired || (final_layer && !forward))) return 1;
     if (!forward) continue;
-    if (norm(L.norm2)) return 1;
+    if (paired) operand = s->xh2, operand_inv = s->xinv2;
+    else if (norm(L.norm2)) return 1;
     // products of the experts up to their outputs; the router's logits lie at the start of the scratch
     const MoeArgs moe = L.c.experts ? moe_args(s, L) : MoeArgs();
     float* const z = s->mix_scratch;
@@ -582,12 +663,12 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
       if (from_norm(L.router, z)) return 1;
       if (stream) {
         float* const act = moe_few_act(moe, rows);
-        if (launch_moe_few(moe, s->hidden, L.norm2.ptr, L.norm2.type, c.eps, rows, z, act, st) || (beside && add_mixer(true)) ||
+        if (launch_moe_few(moe, s->hidden, L.norm2.ptr, L.norm2.type, c.eps, rows, z, act, st) || (beside && !paired && add_mixer(true)) ||
             launch_moe_few_down(moe, rows, z, act, s->hidden, st))
           return 1;
         continue;
       }
-      if (launch_moe_experts(moe, fuse ? nullptr : s->xn, fuse ? s->xh : nullptr, s->xinv, rows, z, st)) return 1;
+      if (launch_moe_experts(moe, fuse ? nullptr : s->xn, fuse ? operand : nullptr, operand_inv, rows, z, st)) return 1;
     }
     const int64_t ff = L.c.gated_width();
     bool prepared = false;
@@ -611,7 +692,7 @@ int enqueue_mixer_layers(Session* s, int64_t rows, int64_t chunk_start, int64_t 
                        : launch_silu_mul(s->gu1, up, rows * ff, s->act, st)))
         return 1;
     }
-    if (beside && add_mixer(true)) return 1;
+    if (beside && !paired && add_mixer(true)) return 1;
     if (ff && to_hidden(L.down, s->act, prepared, final_layer)) return 1;
     if (L.c.experts && launch_moe_combine(moe, rows, s->hidden, st)) return 1;
   }

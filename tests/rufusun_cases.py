@@ -74,7 +74,11 @@ MECHANISMS = {
     "moe_many_experts": model([delta(mlp=moe(70, 2, 8))]),
     "moe_nothing_shared": model([delta(mlp=moe(6, 2, 20, shared=0))]),
     "moe_grouped": model([delta(heads=2, kv_heads=1, dim=16, vdim=16, mlp=moe(6, 2, 64, 1.1, 192))], width=128),
+    "moe_grouped_wide_limit": model([delta(heads=2, kv_heads=1, dim=16, vdim=16, mlp=moe(6, 2, 64, 900.0, 192, 1e6))], width=128),
+    "moe_grouped_narrow_limit": model([delta(heads=2, kv_heads=1, dim=16, vdim=16, mlp=moe(6, 2, 64, 0.03, 192, 0.01))], width=128),
     "moe_grouped_uneven": model([delta(heads=2, kv_heads=1, dim=16, vdim=16, mlp=moe(40, 7, 128, 1.1, 72))], width=256),
+    "odd_widths": model([delta(heads=3, kv_heads=1, dim=7, vdim=9, conv=4, mlp=moe(5, 2, 11, 1.0, 13)),
+                         attention(heads=3, kv_heads=3, dim=9, vdim=5, dims=6, mlp=dense(17))], width=33, vocab=67),
     "loop_of_one": model([delta(), attention(), delta(heads=2)], loop=span(1, 2, 3)),
     "loop_of_all": model([delta(mlp=dense(20)), attention()], loop=span(0, 2, 2)),
 }

@@ -418,7 +418,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_conv_wide_kernel(DeltaArgs a
           const float4& q = x[v][i + t];
           u[k] = fmaf(w[k][t], k == 0 ? q.x : k == 1 ? q.y : k == 2 ? q.z : q.w, u[k]);
         }
-        u[k] = silu_of(u[k]);
+        u[k] = __fdividef(u[k], 1.0f + __expf(-u[k]));  // silu
         ss[i] = fmaf(u[k], u[k], ss[i]);
       }
       y[v][i] = make_float4(u[0], u[1], u[2], u[3]);
@@ -505,15 +505,19 @@ __global__ void __launch_bounds__(DL_THREADS) delta_tokens_kernel(DeltaArgs a, i
     for (int c = lane; c < ne; c += 32) Sg[(int64_t)d * E + c] = S[d * per + c];
 }
 
-// rows x cols floats (16-byte aligned, cols % 4 == 0) into shared memory, zeros up to fill_rows x fill_cols
+// rows x cols floats (16-byte aligned, cols % 4 == 0) into shared memory, zeros up to fill_rows x fill_cols (at most 128)
 template <int THREADS = DL_THREADS>
 __device__ __forceinline__ void stage(float* dst, int pitch, const float* src, int64_t ld, int rows, int cols, int fill_rows,
                                       int fill_cols) {
-  const int q = fill_cols / 4;
-  for (int i = threadIdx.x; i < fill_rows * q; i += THREADS) {
-    const int r = i / q, c = (i - r * q) * 4;
+  const int c = (threadIdx.x & 31) * 4;  // a warp per row
+  if (c >= fill_cols) return;
+  int r = threadIdx.x >> 5;
+  const float* p = src + r * ld + c;
+  float* d = dst + r * pitch + c;
+#pragma unroll 4
+  for (; r < fill_rows; r += THREADS / 32, p += (THREADS / 32) * ld, d += (THREADS / 32) * pitch) {
     const bool live = r < rows && c < cols;
-    cp_async16(dst + r * pitch + c, live ? src + r * ld + c : src, live);
+    cp_async16(d, live ? p : src, live);
   }
 }
 __device__ __forceinline__ void load_a(AFrag& f, const float* p, int pitch) {  // rows g, g + 8; columns t4, t4 + 4

@@ -11,7 +11,7 @@
 //   o_t = sum_{s <= t, s in c} decay^{t-s} (q_t . k_s) v_s + decay^{t+1-first} P_c^T q_t, then norm and
 //   gate                                                   (retention_chunk_out_kernel)
 // Scores, decays and states are 32-bit quantities. Heads of up to 128 x 128 run these products on the tensor
-// cores with every f32 operand as a pair of tf32 terms (x = hi + lo to 2^-22; hi hi + hi lo + lo hi, the
+// cores with every f32 operand as a pair of tf32 terms (x = hi + lo to 2^-21; hi hi + hi lo + lo hi, the
 // "3xTF32" scheme of CUTLASS's examples); sessions that compute in f32 and other head sizes run them on the
 // vector pipes.
 #include <cooperative_groups.h>

@@ -1,4 +1,4 @@
-// f32 products on the tensor cores: every operand as a pair of tf32 terms (x = hi + lo to 2^-22; hi hi + hi lo +
+// f32 products on the tensor cores: every operand as a pair of tf32 terms (x = hi + lo to 2^-21; hi hi + hi lo +
 // lo hi, the "3xTF32" scheme of CUTLASS's examples), mma.sync m16n8k8 fragments.
 #pragma once
 
@@ -10,9 +10,10 @@ struct Tf32Pair {
   uint32_t hi, lo;
 };
 __device__ __forceinline__ Tf32Pair tf32_split(float x) {
+  // integer arithmetic on the bits (hi to nearest, lo cut off): conversions run at a fraction of its rate
   Tf32Pair p;
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(p.hi) : "f"(x));
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(p.lo) : "f"(x - __uint_as_float(p.hi)));
+  p.hi = (__float_as_uint(x) + 0x1000u) & 0xffffe000u;
+  p.lo = __float_as_uint(x - __uint_as_float(p.hi)) & 0xffffe000u;
   return p;
 }
 __device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {

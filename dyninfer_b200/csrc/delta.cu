@@ -17,7 +17,7 @@
 //     solve (I + A) u = beta v - beta b (K S_0), A_ts = beta_t b_t / b_s (k_t . k_s) for s < t. delta_chunk_kernel forms
 //     T = (I + A)^-1 by 16 x 16 blocks, U = T (beta v), W = T (beta b k) and P_ts = b_t / b_s (q_t . k_s) for every chunk at
 //     once; delta_scan_kernel walks the chunks: V = U - W S, o = b (Q S) + P V, S <- b_C S + (K b_C / b)^T V, a
-//     CTA per (head, 32 value columns): half of its warps hold the state in registers and form corrections and updates,
+//     CTA per (head, 32 or 16 value columns): half of its warps hold the state in registers and form corrections and updates,
 //     the other half the outputs. All products with pairs of tf32 terms.
 // delta_finish_kernel applies norm and gate to a portion's rows; delta_finish_operand_kernel leaves them as the dequant
 // GEMM's activation operand.
@@ -524,15 +524,17 @@ __device__ __forceinline__ void load_a(AFrag& f, const float* p, int pitch) {  /
   split_into(f, 0, p[0]), split_into(f, 1, p[8 * pitch]), split_into(f, 2, p[4]), split_into(f, 3, p[8 * pitch + 4]);
 }
 
-// Decays of a chunk: lane 0 .. 31 of one warp, two tokens each. Gd[t] = sum of log g through t.
-__device__ __forceinline__ void chunk_decay(const DeltaArgs& a, const float* gates, int64_t t0, int n, int h, double* Gd, float* beta) {
+// Decays of a chunk, by one warp, two tokens a lane: with G_t the sum of log g through t (in double, kept as two floats, so
+// that differences of large sums are exact), d = [G hi | G lo | beta | beta b_t | b_t | b_C / b_t] of 64 each, b_t = exp(G_t).
+__device__ __forceinline__ void chunk_decay(const DeltaArgs& a, const float* gates, int64_t t0, int n, int h, float* d) {
   const int lane = threadIdx.x & 31;
   double v[2];
+  float beta[2];
 #pragma unroll
   for (int i = 0; i < 2; i++) {
     const int t = 2 * lane + i;
     v[i] = t < n ? (double)gates[(t0 + t) * 2 * a.heads + a.heads + h] : 0.0;
-    if (beta) beta[t] = t < n ? gates[(t0 + t) * 2 * a.heads + h] : 0.f;
+    beta[i] = t < n ? gates[(t0 + t) * 2 * a.heads + h] : 0.f;
   }
   double s = v[0] + v[1];
 #pragma unroll
@@ -540,66 +542,73 @@ __device__ __forceinline__ void chunk_decay(const DeltaArgs& a, const float* gat
     const double other = __shfl_up_sync(0xffffffffu, s, o);
     if (lane >= o) s += other;
   }
-  Gd[2 * lane] = s - v[1], Gd[2 * lane + 1] = s;
+  const double last = __shfl_sync(0xffffffffu, s, 31);
+#pragma unroll
+  for (int i = 0; i < 2; i++) {
+    const int t = 2 * lane + i;
+    const double G = i ? s : s - v[1];
+    const float hi = (float)G, b = expf(hi);
+    d[t] = hi, d[DL_C + t] = (float)(G - (double)hi), d[2 * DL_C + t] = beta[i], d[3 * DL_C + t] = beta[i] * b;
+    d[4 * DL_C + t] = b, d[5 * DL_C + t] = expf((float)(last - G));
+  }
 }
 
 constexpr int DC_D = 128;                   // widest q/k head of the chunk kernels
 constexpr int DC_P = DC_D + 4, DC_S = DL_C + 4;
-constexpr int DC_SMEM = (2 * DL_C * DC_P + 2 * DL_C * DC_S) * 4 + DL_C * 8 + DL_C * 4;
+constexpr int DC_SMEM = (2 * DL_C * DC_P + 2 * DL_C * DC_S + 6 * DL_C) * 4;
 
+constexpr int DC_THREADS = 512;
 // W, U and P of one (chunk, head).
-__global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(DeltaArgs a, int64_t rows) {
+__global__ void __launch_bounds__(DC_THREADS, 2) delta_chunk_kernel(DeltaArgs a, int64_t rows) {
   extern __shared__ __align__(16) float dc_smem[];
   const DeltaScratch sc = carve(a, rows);
   float* ks = dc_smem;                 // [t][DC_P]
   float* qs = ks + DL_C * DC_P;        // [t][DC_P]; then blocks of v
   float* A = qs + DL_C * DC_P;         // [t][DC_S]
   float* T = A + DL_C * DC_S;          // [t][DC_S]
-  double* Gd = reinterpret_cast<double*>(T + DL_C * DC_S);
-  float* beta = reinterpret_cast<float*>(Gd + DL_C);
+  float* dec = T + DL_C * DC_S;        // decays
+  const float *beta = dec + 2 * DL_C, *beta_b = beta + DL_C;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
   const int D = a.dim, E = a.vdim, h = blockIdx.y, j = h / (a.heads / a.kv_heads);
   const int64_t c = blockIdx.x, t0 = c * DL_C, C = channels_of(a), qk = (int64_t)a.kv_heads * D;
   const int n = (int)min((int64_t)DL_C, rows - t0);
   const float* cv = sc.cv + t0 * C;
-  stage(ks, DC_P, cv + qk + (int64_t)j * D, C, n, D, DL_C, D);
-  stage(qs, DC_P, cv + (int64_t)j * D, C, n, D, DL_C, D);
+  stage<DC_THREADS>(ks, DC_P, cv + qk + (int64_t)j * D, C, n, D, DL_C, D);
+  stage<DC_THREADS>(qs, DC_P, cv + (int64_t)j * D, C, n, D, DL_C, D);
   cp_commit();
-  if (warp == 0) chunk_decay(a, sc.gates, t0, n, h, Gd, beta);
+  if (warp == 0) chunk_decay(a, sc.gates, t0, n, h, dec);
   cp_wait<0>();
   __syncthreads();
-  const int mt = warp & 3, nh = warp >> 2;   // 16 tokens x half of the keys (or of the columns)
+  const int mt = warp & 3, nq = warp >> 2;   // 16 tokens x a quarter of the keys (or of the columns)
   {
-    float s[4][4] = {}, p[4][4] = {};
+    float s[2][4] = {}, p[2][4] = {};
+    const int depth = nq <= mt ? D : 0;  // the other blocks' keys are all later than the tokens
 #pragma unroll 2
-    for (int d = 0; d < D; d += 8) {
+    for (int d = 0; d < depth; d += 8) {
       AFrag fk, fq;
       load_a(fk, ks + (16 * mt + g) * DC_P + d + t4, DC_P);
       load_a(fq, qs + (16 * mt + g) * DC_P + d + t4, DC_P);
-      Tf32Pair b0[4], b1[4];
+      Tf32Pair b0[2], b1[2];
 #pragma unroll
-      for (int nt = 0; nt < 4; nt++) {
-        const float* b = ks + (nh * 32 + 8 * nt + g) * DC_P + d + t4;
+      for (int nt = 0; nt < 2; nt++) {
+        const float* b = ks + (nq * 16 + 8 * nt + g) * DC_P + d + t4;
         b0[nt] = tf32_split(b[0]), b1[nt] = tf32_split(b[4]);
       }
-      mma3_split<4>(s, fk, b0, b1);
-      mma3_split<4>(p, fq, b0, b1);
+      mma3_split<2>(s, fk, b0, b1);
+      mma3_split<2>(p, fq, b0, b1);
     }
-    if (tid < DL_C) {
-      float* out = sc.decay + (c * a.heads + h) * 2 * DL_C;
-      out[tid] = expf((float)Gd[tid]), out[DL_C + tid] = expf((float)(Gd[DL_C - 1] - Gd[tid]));
-    }
+    if (tid < 2 * DL_C) sc.decay[(c * a.heads + h) * 2 * DL_C + tid] = dec[4 * DL_C + tid];
     float* P = sc.p + (c * a.heads + h) * DL_C * DL_C;
 #pragma unroll
-    for (int nt = 0; nt < 4; nt++)
+    for (int nt = 0; nt < 2; nt++)
 #pragma unroll
       for (int i = 0; i < 2; i++) {
-        const int t = 16 * mt + g + 8 * i, u = nh * 32 + 8 * nt + 2 * t4;
+        const int t = 16 * mt + g + 8 * i, u = nq * 16 + 8 * nt + 2 * t4;
         float2 pv;
         float av[2];
 #pragma unroll
         for (int e = 0; e < 2; e++) {
-          const float w = u + e <= t ? expf((float)(Gd[t] - Gd[u + e])) : 0.f;
+          const float w = u + e <= t ? expf((dec[t] - dec[u + e]) + (dec[DL_C + t] - dec[DL_C + u + e])) : 0.f;
           (e ? pv.y : pv.x) = p[nt][2 * i + e] * w;
           av[e] = u + e < t ? beta[t] * w * s[nt][2 * i + e] : 0.f;
         }
@@ -609,7 +618,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(DeltaArgs a, in
   }
   __syncthreads();
   // ---- T = (I + A)^-1. Diagonal blocks by forward substitution, thread = (block, column); qs is free
-  for (int i = tid; i < DL_C * DC_S; i += DL_THREADS) T[i] = 0.f;
+  for (int i = tid; i < DL_C * DC_S; i += DC_THREADS) T[i] = 0.f;
   __syncthreads();
   if (tid < DL_C) {
     const int b = tid & ~15, col = tid & 15;
@@ -629,16 +638,19 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(DeltaArgs a, in
   // blocks below: T_ij = -T_ii sum_{k = j .. i-1} A_ik T_kj, one block diagonal after the other
   {
     float* M = qs;  // [block][16][17]
-    const int rr = (tid >> 4) & 15, cc = tid & 15;
+    const int rr = (tid >> 4) & 15, cc = tid & 15, half = tid >> 8;  // two blocks at a time
     for (int dist = 1; dist < 4; dist++) {
-      for (int jb = 0; jb + dist < 4; jb++) {
+      for (int jb = half; jb + dist < 4; jb += 2) {
         const int ib = jb + dist;
         float v = 0.f;
-        for (int k = jb * 16; k < ib * 16; k++) v = fmaf(A[(ib * 16 + rr) * DC_S + k], T[k * DC_S + jb * 16 + cc], v);
+        for (int k0 = jb * 16; k0 < ib * 16; k0 += 16) {
+#pragma unroll
+          for (int k = k0; k < k0 + 16; k++) v = fmaf(A[(ib * 16 + rr) * DC_S + k], T[k * DC_S + jb * 16 + cc], v);
+        }
         M[jb * 272 + rr * 17 + cc] = v;
       }
       __syncthreads();
-      for (int jb = 0; jb + dist < 4; jb++) {
+      for (int jb = half; jb + dist < 4; jb += 2) {
         const int ib = jb + dist;
         float v = 0.f;
 #pragma unroll
@@ -648,22 +660,22 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(DeltaArgs a, in
       __syncthreads();
     }
   }
-  // ---- U = T (beta v), W = T (beta b k): 64 rows x up to 128 columns at a time, a warp 16 rows x half of them
-  auto product = [&](const float* B, int cols, bool decay, float* out, int64_t ld) {
-    float acc[8][4] = {};
+  // ---- U = T (beta v), W = T (beta b k): 64 rows x up to 128 columns at a time, a warp 16 rows x a quarter of them
+  auto product = [&](const float* B, int cols, const float* w, float* out, int64_t ld) {
+    float acc[4][4] = {};
     for (int k = 0; k < 16 * (mt + 1); k += 8) {  // T is lower triangular
       AFrag f;
       load_a(f, T + (16 * mt + g) * DC_S + k + t4, DC_S);
       const int ka = k + t4, kb = ka + 4;
-      const float wa = decay ? beta[ka] * expf((float)Gd[ka]) : beta[ka], wb = decay ? beta[kb] * expf((float)Gd[kb]) : beta[kb];
-      mma3<8>(acc, f, [&](int nt, int half) {
-        const int col = nh * 64 + 8 * nt + g;
+      const float wa = w[ka], wb = w[kb];
+      mma3<4>(acc, f, [&](int nt, int half) {
+        const int col = nq * 32 + 8 * nt + g;
         return col < cols ? (half ? wb * B[kb * DC_P + col] : wa * B[ka * DC_P + col]) : 0.f;
       });
     }
 #pragma unroll
-    for (int nt = 0; nt < 8; nt++) {
-      const int col = nh * 64 + 8 * nt + 2 * t4;
+    for (int nt = 0; nt < 4; nt++) {
+      const int col = nq * 32 + 8 * nt + 2 * t4;
       if (col >= cols) continue;
 #pragma unroll
       for (int i = 0; i < 2; i++)
@@ -673,26 +685,29 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(DeltaArgs a, in
   for (int e0 = 0; e0 < E; e0 += DC_D) {
     const int cols = min(DC_D, E - e0);
     if (e0) __syncthreads();
-    stage(qs, DC_P, cv + 2 * qk + (int64_t)h * E + e0, C, n, cols, DL_C, cols);
+    stage<DC_THREADS>(qs, DC_P, cv + 2 * qk + (int64_t)h * E + e0, C, n, cols, DL_C, cols);
     cp_commit();
-    if (e0 == 0) product(ks, D, true, sc.w + (c * a.heads + h) * DL_C * (int64_t)D, D);
+    if (e0 == 0) product(ks, D, beta_b, sc.w + (c * a.heads + h) * DL_C * (int64_t)D, D);
     cp_wait<0>();
     __syncthreads();
-    product(qs, cols, false, sc.u + (c * a.heads + h) * DL_C * (int64_t)E + e0, E);
+    product(qs, cols, beta, sc.u + (c * a.heads + h) * DL_C * (int64_t)E + e0, E);
   }
 }
 
-constexpr int DS_N = 32;                       // value columns per CTA
 constexpr int DS_THREADS = 512;                // warps 0-7: corrections and state; 8-15: outputs
-constexpr int DS_B = DS_N + 8;                 // pitch of the split operands: conflict-free B fragments
 constexpr int DS_KP = DC_D + 8;
-constexpr int DS_SMEM = (2 * DL_C * DC_P + DL_C * DS_KP + DL_C * DC_S + 2 * DC_D * DS_B + 2 * DL_C * DS_B + 4 * DL_C) * 4;
+constexpr int ds_pitch(int n) { return n % 16 == 8 ? n : n + 8; }  // of the split operands: conflict-free B fragments
+constexpr int ds_smem(int n) {
+  return (2 * DL_C * DC_P + DL_C * DS_KP + DL_C * DC_S + 2 * DC_D * ds_pitch(n) + 2 * DL_C * ds_pitch(n) + 4 * DL_C) * 4;
+}
 
-// The walk over the chunks for one (value slice, head).
+// The walk over the chunks for one (slice of 16 NT value columns, head).
+template <int NT>
 __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a, int64_t rows, int64_t base, int64_t slot) {
-  extern __shared__ __align__(16) float ds_smem[];
+  constexpr int DS_N = 16 * NT, DS_B = ds_pitch(DS_N);
+  extern __shared__ __align__(16) float dn_smem[];
   const DeltaScratch sc = carve(a, rows);
-  float* Ws = ds_smem;                    // [t][DC_P]
+  float* Ws = dn_smem;                    // [t][DC_P]
   float* Qs = Ws + DL_C * DC_P;           // [t][DC_P]
   float* Ks = Qs + DL_C * DC_P;           // [t][DS_KP]
   float* Ps = Ks + DL_C * DS_KP;          // [t][DC_S]
@@ -722,16 +737,16 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a, int
   stage_wq(0);
   stage_kp(0);
   keep_inputs(a, rows, base, slot, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
-  const int mt = warp & 3, nh = (warp >> 2) & 1;  // 16 tokens x 16 value columns
+  const int mt = warp & 3, nh = (warp >> 2) & 1;  // 16 tokens x half of the value columns
   const bool states = warp < 8;
   // warps 0-7: 16 rows of the state as accumulators
   float* Sg = a.state + ((slot * a.heads + h) * D) * (int64_t)E + e0;
   const int d0 = 16 * (warp & 7);
   const bool owns = states && d0 < D;
-  float S[4][4] = {};
+  float S[2 * NT][4] = {};
   if (owns && base > 0) {
 #pragma unroll
-    for (int nt = 0; nt < 4; nt++)
+    for (int nt = 0; nt < 2 * NT; nt++)
 #pragma unroll
       for (int i = 0; i < 4; i++) {
         const int d = d0 + g + 8 * (i >> 1), e = 8 * nt + 2 * t4 + (i & 1);
@@ -740,7 +755,7 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a, int
   }
   auto publish = [&]() {
 #pragma unroll
-    for (int nt = 0; nt < 4; nt++)
+    for (int nt = 0; nt < 2 * NT; nt++)
 #pragma unroll
       for (int i = 0; i < 4; i += 2) {
         const int d = d0 + g + 4 * i, e = 8 * nt + 2 * t4;
@@ -750,14 +765,14 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a, int
       }
   };
   if (owns) publish();
-  float uv[2][4] = {};  // U of the warp's tile, fetched a chunk ahead
+  float uv[NT][4] = {};  // U of the warp's tile, fetched a chunk ahead
   auto fetch_u = [&](int c) {
     const float* U = sc.u + ((int64_t)c * a.heads + h) * DL_C * E + e0;
 #pragma unroll
-    for (int nt = 0; nt < 2; nt++)
+    for (int nt = 0; nt < NT; nt++)
 #pragma unroll
       for (int i = 0; i < 2; i++) {
-        const int t = 16 * mt + g + 8 * i, e = nh * 16 + 8 * nt + 2 * t4;
+        const int t = 16 * mt + g + 8 * i, e = nh * 8 * NT + 8 * nt + 2 * t4;
         const float2 v = e0 + e < E ? *reinterpret_cast<const float2*>(U + t * (int64_t)E + e) : make_float2(0.f, 0.f);
         uv[nt][2 * i] = v.x, uv[nt][2 * i + 1] = v.y;
       }
@@ -775,25 +790,25 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a, int
     cp_wait<1>();
     __syncthreads();  // W, Q, the decays and the state's terms are there
     // ---- W S, Q S
-    float acc[2][4] = {};
+    float acc[NT][4] = {};
     {
       const float* A = (states ? Ws : Qs) + (16 * mt + g) * DC_P + t4;
 #pragma unroll 4
       for (int d = 0; d < D; d += 8) {
         AFrag f;
         load_a(f, A + d, DC_P);
-        Tf32Pair b0[2], b1[2];
+        Tf32Pair b0[NT], b1[NT];
 #pragma unroll
-        for (int nt = 0; nt < 2; nt++) split_at(Sh, Sl, d, nh * 16 + 8 * nt + g, b0[nt], b1[nt]);
-        mma3_split<2>(acc, f, b0, b1);
+        for (int nt = 0; nt < NT; nt++) split_at(Sh, Sl, d, nh * 8 * NT + 8 * nt + g, b0[nt], b1[nt]);
+        mma3_split<NT>(acc, f, b0, b1);
       }
     }
     if (states) {
 #pragma unroll
-      for (int nt = 0; nt < 2; nt++)
+      for (int nt = 0; nt < NT; nt++)
 #pragma unroll
         for (int i = 0; i < 4; i += 2) {
-          const int t = 16 * mt + g + 4 * i, e = nh * 16 + 8 * nt + 2 * t4;
+          const int t = 16 * mt + g + 4 * i, e = nh * 8 * NT + 8 * nt + 2 * t4;
           const Tf32Pair p = tf32_split(uv[nt][i] - acc[nt][i]), q = tf32_split(uv[nt][i + 1] - acc[nt][i + 1]);
           *reinterpret_cast<float2*>(Vh + t * DS_B + e) = make_float2(__uint_as_float(p.hi), __uint_as_float(q.hi));
           *reinterpret_cast<float2*>(Vl + t * DS_B + e) = make_float2(__uint_as_float(p.lo), __uint_as_float(q.lo));
@@ -808,7 +823,7 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a, int
       const float full = bt[DL_C - 1];
       const bool second = d0 + 8 < D;
 #pragma unroll
-      for (int nt = 0; nt < 4; nt++)
+      for (int nt = 0; nt < 2 * NT; nt++)
 #pragma unroll
         for (int i = 0; i < 4; i++) S[nt][i] *= full;
 #pragma unroll 2
@@ -818,25 +833,25 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a, int
         AFrag f;
         split_into(f, 0, ka[0] * wa), split_into(f, 1, second ? ka[8] * wa : 0.f);
         split_into(f, 2, kb[0] * wb), split_into(f, 3, second ? kb[8] * wb : 0.f);
-        Tf32Pair b0[4], b1[4];
+        Tf32Pair b0[2 * NT], b1[2 * NT];
 #pragma unroll
-        for (int nt = 0; nt < 4; nt++) split_at(Vh, Vl, k, 8 * nt + g, b0[nt], b1[nt]);
-        mma3_split<4>(S, f, b0, b1);
+        for (int nt = 0; nt < 2 * NT; nt++) split_at(Vh, Vl, k, 8 * nt + g, b0[nt], b1[nt]);
+        mma3_split<2 * NT>(S, f, b0, b1);
       }
       publish();
     } else if (!states) {
       // ---- o = b Q S + P V (P is lower triangular)
       const float w0 = bt[16 * mt + g], w1 = bt[16 * mt + g + 8];
 #pragma unroll
-      for (int nt = 0; nt < 2; nt++) acc[nt][0] *= w0, acc[nt][1] *= w0, acc[nt][2] *= w1, acc[nt][3] *= w1;
+      for (int nt = 0; nt < NT; nt++) acc[nt][0] *= w0, acc[nt][1] *= w0, acc[nt][2] *= w1, acc[nt][3] *= w1;
 #pragma unroll 2
       for (int k = 0; k < 16 * (mt + 1); k += 8) {
         AFrag f;
         load_a(f, Ps + (16 * mt + g) * DC_S + k + t4, DC_S);
-        Tf32Pair b0[2], b1[2];
+        Tf32Pair b0[NT], b1[NT];
 #pragma unroll
-        for (int nt = 0; nt < 2; nt++) split_at(Vh, Vl, k, nh * 16 + 8 * nt + g, b0[nt], b1[nt]);
-        mma3_split<2>(acc, f, b0, b1);
+        for (int nt = 0; nt < NT; nt++) split_at(Vh, Vl, k, nh * 8 * NT + 8 * nt + g, b0[nt], b1[nt]);
+        mma3_split<NT>(acc, f, b0, b1);
       }
 #pragma unroll
       for (int i = 0; i < 2; i++) {
@@ -844,8 +859,8 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a, int
         if (t >= n) continue;
         float* out = a.out + (t0 + t) * (int64_t)a.heads * E + (int64_t)h * E + e0;
 #pragma unroll
-        for (int nt = 0; nt < 2; nt++) {
-          const int e = nh * 16 + 8 * nt + 2 * t4;
+        for (int nt = 0; nt < NT; nt++) {
+          const int e = nh * 8 * NT + 8 * nt + 2 * t4;
           if (e0 + e < E) *reinterpret_cast<float2*>(out + e) = make_float2(acc[nt][2 * i], acc[nt][2 * i + 1]);
         }
       }
@@ -855,7 +870,7 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a, int
   }
   if (!owns) return;
 #pragma unroll
-  for (int nt = 0; nt < 4; nt++)
+  for (int nt = 0; nt < 2 * NT; nt++)
 #pragma unroll
     for (int i = 0; i < 4; i++) {
       const int d = d0 + g + 8 * (i >> 1), e = 8 * nt + 2 * t4 + (i & 1);
@@ -951,12 +966,15 @@ int launch_delta(const DeltaArgs& a, const StepRows& r, cudaStream_t st) {
   conv<<<grid, DL_THREADS, 0, st>>>(a, r.rows, r.base, r.slot);
   if (chunk_shape(a, r.rows)) {
     const unsigned nc = (unsigned)((r.rows + DL_C - 1) / DL_C);
+    // narrow slices where wide ones would leave half of the GPU idle: the walk's time is its latency then
+    const bool narrow = 2 * a.heads * ((a.vdim + 31) / 32) <= std::max(1, sm_count());
+    const auto scan = narrow ? delta_scan_kernel<1> : delta_scan_kernel<2>;
+    const int cols = narrow ? 16 : 32, smem = ds_smem(cols);
     if (ensure_dynamic_smem(reinterpret_cast<const void*>(delta_chunk_kernel), DC_SMEM) ||
-        ensure_dynamic_smem(reinterpret_cast<const void*>(delta_scan_kernel), DS_SMEM))
+        ensure_dynamic_smem(reinterpret_cast<const void*>(scan), smem))
       return 1;
-    delta_chunk_kernel<<<dim3(nc, (unsigned)a.heads), DL_THREADS, DC_SMEM, st>>>(a, r.rows);
-    delta_scan_kernel<<<dim3((unsigned)((a.vdim + DS_N - 1) / DS_N), (unsigned)a.heads), DS_THREADS, DS_SMEM, st>>>(
-        a, r.rows, r.base, r.slot);
+    delta_chunk_kernel<<<dim3(nc, (unsigned)a.heads), DC_THREADS, DC_SMEM, st>>>(a, r.rows);
+    scan<<<dim3((unsigned)((a.vdim + cols - 1) / cols), (unsigned)a.heads), DS_THREADS, smem, st>>>(a, r.rows, r.base, r.slot);
     count_launch(2);
   } else {
     int nsplit = std::max(1, (a.vdim + 31) / 32);

@@ -727,12 +727,12 @@ attention_merge_kernel(const float* __restrict__ part, int nsplit, float* ctx, i
   __syncthreads();
   for (int64_t idx = threadIdx.x; idx < d; idx += blockDim.x) {
     float o = 0.f, gl = 0.f;
-    for (int s0 = 0; s0 < nsplit; s0 += 8) {  // eight slices' loads in flight
-      float v[8];
+    for (int s0 = 0; s0 < nsplit; s0 += 32) {  // 32 slices' loads in flight
+      float v[32];
 #pragma unroll
-      for (int j = 0; j < 8; j++) v[j] = s0 + j < nsplit ? p0[(s0 + j) * (d + 2) + idx] : 0.f;
+      for (int j = 0; j < 32; j++) v[j] = s0 + j < nsplit ? p0[(s0 + j) * (d + 2) + idx] : 0.f;
 #pragma unroll
-      for (int j = 0; j < 8; j++)
+      for (int j = 0; j < 32; j++)
         if (s0 + j < nsplit) o += v[j] * s_w[s0 + j], gl += s_l[s0 + j] * s_w[s0 + j];
     }
     ctx[r * nh * d + h * d + idx] = o / gl;

@@ -49,7 +49,7 @@ def rufusun_doc(size: str) -> dict:
     moe = {"kind": "moe", "expert": {"ff": ff // 6, "limit": 7.0}, "router": {"experts": 16, "top": 4},
            "shared": {"ff": ff // 3, "limit": 7.0}}
     delta = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}
-    attention = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+    attention = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
                  "rot": {"dims": 128, "base": 5e5}}
     kinds = [{"type": t, "mixer": m, "mlp": f} for f in (dense, moe) for t, m in (("delta", delta), ("attention", attention))]
     return {"layers": [kinds[i % 4] for i in range(layers)], "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6},

@@ -62,7 +62,7 @@ MECHANISMS = {
     "delta": model([delta()]),
     "delta_one_tap": model([delta(heads=3, kv_heads=3, dim=8, vdim=36, conv=1)]),
     "delta_many_taps": model([delta(heads=5, kv_heads=1, dim=20, vdim=12, conv=7)]),
-    "delta_chunks": model([delta(heads=6, kv_heads=3, dim=64, vdim=32, conv=4)], width=64),
+    "delta_chunks": model([delta(heads=6, kv_heads=2, dim=48, vdim=40, conv=4)], width=64),
     "delta_chunks_uneven": model([delta(heads=2, kv_heads=2, dim=40, vdim=72, conv=2)], width=64),
     "delta_chunks_wide": model([delta(heads=2, kv_heads=1, dim=128, vdim=136, conv=6)], width=64),
     "delta_wide_keys": model([delta(heads=2, kv_heads=1, dim=200, vdim=48, conv=4)], width=64),

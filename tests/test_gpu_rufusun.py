@@ -115,6 +115,21 @@ def test_batches_of_unequal_requests_and_reused_slots(native_lib, tmp_path, doc,
         assert len({slot for _, slot in order}) == slots and len(order) == len(lengths)
 
 
+@pytest.mark.parametrize("slots", [20, 70])
+@pytest.mark.parametrize("doc", [cases.mixed(), cases.fast()], ids=["odd_sizes", "fast_paths"])
+def test_wide_decode_steps(native_lib, tmp_path, doc, slots):
+    """Steps of as many rows as the many-row products take: every slot at a position of its own."""
+    seqs = [cases.tokens(4 + i % 5, doc["vocab"], seed=60 + i) for i in range(slots)]
+    want = [evaluate(doc, q) for q in seqs]
+    with load(tmp_path, doc, "serve", chunk=128).create_batched_session(SessionConfig(256, batch_size=slots)) as s:
+        for i, q in enumerate(seqs):
+            s.extend_slot(i, q[:-3], restart=True)
+        for back in (3, 2, 1):
+            _, lg = s.step({i: q[len(q) - back] for i, q in enumerate(seqs)}, want_logits=True)
+            for i, q in enumerate(seqs):
+                assert_close(lg[i][None], want[i][len(q) - back][None], "serve")
+
+
 def test_prompt_between_other_slots_decoding(native_lib, tmp_path):
     """A prompt's portions alternate with decode steps of other slots: neither disturbs the other."""
     doc = cases.fast()
@@ -162,7 +177,7 @@ def test_experts_of_any_range(native_lib, tmp_path, scale):
 def far_key_model(dim, vdim, heads, kv_heads):
     """One attention layer whose queries of token 1 match the key of token 2 alone, by a wide margin, in the dims that
     are not rotated."""
-    doc = cases.model([cases.attention(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, dims=8, scale=0.02, softcap=50.0)], width=64,
+    doc = cases.model([cases.attention(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, dims=8, scale=0.02, softcap=45.0)], width=64,
                       vocab=40, logit_scale=1.0)
     t = cases.weights(doc, 3)
     for name in ("l0.norm1", "final.norm"):
